@@ -1,4 +1,5 @@
-"""ctypes binding of libglorcq_b200.so (the C ABI declared in include/glorcq_b200.h).
+"""ctypes bindings of libglorcq_b200.so (the C ABI declared in include/glorcq_b200.h) and of
+libglorcq_b200_dense.so (include/glorcq_b200_dense.h, the unquantized decoders; built at first use).
 
 There is no fallback: if the library is missing, or a call returns a non-zero status, a
 RuntimeError is raised -- the same exception type the reference's native modules raise through
@@ -120,7 +121,95 @@ _SIGS = {
                                      vp, vp, vp, vp, C.POINTER(MoeEp)]),
 }
 
+
+# ---- unquantized decoders -----------------------------------------------------------------------------
+DT_BF16, DT_F32 = 0, 1
+ACT_NONE, ACT_RELU2, ACT_GELU_ERF = 0, 1, 2
+
+
+class DenseMM(C.Structure):
+    """glq_dense_mm_t"""
+    _fields_ = [(f, C.c_int32) for f in ("dtype", "act", "N", "K", "rows", "n_matrices", "max_slots", "max_slot_rows", "split")] + \
+               [("alpha", C.c_float)] + [(f, vp) for f in ("slot_index", "n_slots", "slot_count", "slot_offset", "entry_row", "x")] + \
+               [("ldx", C.c_int64), ("W", vp), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp)]
+
+
+class MLstm(C.Structure):
+    """glq_mlstm_t"""
+    _fields_ = [(f, C.c_int32) for f in ("dtype", "B", "T", "H", "D", "V", "state_idle")] + \
+               [("gate_cap", C.c_float), ("eps", C.c_float), ("qkvg", vp), ("ldp", C.c_int64), ("gates", vp), ("ldg", C.c_int64)] + \
+               [(f, vp) for f in ("bias_i", "bias_f", "norm_w", "S", "n", "m", "out", "workspace")] + \
+               [("workspace_bytes", C.c_size_t), ("counters", vp)]
+
+
+class Latent(C.Structure):
+    """glq_latent_t"""
+    _fields_ = [(f, C.c_int32) for f in ("dtype", "B", "T", "H", "D", "R", "V", "K", "rot_dims", "max_len")] + \
+               [("scale", C.c_float), ("eps", C.c_float), ("start", vp), ("q", vp), ("ldq", C.c_int64), ("ckr", vp),
+                ("ldk", C.c_int64)] + [(f, vp) for f in ("gate", "norm_w", "cos_t", "sin_t", "cache")] + \
+               [("ldc", C.c_int64)] + [(f, vp) for f in ("ukt", "uv", "out", "kv")] + \
+               [("ldkv", C.c_int64), ("S", C.c_int32), ("max_splits", C.c_int32), ("workspace", vp), ("workspace_bytes", C.c_size_t)]
+
+
+class Route(C.Structure):
+    """glq_route_t"""
+    _fields_ = [(f, C.c_int32) for f in ("n", "E", "identity", "top", "chunk", "reserved")] + [("logits", vp), ("ldl", C.c_int64)] + \
+               [(f, vp) for f in ("correction", "sel", "wts", "entry_scale", "tok_entries", "entry_row", "active", "slot_count",
+                                  "slot_offset", "n_active")] + \
+               [("max_slots", C.c_int32), ("reserved2", C.c_int32), ("block_counts", vp)]
+
+
+_i, _f, _l, _z = C.c_int, C.c_float, C.c_int64, C.c_size_t
+_DENSE_SIGS = {
+    "glq_dense_status_string": (C.c_char_p, [_i]),
+    "glq_dense_last_cuda_error": (_i, []),
+    "glq_dense_debug_error": (_i, [vp, _i]),
+    "glq_dense_matmul": (_i, [C.POINTER(DenseMM), vp]),
+    "glq_dense_matmul_path": (_i, [C.POINTER(DenseMM)]),
+    "glq_dense_embed": (_i, [_i, vp, vp, _i, _i, _i, vp, vp, vp]),
+    "glq_dense_add_norm": (_i, [_i, vp, vp, vp, _f, _i, _i, vp, vp, vp]),
+    "glq_mlstm_slices": (_i, [_i]),
+    "glq_mlstm_workspace_bytes": (_z, [C.POINTER(MLstm), _i]),
+    "glq_mlstm_step": (_i, [C.POINTER(MLstm), vp]),
+    "glq_mlstm_chunk": (_i, [C.POINTER(MLstm), vp]),
+    "glq_latent_prep": (_i, [C.POINTER(Latent), vp]),
+    "glq_latent_absorbed_workspace_bytes": (_z, [C.POINTER(Latent)]),
+    "glq_latent_absorbed": (_i, [C.POINTER(Latent), vp]),
+    "glq_latent_prefill_supported": (_i, [C.POINTER(Latent)]),
+    "glq_latent_prefill": (_i, [C.POINTER(Latent), vp]),
+    "glq_route_max_slots": (_i, [_i, _i, _i, _i]),
+    "glq_route": (_i, [C.POINTER(Route), vp]),
+    "glq_dense_combine_norm": (_i, [_i, vp, _l, vp, vp, _i, vp, vp, _f, _i, _i, vp, vp, vp]),
+    "glq_dense_head_workspace_bytes": (_z, []),
+    "glq_dense_head": (_i, [vp, _l, vp, _i, _i, _i, _f, vp, _l, vp, vp, _z, vp, vp]),
+}
+
 _lib = None
+_dense = None
+
+
+def dense():
+    """The library of the unquantized decoders, compiled first when it is missing or older than its sources."""
+    global _dense
+    if _dense is None:
+        from . import _build
+        L = C.CDLL(_build.build(lib=_build.DENSE_LIB))
+        for name, (res, args) in _DENSE_SIGS.items():
+            fn = getattr(L, name)
+            fn.restype, fn.argtypes = res, args
+        _dense = L
+    return _dense
+
+
+def dense_symbols():
+    return list(_DENSE_SIGS.keys())
+
+
+def check_dense(status: int, what: str):
+    if status != 0:
+        L = dense()
+        extra = f" (cudaError {L.glq_dense_last_cuda_error()})" if status == -4 else ""
+        raise RuntimeError(f"{what}: {L.glq_dense_status_string(status).decode()}{extra}")
 
 
 def lib():

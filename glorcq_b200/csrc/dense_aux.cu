@@ -1,0 +1,268 @@
+// Row kernels of the unquantized decoders: embedding, residual add with the layer norm of the sublayer's output,
+// softmax routing with a correction term and its entry lists, and the weighted sum of the experts' outputs fused with
+// the norm and the residual add that follow it.  One CTA per row; the residual stream and all statistics are float.
+#include "dense_common.cuh"
+#include "moe_plan.cuh"
+
+namespace glq {
+
+constexpr int kRowThreads = 256;
+constexpr int kMaxC = 32768;          // row length; a row is staged in shared memory as float
+
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads) dense_embed_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table,
+                                                                  int C, int vocab, float* __restrict__ x, T* __restrict__ h) {
+    pdl_wait();
+    pdl_release();
+    const size_t row = blockIdx.x;
+    long long id = ids[row];
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    for (int c = threadIdx.x; c < C; c += kRowThreads) {
+        const T v = table[(size_t)id * C + c];
+        x[row * C + c] = to_f(v);
+        h[row * C + c] = v;
+    }
+}
+
+// ys: the sublayer's output row.  x += norm(ys) * w; h = x, or norm(x) * final_w
+template <typename T>
+__device__ __forceinline__ void norm_add_row(float* ys, float* red, const float* __restrict__ w, const float* __restrict__ fw,
+                                             float eps, int C, float* __restrict__ x, T* __restrict__ h) {
+    float s = 0.f;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) s += ys[c];
+    const float mean = block_sum(s, red) / C;
+    s = 0.f;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) {
+        const float d = ys[c] - mean;
+        s += d * d;
+    }
+    const float inv = 1.f / sqrtf(block_sum(s, red) / C + eps);
+    for (int c = threadIdx.x; c < C; c += kRowThreads) {
+        const float v = x[c] + (ys[c] - mean) * inv * w[c];
+        x[c] = v;
+        ys[c] = v;
+        if (!fw) h[c] = from_f<T>(v);
+    }
+    if (!fw) return;
+    s = 0.f;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) s += ys[c];
+    const float mean2 = block_sum(s, red) / C;
+    s = 0.f;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) {
+        const float d = ys[c] - mean2;
+        s += d * d;
+    }
+    const float inv2 = 1.f / sqrtf(block_sum(s, red) / C + eps);
+    for (int c = threadIdx.x; c < C; c += kRowThreads) h[c] = from_f<T>((ys[c] - mean2) * inv2 * fw[c]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads) dense_add_norm_kernel(const float* __restrict__ y, const float* __restrict__ w,
+                                                                     const float* __restrict__ fw, float eps, int C,
+                                                                     float* __restrict__ x, T* __restrict__ h) {
+    extern __shared__ float ys[];
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_release();
+    const size_t o = (size_t)blockIdx.x * C;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) ys[c] = y[o + c];
+    norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
+}
+
+// experts' outputs of a token in slot order; a slot without an entry passes the layer's input through
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads) dense_combine_norm_kernel(const T* __restrict__ eo, long long lde,
+                                                                         const int* __restrict__ tok_entries,
+                                                                         const float* __restrict__ wts, int top,
+                                                                         const float* __restrict__ w, const float* __restrict__ fw,
+                                                                         float eps, int C, float* __restrict__ x, T* __restrict__ h) {
+    extern __shared__ float ys[];
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_release();
+    const size_t row = blockIdx.x, o = row * C;
+    for (int c = threadIdx.x; c < C; c += kRowThreads) {
+        float a = 0.f;
+        for (int j = 0; j < top; ++j) {
+            const int e = tok_entries[row * top + j];
+            a += wts[row * top + j] * (e >= 0 ? to_f(eo[(size_t)e * lde + c]) : x[o + c]);
+        }
+        ys[c] = a;
+    }
+    norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
+}
+
+// ---- routing -------------------------------------------------------------------------------------------
+struct RtParams {
+    const float* logits;
+    const float* correction;
+    long long ldl;
+    int n, E, A, top, chunk;      // A: experts and pass-through experts
+    int* sel;
+    float* wts;
+    float* entry_scale;
+    int* tok_entries;
+    int* entry_row;
+    int* active;
+    int* slot_count;
+    int* slot_offset;
+    int* n_active;
+    int max_slots;
+};
+
+// one token by one warp: s = softmax(logits); `top` times the largest remaining s + correction, lowest index on ties.
+// sc: A floats of shared memory of this warp
+__device__ __forceinline__ void route_corrected(const RtParams& p, int t, int lane, float* sc) {
+    const float* row = p.logits + (size_t)t * p.ldl;
+    float mx = -INFINITY;
+    for (int e = lane; e < p.A; e += 32) mx = fmaxf(mx, row[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float sum = 0.f;
+    for (int e = lane; e < p.A; e += 32) sum += expf(row[e] - mx);
+    sum = warp_sum(sum);
+    for (int e = lane; e < p.A; e += 32) sc[e] = expf(row[e] - mx) / sum + p.correction[e];
+    __syncwarp();
+    for (int j = 0; j < p.top; ++j) {
+        float best = -INFINITY;
+        int be = 0x7fffffff;
+        for (int e = lane; e < p.A; e += 32)
+            if (sc[e] > best) best = sc[e], be = e;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+            if (ob > best || (ob == best && oe < be)) best = ob, be = oe;
+        }
+        // nothing comparable left (scores that are no numbers): a slot of weight zero, on the first expert
+        const bool none = be == 0x7fffffff;
+        if (lane == 0) {
+            const int e = none ? 0 : be;
+            p.sel[(size_t)t * p.top + j] = none ? p.A : e;
+            p.wts[(size_t)t * p.top + j] = none ? 0.f : expf(row[e] - mx) / sum;
+            p.tok_entries[(size_t)t * p.top + j] = -1;
+            if (!none) sc[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
+__global__ void __launch_bounds__(256) dense_route_kernel(const RtParams p) {
+    extern __shared__ float rt_sc[];
+    pdl_wait();
+    pdl_release();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t = blockIdx.x * 8 + warp;
+    if (t < p.n) route_corrected(p, t, lane, rt_sc + (size_t)warp * p.A);
+}
+
+// few entries: routing and lists in one CTA
+__global__ void __launch_bounds__(256) dense_route_plan_kernel(const RtParams p) {
+    extern __shared__ float rt_sc[];
+    int* cnt = reinterpret_cast<int*>(rt_sc + (size_t)8 * p.A);
+    pdl_wait();
+    pdl_release();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int t = warp; t < p.n; t += 8) route_corrected(p, t, lane, rt_sc + (size_t)warp * p.A);
+    __syncthreads();
+    const int ms = p.max_slots;
+    plan_entries<float>(cnt, p.n, p.E, p.top, p.chunk, 0, 1, p.sel, p.wts, p.active, p.n_active, p.slot_count, p.slot_offset,
+                        p.entry_row, p.entry_scale, p.tok_entries, p.active + ms, p.n_active + 1, p.slot_count + ms,
+                        p.slot_offset + ms);
+}
+
+}  // namespace glq
+
+using namespace glq;
+
+template <typename F> static int by_dtype(int dtype, F f) {
+    if (dtype == GLQ_DT_BF16) return f(bf16());
+    if (dtype == GLQ_DT_F32) return f(float());
+    return GLQ_ERR_ARG;
+}
+
+extern "C" int glq_dense_embed(int dtype, const int64_t* ids, const void* table, int rows, int C, int vocab, float* x, void* h,
+                               void* stream) {
+    if (!ids || !table || !x || !h || rows < 0 || C <= 0 || vocab <= 0) return GLQ_ERR_ARG;
+    if (rows == 0) return GLQ_OK;
+    return by_dtype(dtype, [&](auto z) {
+        using T = decltype(z);
+        return dn_launch(dense_embed_kernel<T>, dim3(rows), kRowThreads, 0, stream, ids, (const T*)table, C, vocab, x, (T*)h);
+    });
+}
+
+extern "C" int glq_dense_add_norm(int dtype, const float* y, const float* w, const float* final_w, float eps, int rows, int C,
+                                  float* x, void* h, void* stream) {
+    if (!y || !w || !x || !h || rows < 0 || C <= 0) return GLQ_ERR_ARG;
+    if (C > kMaxC) return GLQ_ERR_UNSUPPORTED;
+    if (rows == 0) return GLQ_OK;
+    return by_dtype(dtype, [&](auto z) {
+        using T = decltype(z);
+        return dn_launch(dense_add_norm_kernel<T>, dim3(rows), kRowThreads, (size_t)C * 4, stream, y, w, final_w, eps, C, x, (T*)h);
+    });
+}
+
+extern "C" int glq_dense_combine_norm(int dtype, const void* entry_out, int64_t lde, const int32_t* tok_entries, const float* wts,
+                                      int top, const float* w, const float* final_w, float eps, int rows, int C, float* x, void* h,
+                                      void* stream) {
+    if (!entry_out || !tok_entries || !wts || !w || !x || !h || top <= 0 || rows < 0 || C <= 0) return GLQ_ERR_ARG;
+    if (C > kMaxC) return GLQ_ERR_UNSUPPORTED;
+    if (rows == 0) return GLQ_OK;
+    return by_dtype(dtype, [&](auto z) {
+        using T = decltype(z);
+        return dn_launch(dense_combine_norm_kernel<T>, dim3(rows), kRowThreads, (size_t)C * 4, stream, (const T*)entry_out,
+                         (long long)lde, tok_entries, wts, top, w, final_w, eps, C, x, (T*)h);
+    });
+}
+
+extern "C" int glq_route_max_slots(int n, int E, int top, int chunk) {
+    const long nk = (long)n * top;
+    const long m = std::min<long>(E, nk) + (chunk > 0 ? nk / chunk : 0);
+    return (int)std::max<long>(1, std::min(m, nk));
+}
+
+extern "C" int glq_route(const glq_route_t* a, void* stream) {
+    if (!a || a->n < 0 || a->E <= 0 || a->identity < 0 || a->top <= 0 || a->top > a->E + a->identity) return GLQ_ERR_ARG;
+    if (!a->logits || !a->correction || !a->sel || !a->wts || !a->entry_scale || !a->tok_entries || !a->entry_row || !a->active ||
+        !a->slot_count || !a->slot_offset || !a->n_active)
+        return GLQ_ERR_ARG;
+    if (a->E + a->identity > 4096) return GLQ_ERR_UNSUPPORTED;
+    if (a->n == 0) return GLQ_OK;
+    if (a->max_slots < glq_route_max_slots(a->n, a->E, a->top, a->chunk)) return GLQ_ERR_WORKSPACE;
+    RtParams p{};
+    p.logits = a->logits;
+    p.correction = a->correction;
+    p.ldl = a->ldl;
+    p.n = a->n;
+    p.E = a->E;
+    p.A = a->E + a->identity;
+    p.top = a->top;
+    p.chunk = a->chunk;
+    p.sel = a->sel;
+    p.wts = a->wts;
+    p.entry_scale = a->entry_scale;
+    p.tok_entries = a->tok_entries;
+    p.entry_row = a->entry_row;
+    p.active = a->active;
+    p.slot_count = a->slot_count;
+    p.slot_offset = a->slot_offset;
+    p.n_active = a->n_active;
+    p.max_slots = a->max_slots;
+    const int nk = a->n * a->top;
+    const size_t sc = (size_t)8 * p.A * 4;
+    if (nk < 1024) return dn_launch(dense_route_plan_kernel, dim3(1), 256, sc + (size_t)2 * p.E * 4, stream, p);
+    if (!a->block_counts) return GLQ_ERR_ARG;
+    int st = dn_launch(dense_route_kernel, dim3(cdiv_i(a->n, 8)), 256, sc, stream, p);
+    if (st != GLQ_OK) return st;
+    // the list kernels are plain launches: they start when their predecessor is done
+    cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+    const int nb = cdiv_i(nk, kPlanChunk), ms = p.max_slots;
+    moe_plan_count_kernel<<<nb, 32, p.E * sizeof(int), s>>>(p.sel, nk, p.E, a->block_counts);
+    moe_plan_lists_kernel<<<1, 1024, 2 * p.E * sizeof(int), s>>>(a->block_counts, nb, nk, p.E, p.chunk, 0, 1, p.active, p.n_active,
+                                                                 p.slot_count, p.slot_offset, p.active + ms, p.n_active + 1,
+                                                                 p.slot_count + ms, p.slot_offset + ms);
+    moe_plan_scatter_kernel<float><<<nb, 32, p.E * sizeof(int), s>>>(p.sel, p.wts, nk, p.E, p.top, a->block_counts, p.entry_row,
+                                                                     p.entry_scale, p.tok_entries);
+    DN_CUDA(cudaGetLastError());
+    return GLQ_OK;
+}

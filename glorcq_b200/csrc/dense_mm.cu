@@ -1,0 +1,565 @@
+// Products with unquantized row-major weights, y = alpha * act(x . W^T), plain or over a device-side list of problems
+// (the experts of a mixture), in three forms:
+//   * few rows per problem (a decode step): a streaming kernel in the manner of the output projection (lm_head.cu):
+//     16 weight rows per warp tile, k split over the warps of a CTA, up to 8 activation rows as the columns of the
+//     tensor-core op; the first weight loads are issued before the kernel waits for its predecessor;
+//   * many rows: a persistent tcgen05 kernel; activation and weight tiles arrive by TMA (128-byte swizzle), the
+//     accumulator is double-buffered in tensor memory so that the epilogue of a tile overlaps the next tile's products;
+//   * float32, or rows that are no multiple of 16 bytes: a tiled kernel on the CUDA cores.
+// Rows sums are taken in a fixed order in all three: results do not depend on what else is in the batch.
+#include <cuda.h>
+
+#include <cstdlib>
+#include <mutex>
+
+#include "dense_common.cuh"
+
+namespace glq {
+thread_local int g_dense_cuda_error = 0;
+
+struct DmParams {
+    const void* x;
+    const void* W;
+    void* y;
+    float* y32;
+    const int* slot_index;
+    const int* n_slots;
+    const int* slot_count;
+    const int* slot_offset;
+    const int* entry_row;
+    long long ldx, ldy, ldy32;
+    int N, K, rows, slots, split, act;
+    float alpha;
+    int vec_y, vec_y32;
+};
+
+struct DmSlot {
+    int mat, off, cnt;
+};
+__device__ __forceinline__ DmSlot dm_slot(const DmParams& p, int s) {
+    if (!p.slot_index) return {0, 0, p.rows};
+    if (s >= __ldg(p.n_slots)) return {0, 0, 0};
+    return {__ldg(p.slot_index + s), __ldg(p.slot_offset + s), __ldg(p.slot_count + s)};
+}
+
+template <typename T> __device__ __forceinline__ void dm_store(const DmParams& p, int row, int n, float v) {
+    if (n < p.split) reinterpret_cast<T*>(p.y)[(size_t)row * p.ldy + n] = from_f<T>(v);
+    else p.y32[(size_t)row * p.ldy32 + (n - p.split)] = v;
+}
+
+// =====================================================================================================
+// streaming kernel: up to 8 rows per slot
+// =====================================================================================================
+__device__ __forceinline__ uint4 dm_ldg(const uint4* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+                 : "l"(p));
+    return v;
+}
+constexpr int kDmDepth = 8;
+
+template <int SPLIT>   // warps that share one 16-row tile
+__global__ void __launch_bounds__(kThreads, 2) dense_stream_kernel(const DmParams p) {
+    constexpr int TILES = kWarpsPerCta / SPLIT;
+    extern __shared__ __align__(16) unsigned char dm_smem[];
+    const int K = p.K, KP = (K + 31) / 32 * 32, XS = KP + 32;      // padded activation rows: distinct banks
+    bf16* xs = reinterpret_cast<bf16*>(dm_smem);
+    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * XS * 2);
+    const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    const int g = lane >> 2, t = lane & 3;
+    const int tw = w / SPLIT, s = w % SPLIT;
+    const int chunks = KP / 32;
+    const int c_lo = (int)((long)s * chunks / SPLIT), c_hi = (int)((long)(s + 1) * chunks / SPLIT);
+    const int ntiles = (p.N + 15) / 16;
+    const bool plain = p.slot_index == nullptr;
+    DmSlot sl{0, 0, p.rows};
+    if (!plain) {
+        pdl_wait();
+        pdl_release();
+        sl = dm_slot(p, blockIdx.y);
+        if (sl.cnt == 0) return;
+    }
+    const bf16* Wm = reinterpret_cast<const bf16*>(p.W) + (size_t)sl.mat * p.N * K;
+    const int iters = (ntiles + TILES * (int)gridDim.x - 1) / (TILES * (int)gridDim.x);
+    for (int it = 0; it < iters; ++it) {
+        const int tile = (it * (int)gridDim.x + (int)blockIdx.x) * TILES + tw;
+        const bool live = tile < ntiles;
+        const int r0 = min(tile * 16 + g, p.N - 1), r1 = min(tile * 16 + g + 8, p.N - 1);
+        const bf16* w0 = Wm + (size_t)r0 * K + t * 8;
+        const bf16* w1 = Wm + (size_t)r1 * K + t * 8;
+        const int lim = K - 8 - t * 8;      // this lane's 8 channels of chunk c exist when 32 c <= lim
+        uint4 qa[kDmDepth], qb[kDmDepth];
+        auto fetch = [&](int c, int d) {
+            const bool ok = live && c < c_hi && 32 * c <= lim;
+            qa[d] = ok ? dm_ldg(reinterpret_cast<const uint4*>(w0 + 32 * c)) : make_uint4(0, 0, 0, 0);
+            qb[d] = ok ? dm_ldg(reinterpret_cast<const uint4*>(w1 + 32 * c)) : make_uint4(0, 0, 0, 0);
+        };
+#pragma unroll
+        for (int d = 0; d < kDmDepth; ++d) fetch(c_lo + d, d);
+        for (int rb = 0; rb < sl.cnt; rb += 8) {
+            const int nr = min(8, sl.cnt - rb);
+            if (it == 0 || sl.cnt > 8) {
+                if (plain && it == 0 && rb == 0) {
+                    pdl_wait();
+                    pdl_release();
+                }
+                __syncthreads();
+                for (int i = tid; i < 8 * (KP / 8); i += kThreads) {
+                    const int row = i / (KP / 8), c = i % (KP / 8);
+                    uint4 v = make_uint4(0, 0, 0, 0);
+                    if (row < nr && c * 8 < K) {
+                        const int e = sl.off + rb + row;
+                        const long long xr = p.entry_row ? p.entry_row[e] : e;
+                        v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.x) + xr * p.ldx + c * 8);
+                    }
+                    *reinterpret_cast<uint4*>(xs + (size_t)row * XS + c * 8) = v;
+                }
+                __syncthreads();
+            }
+            if (rb > 0) {
+#pragma unroll
+                for (int d = 0; d < kDmDepth; ++d) fetch(c_lo + d, d);
+            }
+            float acc[4] = {0.f, 0.f, 0.f, 0.f};
+            const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)g * XS) + t;
+            for (int c0 = c_lo; c0 < c_hi; c0 += kDmDepth) {
+#pragma unroll
+                for (int d = 0; d < kDmDepth; ++d) {
+                    const int c = c0 + d;
+                    if (c < c_hi) {
+                        const uint4 a = qa[d], b = qb[d];
+                        fetch(c + kDmDepth, d);
+                        const uint4 xv = xb[c * 4];
+                        mma_bf16(acc, a.x, b.x, a.y, b.y, xv.x, xv.y);
+                        mma_bf16(acc, a.z, b.z, a.w, b.w, xv.z, xv.w);
+                    }
+                }
+            }
+            if (s != 0) red[w * 32 + lane] = make_float4(acc[0], acc[1], acc[2], acc[3]);
+            __syncthreads();
+            if (s == 0 && live) {
+                for (int s2 = 1; s2 < SPLIT; ++s2) {
+                    const float4 v = red[(w + s2) * 32 + lane];
+                    acc[0] += v.x;
+                    acc[1] += v.y;
+                    acc[2] += v.z;
+                    acc[3] += v.w;
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
+                    if (row < nr && n < p.N) dm_store<bf16>(p, sl.off + rb + row, n, p.alpha * act_dyn(p.act, acc[i]));
+                }
+            }
+            __syncthreads();
+        }
+    }
+}
+
+// =====================================================================================================
+// generic kernel: any type, any size
+// =====================================================================================================
+template <typename T>
+__global__ void __launch_bounds__(256) dense_generic_kernel(const DmParams p) {
+    __shared__ float xs[16][65], ws[16][65];
+    pdl_wait();
+    pdl_release();
+    const DmSlot sl = dm_slot(p, blockIdx.z);
+    const int n0 = blockIdx.x * 64;
+    const T* Wm = reinterpret_cast<const T*>(p.W) + (size_t)sl.mat * p.N * p.K;
+    const T* X = reinterpret_cast<const T*>(p.x);
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    for (int m0 = blockIdx.y * 64; m0 < sl.cnt; m0 += gridDim.y * 64) {
+        float acc[4][4] = {};
+        for (int k0 = 0; k0 < p.K; k0 += 16) {
+            __syncthreads();
+            for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+                const int r = i >> 4, kk = i & 15;
+                const bool kin = k0 + kk < p.K;
+                float xv = 0.f, wv = 0.f;
+                if (kin && m0 + r < sl.cnt) {
+                    const int e = sl.off + m0 + r;
+                    const long long xr = p.entry_row ? p.entry_row[e] : e;
+                    xv = to_f(X[xr * p.ldx + k0 + kk]);
+                }
+                if (kin && n0 + r < p.N) wv = to_f(Wm[(size_t)(n0 + r) * p.K + k0 + kk]);
+                xs[kk][r] = xv;
+                ws[kk][r] = wv;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int kk = 0; kk < 16; ++kk)
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[i][j] += xs[kk][ty + 16 * i] * ws[kk][tx + 16 * j];
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int m = m0 + ty + 16 * i, n = n0 + tx + 16 * j;
+                if (m < sl.cnt && n < p.N) dm_store<T>(p, sl.off + m, n, p.alpha * act_dyn(p.act, acc[i][j]));
+            }
+    }
+}
+
+// entry rows of x -> consecutive rows (the token operand of the grouped tensor-core kernel)
+__global__ void __launch_bounds__(256) dense_gather_kernel(const DmParams p, bf16* __restrict__ out) {
+    pdl_wait();
+    pdl_release();
+    const int last = __ldg(p.n_slots) - 1;
+    const int total = last < 0 ? 0 : __ldg(p.slot_offset + last) + __ldg(p.slot_count + last);
+    const int vec = p.K / 8;
+    for (int e = blockIdx.x; e < total; e += gridDim.x) {
+        const uint4* src = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.x) + (long long)p.entry_row[e] * p.ldx);
+        uint4* dst = reinterpret_cast<uint4*>(out + (size_t)e * p.K);
+        for (int i = threadIdx.x; i < vec; i += 256) dst[i] = src[i];
+    }
+}
+
+// =====================================================================================================
+// tcgen05 kernel: 128 rows x TN features per tile
+// =====================================================================================================
+constexpr int kDtThreads = 192;        // warp 0: TMA, warp 1: MMA, warps 2..5: epilogue
+constexpr int kDtMaxSlots = 1024;
+
+template <int TN> struct DtCfg {
+    static constexpr int A_BYTES = 128 * 128, B_BYTES = TN * 128, STAGE = A_BYTES + B_BYTES;
+    static constexpr int S = (208 * 1024) / STAGE > 6 ? 6 : (208 * 1024) / STAGE;
+    static constexpr size_t SMEM = (size_t)S * STAGE + 1024;
+};
+
+// both operands bf16, K-major, fp32 accumulator, M = 128
+__host__ __device__ constexpr uint32_t dt_idesc(int n) { return tc_idesc(n) | (1u << 7) | (1u << 10); }
+
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
+        "l"(map), "r"(x), "r"(y), "r"(bar)
+        : "memory");
+}
+
+template <int TN>
+__global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_constant__ CUtensorMap ma,
+                                                                const __grid_constant__ CUtensorMap mb, const DmParams p) {
+    using C = DtCfg<TN>;
+    constexpr int S = C::S;
+    extern __shared__ unsigned char dt_smem_raw[];
+    __shared__ __align__(8) unsigned long long bars[2 * S + 4];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_dead;
+    __shared__ int s_pre[kDtMaxSlots + 1];      // row tiles before each slot
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t sbase = (smem_u32(dt_smem_raw) + 1023u) & ~1023u;
+    const uint32_t full = smem_u32(bars), empty = full + 8 * S, afull = full + 16 * S, aempty = afull + 16;
+    volatile int* dead = &s_dead;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < S; ++s) {
+            mbar_init(full + 8 * s, 1);
+            mbar_init(empty + 8 * s, 1);
+        }
+        for (int b = 0; b < 2; ++b) {
+            mbar_init(afull + 8 * b, 1);
+            mbar_init(aempty + 8 * b, 4);
+        }
+        s_dead = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) tc_alloc(smem_u32(&s_tmem), 2 * TN);
+    pdl_wait();
+    pdl_release();
+    const int nslots = p.slot_index ? min(__ldg(p.n_slots), p.slots) : 1;
+    if (warp == 0) {
+        int base = 0;
+        for (int s0 = 0; s0 < nslots; s0 += 32) {
+            const int s = s0 + lane;
+            int v = 0;
+            if (s < nslots) v = ((p.slot_index ? __ldg(p.slot_count + s) : p.rows) + 127) / 128;
+            int inc = v;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int u = __shfl_up_sync(0xffffffffu, inc, o);
+                if (lane >= o) inc += u;
+            }
+            if (s < nslots) s_pre[s + 1] = base + inc;
+            base += __shfl_sync(0xffffffffu, inc, 31);
+        }
+        if (lane == 0) s_pre[0] = 0;
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s_tmem;
+    const int nft = (p.N + TN - 1) / TN;
+    const int total = s_pre[nslots] * nft;
+    const int nk = (p.K + 63) / 64;
+    // tile -> (slot, row tile, feature tile): row tiles of a slot run fastest, so that they share a weight tile
+    auto locate = [&](int tile, int& slot, int& mt, int& ft) {
+        int lo = 0, hi = nslots;
+        while (hi - lo > 1) {
+            const int mid = (lo + hi) >> 1;
+            if (s_pre[mid] * nft <= tile) lo = mid;
+            else hi = mid;
+        }
+        slot = lo;
+        const int m = s_pre[lo + 1] - s_pre[lo], l = tile - s_pre[lo] * nft;
+        ft = l / m;
+        mt = l - ft * m;
+    };
+
+    if (warp == 0) {
+        if (lane == 0) {
+            int s = 0, issued = 0;
+            uint32_t ph = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
+                int slot, mt, ft;
+                locate(tile, slot, mt, ft);
+                const DmSlot sl = dm_slot(p, slot);
+                const int row = sl.off + mt * 128, wrow = sl.mat * p.N + ft * TN;
+                for (int k = 0; k < nk; ++k) {
+                    ok = tc_wait(empty + 8 * s, ph ^ 1u, dead, 110);
+                    if (!ok) break;
+                    const uint32_t a = sbase + (uint32_t)s * C::STAGE;
+                    mbar_expect_tx(full + 8 * s, C::STAGE);
+                    tma_load_2d(a, &ma, k * 64, row, full + 8 * s);
+                    tma_load_2d(a + C::A_BYTES, &mb, k * 64, wrow, full + 8 * s);
+                    ++issued;
+                    if (++s == S) {
+                        s = 0;
+                        ph ^= 1u;
+                    }
+                }
+            }
+            if (*dead) {   // copies in flight must land before the CTA leaves (bounded)
+                for (int i = 0; i < S && i < issued; ++i) {
+                    if (--s < 0) {
+                        s = S - 1;
+                        ph ^= 1u;
+                    }
+                    const unsigned long long t0 = global_ns();
+                    while (!mbar_test_wait(full + 8 * s, ph) && global_ns() - t0 < 2000000ull) __nanosleep(64);
+                }
+            }
+        }
+        __syncwarp();
+    } else if (warp == 1) {
+        if (lane == 0) {
+            int s = 0, buf = 0;
+            uint32_t ph = 0, aph = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
+                ok = tc_wait(aempty + 8 * buf, aph ^ 1u, dead, 111);
+                if (!ok) break;
+                tc_fence_after();
+                for (int k = 0; k < nk; ++k) {
+                    ok = tc_wait(full + 8 * s, ph, dead, 112);
+                    if (!ok) break;
+                    tc_fence_after();
+                    const uint32_t a = sbase + (uint32_t)s * C::STAGE;
+#pragma unroll
+                    for (int kk = 0; kk < 4; ++kk)
+                        tc_mma_f16(tmem + (uint32_t)(buf * TN), tc_smem_desc(a + 32u * kk), tc_smem_desc(a + C::A_BYTES + 32u * kk),
+                                   dt_idesc(TN), (k | kk) != 0);
+                    tc_commit(empty + 8 * s);
+                    if (++s == S) {
+                        s = 0;
+                        ph ^= 1u;
+                    }
+                }
+                if (ok) tc_commit(afull + 8 * buf);
+                buf ^= 1;
+                if (buf == 0) aph ^= 1u;
+            }
+        }
+        __syncwarp();
+    } else {
+        const int q = warp & 3;      // tensor memory lanes 32 q .. 32 q + 31
+        int buf = 0;
+        uint32_t aph = 0;
+        for (int tile = blockIdx.x; tile < total; tile += gridDim.x) {
+            int slot, mt, ft;
+            locate(tile, slot, mt, ft);
+            const DmSlot sl = dm_slot(p, slot);
+            if (!tc_wait(afull + 8 * buf, aph, dead, 113)) break;
+            __syncwarp();
+            tc_fence_after();
+            const int r = mt * 128 + q * 32 + lane;
+            const bool rin = r < sl.cnt;
+            const size_t orow = (size_t)(sl.off + r);
+#pragma unroll 1
+            for (int c0 = 0; c0 < TN; c0 += 16) {
+                const int n0 = ft * TN + c0;
+                if (n0 >= p.N) break;
+                uint32_t v[16];
+                __syncwarp();
+                tc_ld16(tmem + (uint32_t)(buf * TN + c0) + ((uint32_t)(q * 32) << 16), v);
+                tc_ld_wait();
+                if (!rin) continue;
+                float f[16];
+#pragma unroll
+                for (int j = 0; j < 16; ++j) f[j] = p.alpha * act_dyn(p.act, __uint_as_float(v[j]));
+                if (n0 + 16 <= p.split && p.vec_y) {
+                    uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.y) + orow * p.ldy + n0);
+                    dst[0] = make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
+                    dst[1] = make_uint4(pack_bf2(f[8], f[9]), pack_bf2(f[10], f[11]), pack_bf2(f[12], f[13]), pack_bf2(f[14], f[15]));
+                } else if (n0 >= p.split && n0 + 16 <= p.N && p.vec_y32) {
+                    float4* dst = reinterpret_cast<float4*>(p.y32 + orow * p.ldy32 + (n0 - p.split));
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) dst[j] = make_float4(f[4 * j], f[4 * j + 1], f[4 * j + 2], f[4 * j + 3]);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        if (n0 + j < p.N) dm_store<bf16>(p, (int)orow, n0 + j, f[j]);
+                }
+            }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(aempty + 8 * buf);
+            buf ^= 1;
+            if (buf == 0) aph ^= 1u;
+        }
+    }
+    __syncthreads();
+    if (warp == 1) {
+        tc_fence_after();
+        tc_dealloc(tmem, 2 * TN);
+    }
+}
+
+// ---- host ---------------------------------------------------------------------------------------------
+typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+static EncodeTiled encode_tiled() {
+    static EncodeTiled fn = [] {
+        void* p = nullptr;
+        cudaDriverEntryPointQueryResult st;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &st) != cudaSuccess ||
+            st != cudaDriverEntryPointSuccess)
+            p = nullptr;
+        return reinterpret_cast<EncodeTiled>(p);
+    }();
+    return fn;
+}
+// (rows, K) bf16 with row stride ld elements; boxes of 64 columns x box_rows, 128-byte swizzle, zeros outside
+static bool make_map(CUtensorMap* m, const void* base, long rows, long K, long ld, int box_rows) {
+    const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {64, (cuuint32_t)box_rows}, es[2] = {1, 1};
+    return encode_tiled()(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, es,
+                          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <int TN>
+static int launch_dt(const DmParams& p, const void* xa, long xrows, long ldx, long nmat, long tiles, void* stream) {
+    CUtensorMap ma, mb;
+    if (!make_map(&ma, xa, xrows, p.K, ldx, 128) || !make_map(&mb, p.W, nmat * p.N, p.K, p.K, TN)) return GLQ_ERR_UNSUPPORTED;
+    const int grid = (int)std::max<long>(1, std::min<long>(tiles, dn_sms()));
+    return dn_launch(dense_tc_kernel<TN>, dim3(grid), kDtThreads, DtCfg<TN>::SMEM, stream, ma, mb, p);
+}
+
+}  // namespace glq
+
+using namespace glq;
+
+extern "C" const char* glq_dense_status_string(int status) {
+    switch (status) {
+        case GLQ_OK: return "ok";
+        case GLQ_ERR_ARG: return "invalid argument";
+        case GLQ_ERR_ALIGN: return "misaligned pointer or leading dimension";
+        case GLQ_ERR_UNSUPPORTED: return "unsupported shape";
+        case GLQ_ERR_CUDA: return "CUDA error";
+        case GLQ_ERR_WORKSPACE: return "workspace too small";
+    }
+    return "unknown status";
+}
+extern "C" int glq_dense_last_cuda_error(void) { return g_dense_cuda_error; }
+extern "C" int glq_dense_debug_error(unsigned long long* out4, int clear) {
+    DN_CUDA(cudaMemcpyFromSymbol(out4, g_glq_err, 4 * sizeof(unsigned long long)));
+    if (clear) {
+        const unsigned long long z[4] = {0, 0, 0, 0};
+        DN_CUDA(cudaMemcpyToSymbol(g_glq_err, z, sizeof(z)));
+    }
+    return GLQ_OK;
+}
+
+// rows per problem up to which the streaming kernel runs (weights are read once per 8 rows)
+static constexpr int kStreamRows = 8;
+
+extern "C" int glq_dense_matmul_path(const glq_dense_mm_t* a) {
+    if (a->dtype != GLQ_DT_BF16 || a->K % 8 || a->ldx % 8 || !al16(a->x) || !al16(a->W)) return 0;
+    const int rows = a->slot_index ? a->max_slot_rows : a->rows;
+    if (rows <= kStreamRows && a->K <= 12288) return 1;
+    if ((a->slot_index && a->max_slots > kDtMaxSlots) || (a->entry_row && !a->gather) || !encode_tiled()) return 0;
+    return 2;
+}
+
+extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
+    if (!a || a->N <= 0 || a->K <= 0 || a->rows < 0 || a->split < 0 || a->split > a->N) return GLQ_ERR_ARG;
+    if (a->dtype != GLQ_DT_BF16 && a->dtype != GLQ_DT_F32) return GLQ_ERR_ARG;
+    if (a->rows == 0) return GLQ_OK;
+    const bool grouped = a->slot_index != nullptr;
+    if (!a->x || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
+    if (grouped && (!a->n_slots || !a->slot_count || !a->slot_offset || a->max_slots <= 0 || a->max_slot_rows <= 0 || a->n_matrices <= 0))
+        return GLQ_ERR_ARG;
+    if (!grouped && a->entry_row) return GLQ_ERR_ARG;
+    DmParams p{};
+    p.x = a->x;
+    p.W = a->W;
+    p.y = a->y;
+    p.y32 = a->y32;
+    p.slot_index = a->slot_index;
+    p.n_slots = a->n_slots;
+    p.slot_count = a->slot_count;
+    p.slot_offset = a->slot_offset;
+    p.entry_row = a->entry_row;
+    p.ldx = a->ldx;
+    p.ldy = a->ldy;
+    p.ldy32 = a->ldy32;
+    p.N = a->N;
+    p.K = a->K;
+    p.rows = a->rows;
+    p.slots = grouped ? a->max_slots : 1;
+    p.split = a->split;
+    p.act = a->act;
+    p.alpha = a->alpha;
+    p.vec_y = a->y && al16(a->y) && a->ldy % 8 == 0;
+    p.vec_y32 = a->y32 && al16(a->y32) && a->ldy32 % 4 == 0 && a->split % 4 == 0;
+    const int path = glq_dense_matmul_path(a);
+    const int rows_max = grouped ? a->max_slot_rows : a->rows;
+    if (path == 1) {
+        const size_t smem = (size_t)8 * ((a->K + 31) / 32 * 32 + 32) * 2 + (size_t)kWarpsPerCta * 32 * sizeof(float4);
+        const int tiles = cdiv_i(a->N, 16), want = 2 * dn_sms();
+        // few tiles: all eight warps of a CTA share one
+        if ((long)tiles * p.slots <= want * 2)
+            return dn_launch(dense_stream_kernel<8>, dim3(std::min(tiles, want), p.slots), kThreads, smem, stream, p);
+        return dn_launch(dense_stream_kernel<4>, dim3(std::min(cdiv_i(tiles, 2), want), p.slots), kThreads, smem, stream, p);
+    }
+    if (path == 2) {
+        const void* xa = a->x;
+        long ldx = a->ldx;
+        if (a->entry_row) {
+            if (!al16(a->gather)) return GLQ_ERR_ALIGN;
+            const int st = dn_launch(dense_gather_kernel, dim3(std::min(a->rows, 8 * dn_sms())), 256, 0, stream, p,
+                                     reinterpret_cast<bf16*>(a->gather));
+            if (st != GLQ_OK) return st;
+            xa = a->gather;
+            ldx = a->K;
+            p.entry_row = nullptr;
+        }
+        const long mt = grouped ? a->rows / 128 + p.slots : cdiv_i(a->rows, 128);
+        const long sms = dn_sms();
+        const long nmat = grouped ? a->n_matrices : 1;
+        // widest feature tile that still gives every SM work
+        if (a->N > 128 && mt * cdiv_i(a->N, 256) >= sms) return launch_dt<256>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 256), stream);
+        if (a->N > 64 && mt * cdiv_i(a->N, 128) >= sms) return launch_dt<128>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 128), stream);
+        return launch_dt<64>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 64), stream);
+    }
+    const dim3 grid(cdiv_i(a->N, 64), std::min(cdiv_i(rows_max, 64), 1024), p.slots);
+    if (grid.z > 65535) return GLQ_ERR_UNSUPPORTED;
+    if (a->dtype == GLQ_DT_F32) return dn_launch(dense_generic_kernel<float>, grid, 256, 0, stream, p);
+    return dn_launch(dense_generic_kernel<bf16>, grid, 256, 0, stream, p);
+}

@@ -1,0 +1,644 @@
+// Matrix-memory recurrence with exponential gates and a running log maximum (mLSTM; Beck et al., "xLSTM: Extended Long
+// Short-Term Memory").  Per head, S (D, V), n (D) and m are float and carried from call to call:
+//     m' = max(f + m, i);  S' = e^(f+m-m') S + e^(i-m') k v^T;  n' = e^(f+m-m') n + e^(i-m') k
+//     o = S'^T q / (max(|n'.q|, e^-m') + 1e-6)
+// Two forms of the same recurrence:
+//   * step: the recurrence itself, one position after the other.  A CTA owns 32 value columns of a head; the CTA of a
+//     head that arrives last applies the per-head norm and the output gate, so a decode step is one launch.
+//   * chunk: 64 positions at a time on the tensor cores.  With b the running sum of f inside a chunk, a_s = i_s - b_s
+//     and r_t = b_t - m_t, position s reaches position t of its chunk with weight e^(r_t + a_s) and the state at the
+//     chunk's start with e^(r_t + m_start); m_t = b_t + max(m_start, max_{s<=t} a_s) is the recurrence's own maximum.
+//     Every float operand of a tensor-core product (scaled keys, state, weights) goes in as a sum of two bf16 numbers.
+// State layout: S (B, H, slices, D, 32), n (B, H, slices, D) and m (B, H, slices), the last two once per 32-column
+// slice, so that no CTA reads what another one is about to write.
+#include "dense_common.cuh"
+
+namespace glq {
+
+constexpr int kSl = 32;            // value columns of a slice
+constexpr int kL = 64;             // positions of a chunk
+
+struct MlParams {
+    const void* qkvg;
+    const float* gates;
+    const float* bias_i;
+    const float* bias_f;
+    const float* norm_w;
+    float* S;
+    float* n;
+    float* m;
+    void* out;
+    float* o;                      // (B * Tall, H * V)
+    int* counters;
+    long long ldp, ldg;
+    int B, T, H, D, V, slices;
+    int state_idle;
+    int t0, Tall;                  // this call's positions: t0 .. t0 + T - 1 of the Tall rows of a sequence
+    float cap, eps, scale;
+    // chunk form
+    float *r, *a, *mt, *min_, *nbuf;
+    bf16 *Shi, *Slo;
+    int nc, Dp, Vp;
+};
+
+__device__ __forceinline__ float log_i(const MlParams& p, size_t row, int h) {
+    return p.cap * tanhf((p.gates[row * p.ldg + h] + p.bias_i[h]) / p.cap);
+}
+__device__ __forceinline__ float log_f(const MlParams& p, size_t row, int h) {
+    const float z = p.cap * tanhf((p.gates[row * p.ldg + p.H + h] + p.bias_f[h]) / p.cap);
+    return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+}
+
+// rows row0 .. of head h: out = rms_norm(o) * w * sigmoid(g); one warp per row
+template <typename T>
+__device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, int h, int lane) {
+    const float* o = p.o + row * p.H * p.V + (size_t)h * p.V;
+    const T* g = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)p.H * (2 * p.D + p.V) + (size_t)h * p.V;
+    T* out = reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V;
+    float ss = 0.f;
+    for (int v = lane; v < p.V; v += 32) {
+        const float x = __ldcg(o + v);
+        ss += x * x;
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / p.V + p.eps);
+    for (int v = lane; v < p.V; v += 32) out[v] = from_f<T>(__ldcg(o + v) * inv * p.norm_w[h * p.V + v] * sigmoid_f(to_f(g[v])));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) mlstm_step_kernel(const MlParams p) {
+    extern __shared__ float ml_smem[];
+    float* sq = ml_smem;                 // [D]
+    float* sk = sq + p.D;                // [D]
+    __shared__ float sv[kSl], part[8][kSl], dpart[8];
+    __shared__ int s_last;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int sl = blockIdx.x, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
+    const int D = p.D, V = p.V, v0 = sl * kSl, vw = min(kSl, V - v0);
+    const size_t bh = (size_t)b * p.H + h;
+    float* S = p.S + (bh * p.slices + sl) * (size_t)D * kSl;
+    float* n = p.n + (bh * p.slices + sl) * (size_t)D;
+    float* mp = p.m + bh * p.slices + sl;
+    const int rr = warp * 4 + (lane >> 3), cc = (lane & 7) * 4;
+    constexpr int U = 8;
+    float4 pre[U];
+    // a state that the preceding launch does not touch is requested before the wait for the projections
+    if (!p.state_idle) pdl_wait();
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int d = rr + 32 * u;
+        pre[u] = d < D ? *reinterpret_cast<const float4*>(S + (size_t)d * kSl + cc) : make_float4(0, 0, 0, 0);
+    }
+    float m = *mp;
+    pdl_wait();
+    pdl_release();
+    for (int t = 0; t < p.T; ++t) {
+        const size_t row = (size_t)b * p.Tall + p.t0 + t;
+        const T* q = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)h * D;
+        const T* k = q + (size_t)p.H * D;
+        const T* v = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)2 * p.H * D + (size_t)h * V + v0;
+        __syncthreads();
+        for (int d = tid; d < D; d += 256) {
+            sq[d] = to_f(q[d]) * p.scale;
+            sk[d] = to_f(k[d]);
+        }
+        if (tid < kSl) sv[tid] = tid < vw ? to_f(v[tid]) : 0.f;
+        const float li = log_i(p, row, h), lf = log_f(p, row, h);
+        const float mn = fmaxf(lf + m, li);
+        const float keep = expf(lf + m - mn), add = expf(li - mn);
+        m = mn;
+        __syncthreads();
+        const float4 vv = make_float4(sv[cc], sv[cc + 1], sv[cc + 2], sv[cc + 3]);
+        float4 acc = make_float4(0, 0, 0, 0);
+        for (int d0 = 0; d0 < D; d0 += 32 * U) {
+            if (t > 0 || d0 > 0) {
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    const int d = d0 + rr + 32 * u;
+                    pre[u] = d < D ? *reinterpret_cast<const float4*>(S + (size_t)d * kSl + cc) : make_float4(0, 0, 0, 0);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int d = d0 + rr + 32 * u;
+                if (d < D) {
+                    const float kd = add * sk[d], qd = sq[d];
+                    float4 s = pre[u];
+                    s.x = keep * s.x + kd * vv.x;
+                    s.y = keep * s.y + kd * vv.y;
+                    s.z = keep * s.z + kd * vv.z;
+                    s.w = keep * s.w + kd * vv.w;
+                    *reinterpret_cast<float4*>(S + (size_t)d * kSl + cc) = s;
+                    acc.x += s.x * qd;
+                    acc.y += s.y * qd;
+                    acc.z += s.z * qd;
+                    acc.w += s.w * qd;
+                }
+            }
+        }
+        float den = 0.f;
+        for (int d = tid; d < D; d += 256) {
+            const float nn = keep * n[d] + add * sk[d];
+            n[d] = nn;
+            den += nn * sq[d];
+        }
+#pragma unroll
+        for (int o = 8; o < 32; o <<= 1) {
+            acc.x += __shfl_xor_sync(0xffffffffu, acc.x, o);
+            acc.y += __shfl_xor_sync(0xffffffffu, acc.y, o);
+            acc.z += __shfl_xor_sync(0xffffffffu, acc.z, o);
+            acc.w += __shfl_xor_sync(0xffffffffu, acc.w, o);
+        }
+        den = warp_sum(den);
+        if (lane < 8) *reinterpret_cast<float4*>(&part[warp][cc]) = acc;
+        if (lane == 0) dpart[warp] = den;
+        __syncthreads();
+        if (tid < vw) {
+            float num = 0.f, dd = 0.f;
+#pragma unroll
+            for (int w = 0; w < 8; ++w) {
+                num += part[w][tid];
+                dd += dpart[w];
+            }
+            __stcg(p.o + row * p.H * V + (size_t)h * V + v0 + tid, num / (fmaxf(fabsf(dd), expf(-m)) + 1e-6f));
+        }
+    }
+    if (tid == 0) *mp = m;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        const int old = atomicAdd(p.counters + bh, 1);
+        s_last = old == p.slices - 1;
+        if (s_last) p.counters[bh] = 0;
+    }
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    for (int t = warp; t < p.T; t += 8) head_norm_gate<T>(p, (size_t)b * p.Tall + p.t0 + t, h, lane);
+}
+
+// ---- chunk form ------------------------------------------------------------------------------------------
+// gates of a head for all chunks: r, a, m of every position (positions past T weigh nothing), m at every chunk's start
+__global__ void __launch_bounds__(256) mlstm_gate_kernel(const MlParams p) {
+    extern __shared__ float ml_smem[];
+    float* ctot = ml_smem;               // [nc] sum of f
+    float* cmax = ctot + p.nc;           // [nc] max of a
+    float* cm = cmax + p.nc;             // [nc] m at the chunk's start
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int h = blockIdx.x % p.H, b = blockIdx.x / p.H;
+    const size_t bh = blockIdx.x, base = bh * (size_t)p.nc * kL;
+    pdl_wait();
+    pdl_release();
+    for (int c = warp; c < p.nc; c += 8) {
+        float f[2], li[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int t = c * kL + 2 * lane + e;
+            const size_t row = (size_t)b * p.Tall + p.t0 + t;
+            f[e] = t < p.T ? log_f(p, row, h) : 0.f;
+            li[e] = t < p.T ? log_i(p, row, h) : -INFINITY;
+        }
+        float sum = f[0] + f[1];
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += u;
+        }
+        const float b1 = sum, b0 = sum - f[1];
+        const float a0 = li[0] - b0, a1 = li[1] - b1;
+        float mx = fmaxf(a0, a1);
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, mx, o);
+            if (lane >= o) mx = fmaxf(mx, u);
+        }
+        const float prev = __shfl_up_sync(0xffffffffu, mx, 1);
+        const size_t i = base + c * kL + 2 * lane;
+        p.a[i] = a0;
+        p.a[i + 1] = a1;
+        p.r[i] = b0;                     // b and the running maximum for now
+        p.r[i + 1] = b1;
+        p.mt[i] = lane ? fmaxf(prev, a0) : a0;
+        p.mt[i + 1] = mx;
+        if (lane == 31) {
+            ctot[c] = b1;
+            cmax[c] = mx;
+        }
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        float m = p.m[bh * p.slices];
+        for (int c = 0; c < p.nc; ++c) {
+            cm[c] = m;
+            p.min_[bh * p.nc + c] = m;
+            m = ctot[c] + fmaxf(m, cmax[c]);
+        }
+        for (int s = 0; s < p.slices; ++s) p.m[bh * p.slices + s] = m;
+    }
+    __syncthreads();
+    for (int c = warp; c < p.nc; c += 8) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const size_t i = base + c * kL + 2 * lane + e;
+            const float bb = p.r[i], mm = bb + fmaxf(cm[c], p.mt[i]);
+            p.mt[i] = mm;
+            p.r[i] = bb - mm;
+        }
+    }
+}
+
+constexpr int kTd = 64, kLd = 72;        // tile width, row stride of a 64-wide shared-memory tile (bf16)
+
+// state at every chunk's start (as two bf16 planes, and n) and after the last chunk; one CTA owns 64 x 64 of a head's S
+__global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
+    __shared__ __align__(16) bf16 ks[2][kL * kLd], vs[2][kL * kLd];
+    __shared__ float ws[kL];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.z % p.H, b = blockIdx.z / p.H;
+    const int d0 = blockIdx.x * kTd, v0 = blockIdx.y * kTd;
+    const size_t bh = blockIdx.z;
+    const bf16* kb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)p.H * p.D + (size_t)h * p.D;
+    const bf16* vb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)2 * p.H * p.D + (size_t)h * p.V;
+    auto load = [&](int c, int buf) {
+        for (int i = tid; i < kL * 8; i += 128) {
+            const int s = i >> 3, cc = (i & 7) * 8, tt = c * kL + s;
+            const size_t row = ((size_t)b * p.Tall + p.t0 + (tt < p.T ? tt : 0)) * p.ldp;
+            const bool kl = tt < p.T && d0 + cc < p.D, vl = tt < p.T && v0 + cc < p.V;
+            cpa16(smem_u32(&ks[buf][s * kLd + cc]), kl ? kb + row + d0 + cc : kb, kl);
+            cpa16(smem_u32(&vs[buf][s * kLd + cc]), vl ? vb + row + v0 + cc : vb, vl);
+        }
+        cpa_commit();
+    };
+    const int dr[2] = {d0 + 16 * warp + g, d0 + 16 * warp + g + 8};
+    float acc[8][4], nacc[2];
+    pdl_wait();
+    pdl_release();
+    load(0, 0);
+    const size_t slb = bh * p.slices;
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int v = v0 + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
+            acc[j][e] = d < p.D && v < p.V ? p.S[((slb + v / kSl) * p.D + d) * kSl + v % kSl] : 0.f;
+        }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) nacc[e] = dr[e] < p.D ? p.n[(slb + v0 / kSl) * p.D + dr[e]] : 0.f;
+    for (int c = 0; c < p.nc; ++c) {
+        const size_t bc = bh * p.nc + c;
+        if (c + 1 < p.nc) {
+            load(c + 1, (c + 1) & 1);
+            cpa_wait<1>();
+        } else {
+            cpa_wait<0>();
+        }
+        const float rl = p.r[bc * kL + kL - 1];
+        if (tid < kL) ws[tid] = expf(rl + p.a[bc * kL + tid]);
+        // the state this chunk starts from
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                uint32_t hi, lo;
+                split_bf2(acc[j][2 * e], acc[j][2 * e + 1], hi, lo);
+                const size_t o = (bc * p.Dp + dr[e]) * p.Vp + v0 + 8 * j + 2 * t;
+                *reinterpret_cast<uint32_t*>(p.Shi + o) = hi;
+                *reinterpret_cast<uint32_t*>(p.Slo + o) = lo;
+            }
+        if (blockIdx.y == 0 && t == 0) {
+            p.nbuf[bc * p.Dp + dr[0]] = nacc[0];
+            p.nbuf[bc * p.Dp + dr[1]] = nacc[1];
+        }
+        __syncthreads();
+        const float keep = expf(rl + p.min_[bc]);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[j][e] *= keep;
+        float ns[2] = {0.f, 0.f};
+        const bf16* kt = ks[c & 1];
+        const bf16* vt = vs[c & 1];
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            uint32_t a[4], hi[4], lo[4];
+            ldsm4_t(smem_u32(kt + (16 * kk + (lane >> 4) * 8 + (lane & 7)) * kLd + 16 * warp + ((lane >> 3) & 1) * 8), a[0], a[1], a[2], a[3]);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int s = 16 * kk + 2 * t + 8 * (i >> 1);
+                const float x = bf_lo(a[i]) * ws[s], y = bf_hi(a[i]) * ws[s + 1];
+                ns[i & 1] += x + y;
+                split_bf2(x, y, hi[i], lo[i]);
+            }
+#pragma unroll
+            for (int jp = 0; jp < 4; ++jp) {
+                uint32_t b0, b1, b2, b3;
+                ldsm4_t(smem_u32(vt + (16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
+                mma_bf16(acc[2 * jp], hi[0], hi[1], hi[2], hi[3], b0, b1);
+                mma_bf16(acc[2 * jp], lo[0], lo[1], lo[2], lo[3], b0, b1);
+                mma_bf16(acc[2 * jp + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+                mma_bf16(acc[2 * jp + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 1);
+            ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 2);
+            nacc[e] = keep * nacc[e] + ns[e];
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int v = v0 + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
+            if (d < p.D && v < p.V) p.S[((slb + v / kSl) * p.D + d) * kSl + v % kSl] = acc[j][e];
+        }
+    if (t == 0)
+        for (int s = v0 / kSl; s < min(p.slices, (v0 + kTd) / kSl); ++s)
+#pragma unroll
+            for (int e = 0; e < 2; ++e)
+                if (dr[e] < p.D) p.n[(slb + s) * p.D + dr[e]] = nacc[e];
+}
+
+// outputs of a chunk: 64 positions x VT value columns of a head
+template <int VT>
+__global__ void __launch_bounds__(128) mlstm_out_kernel(const MlParams p) {
+    constexpr int LV = VT + 8, NV = VT / 8;
+    extern __shared__ __align__(16) unsigned char ml_raw[];
+    bf16* qs = reinterpret_cast<bf16*>(ml_raw);          // [64][72]
+    bf16* ks = qs + kL * kLd;                            // [64][72]
+    bf16* sh = ks + kL * kLd;                            // [64][LV]
+    bf16* slo = sh + kTd * LV;                           // [64][LV]
+    bf16* vs = slo + kTd * LV;                           // [64][LV]
+    __shared__ float sa[kL], sr[kL], sm[kL], sqn[kL], sn[kTd];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.z % p.H, b = blockIdx.z / p.H, c = blockIdx.y, v0 = blockIdx.x * VT;
+    const size_t bc = (size_t)blockIdx.z * p.nc + c;
+    const bf16* base = reinterpret_cast<const bf16*>(p.qkvg);
+    pdl_wait();
+    pdl_release();
+    auto row_of = [&](int s) { return ((size_t)b * p.Tall + p.t0 + c * kL + s) * p.ldp; };
+    for (int i = tid; i < kL * (VT / 8); i += 128) {
+        const int s = i / (VT / 8), cc = (i % (VT / 8)) * 8;
+        const bool live = c * kL + s < p.T && v0 + cc < p.V;
+        cpa16(smem_u32(vs + s * LV + cc), live ? base + row_of(s) + (size_t)2 * p.H * p.D + (size_t)h * p.V + v0 + cc : base, live);
+    }
+    if (tid < kL) {
+        sa[tid] = p.a[bc * kL + tid];
+        sr[tid] = p.r[bc * kL + tid];
+        sm[tid] = p.mt[bc * kL + tid];
+    }
+    float qk[8][4], acc[NV][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) qk[j][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+    float qn = 0.f;                                      // row tid / 2, half tid % 2 of q . n
+    for (int d0 = 0; d0 < p.Dp; d0 += kTd) {
+        __syncthreads();
+        for (int i = tid; i < kL * 8; i += 128) {
+            const int s = i >> 3, cc = (i & 7) * 8;
+            const bool live = c * kL + s < p.T && d0 + cc < p.D;
+            const bf16* src = live ? base + row_of(s) + (size_t)h * p.D + d0 + cc : base;
+            cpa16(smem_u32(qs + s * kLd + cc), src, live);
+            cpa16(smem_u32(ks + s * kLd + cc), live ? src + (size_t)p.H * p.D : base, live);
+        }
+        for (int i = tid; i < kTd * (VT / 8); i += 128) {
+            const int d = i / (VT / 8), cc = (i % (VT / 8)) * 8;
+            const bool live = v0 + cc < p.Vp;
+            const size_t o = (bc * p.Dp + d0 + d) * p.Vp + v0 + cc;
+            cpa16(smem_u32(sh + d * LV + cc), p.Shi + (live ? o : 0), live);
+            cpa16(smem_u32(slo + d * LV + cc), p.Slo + (live ? o : 0), live);
+        }
+        cpa_commit();
+        if (tid < kTd) sn[tid] = p.nbuf[bc * p.Dp + d0 + tid];
+        cpa_wait<0>();
+        __syncthreads();
+        {
+            const bf16* qr = qs + (tid >> 1) * kLd + (tid & 1) * 32;
+            const float* nr = sn + (tid & 1) * 32;
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) {
+                const uint32_t w = *reinterpret_cast<const uint32_t*>(qr + i);
+                qn += bf_lo(w) * nr[i] + bf_hi(w) * nr[i + 1];
+            }
+        }
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            uint32_t a0, a1, a2, a3;
+            ldsm4(smem_u32(qs + (16 * warp + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 16 * kk + (lane >> 4) * 8), a0, a1, a2, a3);
+#pragma unroll
+            for (int jp = 0; jp < 4; ++jp) {
+                if (jp > warp) continue;                 // keys after every query of this warp
+                uint32_t b0, b1, b2, b3;
+                ldsm4(smem_u32(ks + (16 * jp + (lane & 7) + (lane >> 4) * 8) * kLd + 16 * kk + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
+                mma_bf16(qk[2 * jp], a0, a1, a2, a3, b0, b1);
+                mma_bf16(qk[2 * jp + 1], a0, a1, a2, a3, b2, b3);
+            }
+            const int srow = 16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8;
+#pragma unroll
+            for (int jp = 0; jp < NV / 2; ++jp) {
+                uint32_t b0, b1, b2, b3;
+                ldsm4_t(smem_u32(sh + srow * LV + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
+                mma_bf16(acc[2 * jp], a0, a1, a2, a3, b0, b1);
+                mma_bf16(acc[2 * jp + 1], a0, a1, a2, a3, b2, b3);
+                ldsm4_t(smem_u32(slo + srow * LV + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
+                mma_bf16(acc[2 * jp], a0, a1, a2, a3, b0, b1);
+                mma_bf16(acc[2 * jp + 1], a0, a1, a2, a3, b2, b3);
+            }
+        }
+    }
+    qn += __shfl_xor_sync(0xffffffffu, qn, 1);
+    if ((tid & 1) == 0) sqn[tid >> 1] = qn;
+    __syncthreads();
+    const int tr[2] = {16 * warp + g, 16 * warp + g + 8};
+    const float m0 = p.min_[bc];
+    float den[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const float w = expf(sr[tr[e]] + m0) * p.scale;
+        den[e] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            acc[j][2 * e] *= w;
+            acc[j][2 * e + 1] *= w;
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int s = 8 * j + 2 * t + (e & 1), tt = tr[e >> 1];
+            const float v = s <= tt ? qk[j][e] * p.scale * expf(sr[tt] + sa[s]) : 0.f;
+            qk[j][e] = v;
+            den[e >> 1] += v;
+        }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+        if (kk > warp) continue;
+        uint32_t hi[4], lo[4];
+        split_bf2(qk[2 * kk][0], qk[2 * kk][1], hi[0], lo[0]);
+        split_bf2(qk[2 * kk][2], qk[2 * kk][3], hi[1], lo[1]);
+        split_bf2(qk[2 * kk + 1][0], qk[2 * kk + 1][1], hi[2], lo[2]);
+        split_bf2(qk[2 * kk + 1][2], qk[2 * kk + 1][3], hi[3], lo[3]);
+        const int srow = 16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8;
+#pragma unroll
+        for (int jp = 0; jp < NV / 2; ++jp) {
+            uint32_t b0, b1, b2, b3;
+            ldsm4_t(smem_u32(vs + srow * LV + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
+            mma_bf16(acc[2 * jp], hi[0], hi[1], hi[2], hi[3], b0, b1);
+            mma_bf16(acc[2 * jp], lo[0], lo[1], lo[2], lo[3], b0, b1);
+            mma_bf16(acc[2 * jp + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
+            mma_bf16(acc[2 * jp + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        den[e] += __shfl_xor_sync(0xffffffffu, den[e], 1);
+        den[e] += __shfl_xor_sync(0xffffffffu, den[e], 2);
+        const int tt = tr[e];
+        den[e] += expf(sr[tt] + m0) * p.scale * sqn[tt];
+        const float inv = 1.f / (fmaxf(fabsf(den[e]), expf(-sm[tt])) + 1e-6f);
+        if (c * kL + tt < p.T) {
+            float* o = p.o + ((size_t)b * p.Tall + p.t0 + c * kL + tt) * p.H * p.V + (size_t)h * p.V;
+#pragma unroll
+            for (int j = 0; j < NV; ++j) {
+                const int v = v0 + 8 * j + 2 * t;
+                if (v < p.V) *reinterpret_cast<float2*>(o + v) = make_float2(acc[j][2 * e] * inv, acc[j][2 * e + 1] * inv);
+            }
+        }
+    }
+}
+
+// one warp per (row, head)
+__global__ void __launch_bounds__(256) mlstm_norm_kernel(const MlParams p) {
+    pdl_wait();
+    pdl_release();
+    const long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (i >= (long long)p.B * p.T * p.H) return;
+    const int h = (int)(i % p.H);
+    const long long bt = i / p.H;
+    head_norm_gate<bf16>(p, (size_t)(bt / p.T) * p.Tall + p.t0 + bt % p.T, h, threadIdx.x & 31);
+}
+
+}  // namespace glq
+
+using namespace glq;
+
+extern "C" int glq_mlstm_slices(int V) { return (V + kSl - 1) / kSl; }
+
+static inline size_t up256d(size_t v) { return (v + 255) / 256 * 256; }
+static constexpr int kSegment = 4096;      // positions the chunk form takes at a time (bounds its workspace)
+
+struct MlWs {
+    size_t o, r, a, mt, min_, nbuf, hi, lo, total;
+};
+static MlWs ml_ws(const glq_mlstm_t* a, bool chunked) {
+    MlWs w{};
+    size_t at = 0;
+    auto take = [&](size_t bytes) {
+        const size_t v = at;
+        at += up256d(bytes);
+        return v;
+    };
+    w.o = take((size_t)a->B * a->T * a->H * a->V * 4);
+    if (chunked) {
+        const size_t bh = (size_t)a->B * a->H, nc = cdiv_i(std::min(a->T, kSegment), kL), Dp = (a->D + 63) / 64 * 64, Vp = (a->V + 63) / 64 * 64;
+        w.r = take(bh * nc * kL * 4);
+        w.a = take(bh * nc * kL * 4);
+        w.mt = take(bh * nc * kL * 4);
+        w.min_ = take(bh * nc * 4);
+        w.nbuf = take(bh * nc * Dp * 4);
+        w.hi = take(bh * nc * Dp * Vp * 2);
+        w.lo = take(bh * nc * Dp * Vp * 2);
+    }
+    w.total = at;
+    return w;
+}
+extern "C" size_t glq_mlstm_workspace_bytes(const glq_mlstm_t* a, int chunked) { return ml_ws(a, chunked != 0).total; }
+
+static int ml_params(const glq_mlstm_t* a, MlParams& p, bool chunked) {
+    if (!a || a->B <= 0 || a->T < 0 || a->H <= 0 || a->D <= 0 || a->V <= 0 || !(a->gate_cap > 0.f)) return GLQ_ERR_ARG;
+    if (!a->qkvg || !a->gates || !a->bias_i || !a->bias_f || !a->norm_w || !a->S || !a->n || !a->m || !a->out || !a->workspace || !a->counters)
+        return GLQ_ERR_ARG;
+    if (!al16(a->S) || !al16(a->workspace)) return GLQ_ERR_ALIGN;
+    const MlWs w = ml_ws(a, chunked);
+    if (a->workspace_bytes < w.total) return GLQ_ERR_WORKSPACE;
+    if (a->D > 8192 || (long)a->B * a->H > 65535) return GLQ_ERR_UNSUPPORTED;
+    char* ws = reinterpret_cast<char*>(a->workspace);
+    p.qkvg = a->qkvg;
+    p.gates = a->gates;
+    p.bias_i = a->bias_i;
+    p.bias_f = a->bias_f;
+    p.norm_w = a->norm_w;
+    p.S = a->S;
+    p.n = a->n;
+    p.m = a->m;
+    p.out = a->out;
+    p.o = reinterpret_cast<float*>(ws + w.o);
+    p.counters = a->counters;
+    p.ldp = a->ldp;
+    p.ldg = a->ldg;
+    p.B = a->B;
+    p.T = p.Tall = a->T;
+    p.H = a->H;
+    p.D = a->D;
+    p.V = a->V;
+    p.slices = glq_mlstm_slices(a->V);
+    p.state_idle = a->state_idle;
+    p.cap = a->gate_cap;
+    p.eps = a->eps;
+    p.scale = (float)(1.0 / sqrt((double)a->D));
+    if (chunked) {
+        p.r = reinterpret_cast<float*>(ws + w.r);
+        p.a = reinterpret_cast<float*>(ws + w.a);
+        p.mt = reinterpret_cast<float*>(ws + w.mt);
+        p.min_ = reinterpret_cast<float*>(ws + w.min_);
+        p.nbuf = reinterpret_cast<float*>(ws + w.nbuf);
+        p.Shi = reinterpret_cast<bf16*>(ws + w.hi);
+        p.Slo = reinterpret_cast<bf16*>(ws + w.lo);
+        p.Dp = (a->D + 63) / 64 * 64;
+        p.Vp = (a->V + 63) / 64 * 64;
+    }
+    return GLQ_OK;
+}
+
+extern "C" int glq_mlstm_step(const glq_mlstm_t* a, void* stream) {
+    MlParams p{};
+    const int st = ml_params(a, p, false);
+    if (st != GLQ_OK) return st;
+    if (p.T == 0) return GLQ_OK;
+    const dim3 grid(p.slices, p.B * p.H);
+    const size_t smem = (size_t)2 * p.D * 4;
+    if (a->dtype == GLQ_DT_BF16) return dn_launch(mlstm_step_kernel<bf16>, grid, 256, smem, stream, p);
+    if (a->dtype == GLQ_DT_F32) return dn_launch(mlstm_step_kernel<float>, grid, 256, smem, stream, p);
+    return GLQ_ERR_ARG;
+}
+
+extern "C" int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream) {
+    if (!a || a->dtype != GLQ_DT_BF16) return GLQ_ERR_ARG;
+    if (a->D % 8 || a->V % 8 || a->ldp % 8) return GLQ_ERR_UNSUPPORTED;
+    MlParams p{};
+    int st = ml_params(a, p, true);
+    if (st != GLQ_OK) return st;
+    if (!al16(a->qkvg)) return GLQ_ERR_ALIGN;
+    const int bh = p.B * p.H;
+    for (p.t0 = 0; p.t0 < p.Tall; p.t0 += kSegment) {
+        p.T = std::min(kSegment, p.Tall - p.t0);
+        p.nc = cdiv_i(p.T, kL);
+        if ((st = dn_launch(mlstm_gate_kernel, dim3(bh), 256, (size_t)3 * p.nc * 4, stream, p)) != GLQ_OK) return st;
+        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 128, 0, stream, p)) != GLQ_OK) return st;
+        constexpr size_t fixed = (size_t)2 * kL * kLd * 2;
+        if (p.V > 64)
+            st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, fixed + (size_t)3 * 64 * 136 * 2, stream, p);
+        else
+            st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, fixed + (size_t)3 * 64 * 72 * 2, stream, p);
+        if (st != GLQ_OK) return st;
+        if ((st = dn_launch(mlstm_norm_kernel, dim3(cdiv_i((long)p.B * p.T * p.H, 8)), 256, 0, stream, p)) != GLQ_OK) return st;
+    }
+    return GLQ_OK;
+}

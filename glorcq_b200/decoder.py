@@ -55,6 +55,15 @@ class StaticKVCache:
         self.k.zero_()
         self.v.zero_()
 
+    def snapshot(self, positions):
+        """Entries below `positions`, for ``restore`` after trial steps there (see glorcq_b200.cache)."""
+        return self.k[:, :, :, :positions].clone(), self.v[:, :, :, :positions].clone()
+
+    def restore(self, saved):
+        n = saved[0].shape[3]
+        self.k[:, :, :, :n].copy_(saved[0])
+        self.v[:, :, :, :n].copy_(saved[1])
+
     def update(self, layer, k_new, v_new, cache_position):
         """Write (B, kv_heads, T, D) at positions cache_position (T,) and return the layer's full buffers."""
         b = k_new.shape[0]
@@ -307,6 +316,9 @@ class GLoRCQDecoder(nn.Module):
         self._own_cache = None
         self._lm_ws = {}
         self.last_argmax = None     # (B * kept positions,) int64 greedy tokens of the last forward, when the kernel ran
+
+    def make_cache(self, max_batch_size, max_cache_len):
+        return StaticKVCache(self.config, max_batch_size, max_cache_len, self.embed_tokens.device, self.embed_tokens.dtype)
 
     def _tables(self, need, device):
         if self._rope is None or self._rope[0].shape[0] < need:

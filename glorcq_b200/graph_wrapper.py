@@ -30,8 +30,10 @@ class GLoRCQGraphWrapper:
         self.max_seq_len = max_seq_len
         self.device = next(model.parameters()).device
         self.dtype = next(model.parameters()).dtype
-        self.static_cache = StaticCache(config=model.config, max_batch_size=max_batch_size, max_cache_len=max_seq_len,
-                                        device=self.device, dtype=self.dtype)
+        # a model of this package makes its own cache (key/value positions, latents, recurrent state)
+        self.static_cache = model.make_cache(max_batch_size, max_seq_len) if hasattr(model, "make_cache") else \
+            StaticCache(config=model.config, max_batch_size=max_batch_size, max_cache_len=max_seq_len, device=self.device,
+                        dtype=self.dtype)
         self.static_input_ids = torch.zeros((max_batch_size, 1), dtype=torch.long, device=self.device)
         self.static_cache_position = torch.zeros((1,), dtype=torch.long, device=self.device)
         self.static_logits = None
@@ -55,7 +57,15 @@ class GLoRCQGraphWrapper:
 
     def capture_graph(self):
         """Allocation pass, three warm-up steps on a side stream, then the recorded step
-        (inference/graph_wrapper.py:69-130)."""
+        (inference/graph_wrapper.py:69-130).  The steps run at positions 0 and 10 of the static cache and advance
+        recurrent state; what they overwrite is put back, so a capture may happen in the middle of a sequence."""
+        saved = self.static_cache.snapshot(11) if hasattr(self.static_cache, "snapshot") else None
+        self._capture()
+        if saved is not None:
+            self.static_cache.restore(saved)
+        torch.cuda.synchronize()
+
+    def _capture(self):
         self.model.eval()
         self._set_moe_graph_mode(True)
         with torch.no_grad():
@@ -95,6 +105,24 @@ class GLoRCQGraphWrapper:
         return self.static_logits
 
     @torch.no_grad()
+    def step(self, input_ids, position, logits_to_keep=1):
+        """The next tokens (B, T) of every sequence, starting at `position`: eager for T > 1 (a prompt or a portion
+        of one), the replayed step for T = 1.  Returns logits (B, kept, V); a replayed step's buffer is overwritten
+        by the next one."""
+        T = input_ids.shape[1]
+        if position + T > self.max_seq_len:
+            raise ValueError(f"position {position + T - 1} is beyond max_seq_len {self.max_seq_len}")
+        self._set_moe_graph_mode(T == 1)
+        if T == 1:
+            if self.graph is None:
+                self.capture_graph()
+            logits = self.replay(input_ids, position)
+            return logits[:, logits_to_keep] if torch.is_tensor(logits_to_keep) else logits
+        kw = {"logits_to_keep": logits_to_keep} if self._keep_last_only else {}
+        return self.model(input_ids=input_ids, cache_position=torch.arange(position, position + T, device=self.device),
+                          past_key_values=self.static_cache, use_cache=True, return_dict=False, **kw)[0]
+
+    @torch.no_grad()
     def generate(self, input_ids, max_new_tokens=100):
         """Greedy decoding: eager prefill, graph replay per new token.  Returns (ids (B, T + new),
         seconds) like the reference (inference/graph_wrapper.py:152-212)."""
@@ -103,23 +131,15 @@ class GLoRCQGraphWrapper:
         assert batch_size == self.max_batch_size, \
             f"Input batch_size ({batch_size}) must match max_batch_size ({self.max_batch_size})"
         output_ids = input_ids.clone()
-        self._set_moe_graph_mode(False)
         self.static_cache.reset()
-        kw = {"logits_to_keep": 1} if self._keep_last_only else {}
-        logits = self.model(input_ids=input_ids, cache_position=torch.arange(seq_len, device=self.device),
-                            past_key_values=self.static_cache, use_cache=True, return_dict=False, **kw)[0]
+        logits = self.step(input_ids, 0)
         next_token = torch.argmax(logits[:, -1, :], dim=-1, keepdim=True)
         output_ids = torch.cat([output_ids, next_token], dim=1)
         torch.cuda.synchronize()
         prefill_end = time.time()
         self._set_moe_graph_mode(True)
         if self.graph is None:
-            # capturing runs steps at positions 0 and 10 of the static cache: keep the prompt's entries
-            keep_k, keep_v = self.static_cache.k[:, :, :, :11].clone(), self.static_cache.v[:, :, :, :11].clone()
             self.capture_graph()
-            self.static_cache.k[:, :, :, :11].copy_(keep_k)
-            self.static_cache.v[:, :, :, :11].copy_(keep_v)
-            torch.cuda.synchronize()
             prefill_end = time.time()
         for i in range(max_new_tokens - 1):
             pos = seq_len + i
