@@ -822,7 +822,22 @@ def main():
                          "side); default min(N, 4)")
     ap.add_argument("--replicas", action="store_true",
                     help="with --gpus N > 1: N independent copies of the model instead of expert parallelism")
+    ap.add_argument("--design", choices=["zokunex"], default=None,
+                    help="time another design of the framework beside the quantized decoder of equal size instead: decode and "
+                         "prompt rates of both, and a roofline table of the kernels (see --size, --prompt, --batch, --layers)")
+    ap.add_argument("--size", choices=["small", "medium", "large"], default="medium", help="with --design")
     args = ap.parse_args()
+    if args.design:
+        from glorcq_b200 import _build, benchmark
+        _build.build_all()
+        torch.cuda.set_device(0)
+        sampler = ClockSampler(0)
+        sampler.start()
+        line = benchmark.run(args.size, args.prompt or 4096, max(1, args.steps), args.batch, args.layers or 8, measured_peak_gbs()[0],
+                             measured_peak_tflops()[0], kernels=not args.no_extras)
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+        return
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))

@@ -288,6 +288,54 @@ def make_decoder(hf_config: dict, device, seed=0, qbit=2, attn_bits=4, rank=64, 
                          ep_group=ep_group, peer_exchange_max_tokens=peer_exchange_max_tokens)
 
 
+class _RandomWeights:
+    """{name: tensor} drawn on the device when asked for: a large model's tensors never exist twice."""
+
+    def __init__(self, shapes, device, seed, dtype=torch.bfloat16):
+        self.shapes, self.dtype = shapes, dtype
+        self.g = torch.Generator(device=device)
+        self.g.manual_seed(seed)
+        self.device = device
+
+    def __contains__(self, name):
+        return name in self.shapes
+
+    def __getitem__(self, name):
+        shape = self.shapes[name]
+        leaf = name.split(".", 1)[-1]
+        if leaf.endswith("norm") or leaf in ("norm1", "norm2"):
+            return torch.ones(shape, device=self.device, dtype=self.dtype)
+        gain = {"mix.f.b": 1.0, "mix.i.b": 1.0, "mlp.correction": 0.01}.get(leaf, shape[-1] ** -0.5)
+        t = torch.randn(shape, generator=self.g, device=self.device) * gain
+        return (t + 4 if leaf == "mix.f.b" else t).to(self.dtype)
+
+
+def make_zokunex(cfg, device, seed=0, dtype=torch.bfloat16):
+    """A Zokunex decoder of the given configuration with random weights, built on the device."""
+    from .zokunex import ZokunexDecoder, tensor_shapes
+    return ZokunexDecoder(cfg, _RandomWeights(tensor_shapes(cfg), device, seed), device, dtype)
+
+
+def zokunex_bytes_per_token(cfg, context, batch=1):
+    """Bytes one decode step of `batch` sequences has to move: the weights it touches (bf16; distinct experts at most),
+    the matrix memories (read and written) and the cached latents of `context` positions."""
+    C, n = cfg["width"], 2.0 * cfg["vocab"] * cfg["width"]
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer.get("mlp")
+        H, D, V = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "mlstm":
+            n += 2.0 * C * (2 * H * (D + V) + 2 * H + H * V) + batch * 8.0 * H * D * V
+        else:
+            R, K = m["rot_dim"], m["kv_rank"]
+            n += 2.0 * (C * (H * (D + R) + K + R + H + H * V) + H * K * (D + V)) + batch * context * 2.0 * (K + R)
+        if mlp and mlp["kind"] == "dense":
+            n += 4.0 * C * mlp["ff"]
+        elif mlp:
+            r = mlp["router"]
+            n += 2.0 * C * (r["experts"] + r["identity"]) + min(r["experts"], batch * r["top"]) * 4.0 * C * mlp["expert"]["ff"]
+    return int(n)
+
+
 QWEN15_MOE_A27B = dict(hidden_size=2048, num_hidden_layers=24, num_attention_heads=16, num_key_value_heads=16,
                        vocab_size=151936, num_experts=60, num_experts_per_tok=4, moe_intermediate_size=1408,
                        shared_expert_intermediate_size=5632, norm_topk_prob=False, rms_norm_eps=1e-6,

@@ -85,11 +85,12 @@ class ZokunexDecoder(nn.Module):
         if dtype not in dense.DTYPES:
             raise ValueError(f"dtype {dtype} is not supported")
         shapes = tensor_shapes(cfg)
-        for name, shape in shapes.items():
+        for name in shapes:
             if name not in weights:
                 raise KeyError(f"missing tensor {name}")
-            if tuple(weights[name].shape) != tuple(shape):
-                raise ValueError(f"tensor {name} has shape {tuple(weights[name].shape)}, expected {tuple(shape)}")
+        for name, t in (weights.items() if hasattr(weights, "items") else ()):
+            if name in shapes and tuple(t.shape) != tuple(shapes[name]):
+                raise ValueError(f"tensor {name} has shape {tuple(t.shape)}, expected {tuple(shapes[name])}")
         device = torch.device(device)
         self.raw_config, self.eps, self.logit_scale = cfg, float(cfg["norm"]["eps"]), float(cfg["logit_scale"])
         self.config = SimpleNamespace(vocab_size=cfg["vocab"], hidden_size=cfg["width"], num_hidden_layers=len(cfg["layers"]),

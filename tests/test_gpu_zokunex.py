@@ -16,7 +16,7 @@ from tests import zokunex_cases as Z
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CONFIGS = {"mixed": Z.MIXED, "odd": Z.ODD, "wide": Z.WIDE}
-TOL = {torch.float32: 1e-4, torch.bfloat16: 0.06}
+TOL = {torch.float32: 1e-4, torch.bfloat16: 0.1}
 
 
 @pytest.fixture(scope="module")
