@@ -131,15 +131,16 @@ class DenseMM(C.Structure):
     """glq_dense_mm_t"""
     _fields_ = [(f, C.c_int32) for f in ("dtype", "act", "N", "K", "rows", "n_matrices", "max_slots", "max_slot_rows", "split")] + \
                [("alpha", C.c_float)] + [(f, vp) for f in ("slot_index", "n_slots", "slot_count", "slot_offset", "entry_row", "x")] + \
-               [("ldx", C.c_int64), ("W", vp), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp)]
+               [("ldx", C.c_int64), ("W", vp), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp),
+                ("hn_o", vp), ("hn_g", vp), ("hn_ldg", C.c_int64), ("hn_w", vp), ("hn_heads", C.c_int32), ("hn_eps", C.c_float)]
 
 
 class MLstm(C.Structure):
     """glq_mlstm_t"""
     _fields_ = [(f, C.c_int32) for f in ("dtype", "B", "T", "H", "D", "V", "state_idle")] + \
                [("gate_cap", C.c_float), ("eps", C.c_float), ("qkvg", vp), ("ldp", C.c_int64), ("gates", vp), ("ldg", C.c_int64)] + \
-               [(f, vp) for f in ("bias_i", "bias_f", "norm_w", "S", "n", "m", "out", "workspace")] + \
-               [("workspace_bytes", C.c_size_t), ("counters", vp)]
+               [(f, vp) for f in ("bias_i", "bias_f", "norm_w", "S", "n", "m", "o", "out", "workspace")] + \
+               [("workspace_bytes", C.c_size_t)]
 
 
 class Latent(C.Structure):
@@ -169,7 +170,7 @@ _DENSE_SIGS = {
     "glq_dense_embed": (_i, [_i, vp, vp, _i, _i, _i, vp, vp, vp]),
     "glq_dense_add_norm": (_i, [_i, vp, vp, vp, _f, _i, _i, vp, vp, vp]),
     "glq_mlstm_slices": (_i, [_i]),
-    "glq_mlstm_workspace_bytes": (_z, [C.POINTER(MLstm), _i]),
+    "glq_mlstm_workspace_bytes": (_z, [C.POINTER(MLstm)]),
     "glq_mlstm_step": (_i, [C.POINTER(MLstm), vp]),
     "glq_mlstm_chunk": (_i, [C.POINTER(MLstm), vp]),
     "glq_latent_prep": (_i, [C.POINTER(Latent), vp]),

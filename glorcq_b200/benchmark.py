@@ -140,7 +140,7 @@ def decode_kernels(t, size, context, batch=1):
     states = [MatrixMemoryState(B, H, D, V, dev) for _ in range(n)]
     qkvg, gates = torch.randn(B, 2 * H * (D + V), device=dev).to(bf), torch.randn(B, 2 * H, device=dev)
     one, bias = torch.ones(H * V, device=dev), torch.zeros(H, device=dev)
-    sec = graph_time([lambda st=st: dense.mlstm(qkvg, gates, B, 1, H, D, V, 15.0, 1e-5, bias, bias, one, st, False, True) for st in states])
+    sec = graph_time([lambda st=st: dense.mlstm(qkvg, gates, B, 1, H, D, V, 15.0, 1e-5, bias, bias, one, st, False, True, True) for st in states])
     t.add(f"mLSTM step ({B} x {H} heads, {D} x {V})", sec, B * H * D * V * 8, 0, "decode attention")
 
     hh, d, r, v, k = s["la"]

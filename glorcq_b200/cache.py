@@ -41,7 +41,6 @@ class MatrixMemoryState:
         self.S = torch.zeros(batch, heads, sl, dim, 32, device=device)
         self.n = torch.zeros(batch, heads, sl, dim, device=device)
         self.m = torch.zeros(batch, heads, sl, device=device)
-        self.counters = torch.zeros(batch * heads, device=device, dtype=torch.int32)     # arrival counters, zero between calls
 
     def reset(self):
         self.S.zero_()

@@ -56,7 +56,88 @@ __device__ __forceinline__ void norm_add_row(float* ys, float* red, const float*
     for (int c = threadIdx.x; c < C; c += kRowThreads) h[c] = from_f<T>((ys[c] - mean2) * inv2 * fw[c]);
 }
 
-template <typename T>
+// The same with the row in registers: 8 consecutive values per thread and step, STEPS * 8 * kRowThreads values at most.
+// load(c, v): the sublayer's output at columns c .. c + 7, given x there
+template <typename T> __device__ __forceinline__ void st8(T* p, const float (&v)[8]);
+template <> __device__ __forceinline__ void st8<float>(float* p, const float (&v)[8]) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> __device__ __forceinline__ void st8<bf16>(bf16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]), pack_bf2(v[4], v[5]), pack_bf2(v[6], v[7]));
+}
+__device__ __forceinline__ void ld8(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+}
+__device__ __forceinline__ void ld8(const bf16* p, float (&v)[8]) {
+    const uint4 w = *reinterpret_cast<const uint4*>(p);
+    v[0] = bf_lo(w.x), v[1] = bf_hi(w.x), v[2] = bf_lo(w.y), v[3] = bf_hi(w.y);
+    v[4] = bf_lo(w.z), v[5] = bf_hi(w.z), v[6] = bf_lo(w.w), v[7] = bf_hi(w.w);
+}
+template <typename T, int STEPS, typename F>
+__device__ __forceinline__ void norm_add_row_regs(float* red, const float* __restrict__ w, const float* __restrict__ fw, float eps, int C,
+                                                  float* __restrict__ x, T* __restrict__ h, F load) {
+    float xv[STEPS][8], yv[STEPS][8];
+    float s = 0.f;
+#pragma unroll
+    for (int u = 0; u < STEPS; ++u) {
+        const int c = (u * kRowThreads + threadIdx.x) * 8;
+        if (c < C) {
+            ld8(x + c, xv[u]);
+            load(c, xv[u], yv[u]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s += yv[u][i];
+        }
+    }
+    const float mean = block_sum(s, red) / C;
+    s = 0.f;
+#pragma unroll
+    for (int u = 0; u < STEPS; ++u)
+        if ((u * kRowThreads + threadIdx.x) * 8 < C)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s += (yv[u][i] - mean) * (yv[u][i] - mean);
+    const float inv = 1.f / sqrtf(block_sum(s, red) / C + eps);
+    s = 0.f;
+#pragma unroll
+    for (int u = 0; u < STEPS; ++u) {
+        const int c = (u * kRowThreads + threadIdx.x) * 8;
+        if (c < C) {
+            float wv[8];
+            ld8(w + c, wv);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                xv[u][i] += (yv[u][i] - mean) * inv * wv[i];
+                s += xv[u][i];
+            }
+            st8<float>(x + c, xv[u]);
+            if (!fw) st8<T>(h + c, xv[u]);
+        }
+    }
+    if (!fw) return;
+    const float mean2 = block_sum(s, red) / C;
+    s = 0.f;
+#pragma unroll
+    for (int u = 0; u < STEPS; ++u)
+        if ((u * kRowThreads + threadIdx.x) * 8 < C)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s += (xv[u][i] - mean2) * (xv[u][i] - mean2);
+    const float inv2 = 1.f / sqrtf(block_sum(s, red) / C + eps);
+#pragma unroll
+    for (int u = 0; u < STEPS; ++u) {
+        const int c = (u * kRowThreads + threadIdx.x) * 8;
+        if (c < C) {
+            float wv[8];
+            ld8(fw + c, wv);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) wv[i] *= (xv[u][i] - mean2) * inv2;
+            st8<T>(h + c, wv);
+        }
+    }
+}
+
+// STEPS 0: any width, through shared memory
+template <typename T, int STEPS>
 __global__ void __launch_bounds__(kRowThreads) dense_add_norm_kernel(const float* __restrict__ y, const float* __restrict__ w,
                                                                      const float* __restrict__ fw, float eps, int C,
                                                                      float* __restrict__ x, T* __restrict__ h) {
@@ -65,12 +146,16 @@ __global__ void __launch_bounds__(kRowThreads) dense_add_norm_kernel(const float
     pdl_wait();
     pdl_release();
     const size_t o = (size_t)blockIdx.x * C;
-    for (int c = threadIdx.x; c < C; c += kRowThreads) ys[c] = y[o + c];
-    norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
+    if constexpr (STEPS > 0) {
+        norm_add_row_regs<T, STEPS>(red, w, fw, eps, C, x + o, h + o, [&](int c, const float (&)[8], float (&v)[8]) { ld8(y + o + c, v); });
+    } else {
+        for (int c = threadIdx.x; c < C; c += kRowThreads) ys[c] = y[o + c];
+        norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
+    }
 }
 
 // experts' outputs of a token in slot order; a slot without an entry passes the layer's input through
-template <typename T>
+template <typename T, int STEPS>
 __global__ void __launch_bounds__(kRowThreads) dense_combine_norm_kernel(const T* __restrict__ eo, long long lde,
                                                                          const int* __restrict__ tok_entries,
                                                                          const float* __restrict__ wts, int top,
@@ -81,15 +166,36 @@ __global__ void __launch_bounds__(kRowThreads) dense_combine_norm_kernel(const T
     pdl_wait();
     pdl_release();
     const size_t row = blockIdx.x, o = row * C;
-    for (int c = threadIdx.x; c < C; c += kRowThreads) {
-        float a = 0.f;
-        for (int j = 0; j < top; ++j) {
-            const int e = tok_entries[row * top + j];
-            a += wts[row * top + j] * (e >= 0 ? to_f(eo[(size_t)e * lde + c]) : x[o + c]);
+    if constexpr (STEPS > 0) {
+        norm_add_row_regs<T, STEPS>(red, w, fw, eps, C, x + o, h + o, [&](int c, const float (&xv)[8], float (&v)[8]) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = 0.f;
+#pragma unroll 4
+            for (int j = 0; j < top; ++j) {
+                const int e = __ldg(tok_entries + row * top + j);
+                const float g = __ldg(wts + row * top + j);
+                float u[8];
+                if (e >= 0) {
+                    ld8(eo + (size_t)e * lde + c, u);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) u[i] = xv[i];
+                }
+#pragma unroll
+                for (int i = 0; i < 8; ++i) v[i] += g * u[i];
+            }
+        });
+    } else {
+        for (int c = threadIdx.x; c < C; c += kRowThreads) {
+            float a = 0.f;
+            for (int j = 0; j < top; ++j) {
+                const int e = tok_entries[row * top + j];
+                a += wts[row * top + j] * (e >= 0 ? to_f(eo[(size_t)e * lde + c]) : x[o + c]);
+            }
+            ys[c] = a;
         }
-        ys[c] = a;
+        norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
     }
-    norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
 }
 
 // ---- routing -------------------------------------------------------------------------------------------
@@ -111,17 +217,30 @@ struct RtParams {
 };
 
 // one token by one warp: s = softmax(logits); `top` times the largest remaining s + correction, lowest index on ties.
-// sc: A floats of shared memory of this warp
-__device__ __forceinline__ void route_corrected(const RtParams& p, int t, int lane, float* sc) {
+// sc: 2 * A floats of shared memory of this warp; s_sel, s_wts: the token's choices in shared memory as well, or NULL
+__device__ __forceinline__ void route_corrected(const RtParams& p, int t, int lane, float* sc, int* s_sel, float* s_wts) {
     const float* row = p.logits + (size_t)t * p.ldl;
+    float* score = sc + p.A;
     float mx = -INFINITY;
-    for (int e = lane; e < p.A; e += 32) mx = fmaxf(mx, row[e]);
+    for (int e = lane; e < p.A; e += 32) {
+        const float v = row[e];
+        score[e] = v;
+        sc[e] = p.correction[e];
+        mx = fmaxf(mx, v);
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     float sum = 0.f;
-    for (int e = lane; e < p.A; e += 32) sum += expf(row[e] - mx);
+    for (int e = lane; e < p.A; e += 32) {
+        const float v = expf(score[e] - mx);
+        score[e] = v;
+        sum += v;
+    }
     sum = warp_sum(sum);
-    for (int e = lane; e < p.A; e += 32) sc[e] = expf(row[e] - mx) / sum + p.correction[e];
+    for (int e = lane; e < p.A; e += 32) {
+        score[e] /= sum;
+        sc[e] += score[e];
+    }
     __syncwarp();
     for (int j = 0; j < p.top; ++j) {
         float best = -INFINITY;
@@ -134,14 +253,19 @@ __device__ __forceinline__ void route_corrected(const RtParams& p, int t, int la
             const int oe = __shfl_xor_sync(0xffffffffu, be, o);
             if (ob > best || (ob == best && oe < be)) best = ob, be = oe;
         }
-        // nothing comparable left (scores that are no numbers): a slot of weight zero, on the first expert
+        // nothing comparable left (scores that are no numbers): a pass-through slot of weight zero
         const bool none = be == 0x7fffffff;
         if (lane == 0) {
-            const int e = none ? 0 : be;
-            p.sel[(size_t)t * p.top + j] = none ? p.A : e;
-            p.wts[(size_t)t * p.top + j] = none ? 0.f : expf(row[e] - mx) / sum;
+            const int sel = none ? p.A : be;
+            const float wt = none ? 0.f : score[be];
+            p.sel[(size_t)t * p.top + j] = sel;
+            p.wts[(size_t)t * p.top + j] = wt;
             p.tok_entries[(size_t)t * p.top + j] = -1;
-            if (!none) sc[e] = -INFINITY;
+            if (s_sel) {
+                s_sel[t * p.top + j] = sel;
+                s_wts[t * p.top + j] = wt;
+            }
+            if (!none) sc[be] = -INFINITY;
         }
         __syncwarp();
     }
@@ -153,20 +277,23 @@ __global__ void __launch_bounds__(256) dense_route_kernel(const RtParams p) {
     pdl_release();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * 8 + warp;
-    if (t < p.n) route_corrected(p, t, lane, rt_sc + (size_t)warp * p.A);
+    if (t < p.n) route_corrected(p, t, lane, rt_sc + (size_t)warp * 2 * p.A, nullptr, nullptr);
 }
 
 // few entries: routing and lists in one CTA
+constexpr int kRouteOneCta = 1024;
 __global__ void __launch_bounds__(256) dense_route_plan_kernel(const RtParams p) {
     extern __shared__ float rt_sc[];
-    int* cnt = reinterpret_cast<int*>(rt_sc + (size_t)8 * p.A);
+    __shared__ int s_sel[kRouteOneCta];
+    __shared__ float s_wts[kRouteOneCta];
+    int* cnt = reinterpret_cast<int*>(rt_sc + (size_t)16 * p.A);
     pdl_wait();
     pdl_release();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int t = warp; t < p.n; t += 8) route_corrected(p, t, lane, rt_sc + (size_t)warp * p.A);
+    for (int t = warp; t < p.n; t += 8) route_corrected(p, t, lane, rt_sc + (size_t)warp * 2 * p.A, s_sel, s_wts);
     __syncthreads();
     const int ms = p.max_slots;
-    plan_entries<float>(cnt, p.n, p.E, p.top, p.chunk, 0, 1, p.sel, p.wts, p.active, p.n_active, p.slot_count, p.slot_offset,
+    plan_entries<float>(cnt, p.n, p.E, p.top, p.chunk, 0, 1, s_sel, s_wts, p.active, p.n_active, p.slot_count, p.slot_offset,
                         p.entry_row, p.entry_scale, p.tok_entries, p.active + ms, p.n_active + 1, p.slot_count + ms,
                         p.slot_offset + ms);
 }
@@ -198,7 +325,12 @@ extern "C" int glq_dense_add_norm(int dtype, const float* y, const float* w, con
     if (rows == 0) return GLQ_OK;
     return by_dtype(dtype, [&](auto z) {
         using T = decltype(z);
-        return dn_launch(dense_add_norm_kernel<T>, dim3(rows), kRowThreads, (size_t)C * 4, stream, y, w, final_w, eps, C, x, (T*)h);
+        const bool vec = C % 8 == 0 && al16(y) && al16(w) && al16(x) && al16(h) && al16(final_w);
+        if (vec && C <= 8 * kRowThreads)
+            return dn_launch(dense_add_norm_kernel<T, 1>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
+        if (vec && C <= 32 * kRowThreads)
+            return dn_launch(dense_add_norm_kernel<T, 4>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
+        return dn_launch(dense_add_norm_kernel<T, 0>, dim3(rows), kRowThreads, (size_t)C * 4, stream, y, w, final_w, eps, C, x, (T*)h);
     });
 }
 
@@ -210,8 +342,14 @@ extern "C" int glq_dense_combine_norm(int dtype, const void* entry_out, int64_t 
     if (rows == 0) return GLQ_OK;
     return by_dtype(dtype, [&](auto z) {
         using T = decltype(z);
-        return dn_launch(dense_combine_norm_kernel<T>, dim3(rows), kRowThreads, (size_t)C * 4, stream, (const T*)entry_out,
-                         (long long)lde, tok_entries, wts, top, w, final_w, eps, C, x, (T*)h);
+        const bool vec = C % 8 == 0 && lde % 8 == 0 && al16(entry_out) && al16(w) && al16(x) && al16(h) && al16(final_w);
+        auto go = [&](auto kern, size_t smem) {
+            return dn_launch(kern, dim3(rows), kRowThreads, smem, stream, (const T*)entry_out, (long long)lde, tok_entries, wts, top, w,
+                             final_w, eps, C, x, (T*)h);
+        };
+        if (vec && C <= 8 * kRowThreads) return go(dense_combine_norm_kernel<T, 1>, 0);
+        if (vec && C <= 32 * kRowThreads) return go(dense_combine_norm_kernel<T, 4>, 0);
+        return go(dense_combine_norm_kernel<T, 0>, (size_t)C * 4);
     });
 }
 
@@ -226,7 +364,7 @@ extern "C" int glq_route(const glq_route_t* a, void* stream) {
     if (!a->logits || !a->correction || !a->sel || !a->wts || !a->entry_scale || !a->tok_entries || !a->entry_row || !a->active ||
         !a->slot_count || !a->slot_offset || !a->n_active)
         return GLQ_ERR_ARG;
-    if (a->E + a->identity > 4096) return GLQ_ERR_UNSUPPORTED;
+    if (a->E + a->identity > 2048) return GLQ_ERR_UNSUPPORTED;
     if (a->n == 0) return GLQ_OK;
     if (a->max_slots < glq_route_max_slots(a->n, a->E, a->top, a->chunk)) return GLQ_ERR_WORKSPACE;
     RtParams p{};
@@ -249,8 +387,8 @@ extern "C" int glq_route(const glq_route_t* a, void* stream) {
     p.n_active = a->n_active;
     p.max_slots = a->max_slots;
     const int nk = a->n * a->top;
-    const size_t sc = (size_t)8 * p.A * 4;
-    if (nk < 1024) return dn_launch(dense_route_plan_kernel, dim3(1), 256, sc + (size_t)2 * p.E * 4, stream, p);
+    const size_t sc = (size_t)16 * p.A * 4;
+    if (nk <= kRouteOneCta && a->n <= 128) return dn_launch(dense_route_plan_kernel, dim3(1), 256, sc + (size_t)2 * p.E * 4, stream, p);
     if (!a->block_counts) return GLQ_ERR_ARG;
     int st = dn_launch(dense_route_kernel, dim3(cdiv_i(a->n, 8)), 256, sc, stream, p);
     if (st != GLQ_OK) return st;

@@ -31,6 +31,13 @@ struct DmParams {
     int N, K, rows, slots, split, act;
     float alpha;
     int vec_y, vec_y32;
+    int cluster, xs_max;             // streaming kernel: CTAs that share a tile's k range; activation row stride
+    const float* hn_o;               // streaming kernel: rows made from a recurrence's output (see glq_dense_mm_t)
+    const void* hn_g;
+    const float* hn_w;
+    long long hn_ldg;
+    int hn_heads;
+    float hn_eps;
 };
 
 struct DmSlot {
@@ -57,20 +64,46 @@ __device__ __forceinline__ uint4 dm_ldg(const uint4* p) {
                  : "l"(p));
     return v;
 }
-constexpr int kDmDepth = 8;
+__device__ __forceinline__ uint32_t cluster_rank() {
+    uint32_t r;
+    asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+    return r;
+}
+__device__ __forceinline__ uint32_t cluster_addr(uint32_t saddr, uint32_t rank) {
+    uint32_t a;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(saddr), "r"(rank));
+    return a;
+}
+__device__ __forceinline__ void st_cluster(uint32_t addr, float v) {
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory");
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+constexpr int kDmMaxCluster = 4;
+#ifndef GLQ_DM_DEPTH
+#define GLQ_DM_DEPTH 4
+#define GLQ_DM_CTAS 3
+#endif
 
-template <int SPLIT>   // warps that share one 16-row tile
-__global__ void __launch_bounds__(kThreads, 2) dense_stream_kernel(const DmParams p) {
+// SPLIT warps share one 16-row tile; with p.cluster > 1 the CTAs of a cluster share its k range as well, and the first of
+// them adds the others' sums (in rank order).  DEPTH 16-byte loads per lane and row are in flight.
+template <int SPLIT, int DEPTH, int CTAS>
+__global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmParams p) {
     constexpr int TILES = kWarpsPerCta / SPLIT;
     extern __shared__ __align__(16) unsigned char dm_smem[];
-    const int K = p.K, KP = (K + 31) / 32 * 32, XS = KP + 32;      // padded activation rows: distinct banks
-    bf16* xs = reinterpret_cast<bf16*>(dm_smem);
-    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * XS * 2);
-    const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
+    __shared__ float4 s_part[kDmMaxCluster][32];
+    const int K = p.K, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     const int g = lane >> 2, t = lane & 3;
     const int tw = w / SPLIT, s = w % SPLIT;
-    const int chunks = KP / 32;
-    const int c_lo = (int)((long)s * chunks / SPLIT), c_hi = (int)((long)(s + 1) * chunks / SPLIT);
+    const int cs = p.cluster, rank = cs > 1 ? (int)cluster_rank() : 0;
+    const int bx = (int)blockIdx.x / cs, nbx = (int)gridDim.x / cs;
+    // 32-channel chunks of this CTA, and of this warp inside it
+    const int chunks = (K + 31) / 32;
+    const int a_lo = (int)((long)rank * chunks / cs), a_hi = (int)((long)(rank + 1) * chunks / cs), an = a_hi - a_lo;
+    const int c_lo = a_lo + (int)((long)s * an / SPLIT), c_hi = a_lo + (int)((long)(s + 1) * an / SPLIT);
+    const int XS = (an + 1) * 32;                                  // padded activation rows: distinct banks
+    bf16* xs = reinterpret_cast<bf16*>(dm_smem);
+    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * p.xs_max * 2);
     const int ntiles = (p.N + 15) / 16;
     const bool plain = p.slot_index == nullptr;
     DmSlot sl{0, 0, p.rows};
@@ -78,82 +111,130 @@ __global__ void __launch_bounds__(kThreads, 2) dense_stream_kernel(const DmParam
         pdl_wait();
         pdl_release();
         sl = dm_slot(p, blockIdx.y);
-        if (sl.cnt == 0) return;
+        if (sl.cnt == 0) return;                                   // the whole cluster: its CTAs share blockIdx.y
     }
+    if (cs > 1) cluster_arrive();                                  // "this CTA runs": waited for before its memory is written
     const bf16* Wm = reinterpret_cast<const bf16*>(p.W) + (size_t)sl.mat * p.N * K;
-    const int iters = (ntiles + TILES * (int)gridDim.x - 1) / (TILES * (int)gridDim.x);
+    const int iters = (ntiles + TILES * nbx - 1) / (TILES * nbx);
     for (int it = 0; it < iters; ++it) {
-        const int tile = (it * (int)gridDim.x + (int)blockIdx.x) * TILES + tw;
+        const int tile = (it * nbx + bx) * TILES + tw;
         const bool live = tile < ntiles;
         const int r0 = min(tile * 16 + g, p.N - 1), r1 = min(tile * 16 + g + 8, p.N - 1);
         const bf16* w0 = Wm + (size_t)r0 * K + t * 8;
         const bf16* w1 = Wm + (size_t)r1 * K + t * 8;
         const int lim = K - 8 - t * 8;      // this lane's 8 channels of chunk c exist when 32 c <= lim
-        uint4 qa[kDmDepth], qb[kDmDepth];
+        uint4 qa[DEPTH], qb[DEPTH];
         auto fetch = [&](int c, int d) {
             const bool ok = live && c < c_hi && 32 * c <= lim;
             qa[d] = ok ? dm_ldg(reinterpret_cast<const uint4*>(w0 + 32 * c)) : make_uint4(0, 0, 0, 0);
             qb[d] = ok ? dm_ldg(reinterpret_cast<const uint4*>(w1 + 32 * c)) : make_uint4(0, 0, 0, 0);
         };
 #pragma unroll
-        for (int d = 0; d < kDmDepth; ++d) fetch(c_lo + d, d);
-        for (int rb = 0; rb < sl.cnt; rb += 8) {
-            const int nr = min(8, sl.cnt - rb);
-            if (it == 0 || sl.cnt > 8) {
-                if (plain && it == 0 && rb == 0) {
-                    pdl_wait();
-                    pdl_release();
+        for (int d = 0; d < DEPTH; ++d) fetch(c_lo + d, d);
+        if (it == 0) {
+            if (plain) {
+                pdl_wait();
+                pdl_release();
+            }
+            if (p.hn_o) {
+                // rows = per-head RMS norm of hn_o, times its weight, times the sigmoid of the gate; warp = (row, head)
+                const int V = K / p.hn_heads;
+                for (int i = w; i < 8 * p.hn_heads; i += kWarpsPerCta) {
+                    const int row = i / p.hn_heads, k0 = (i % p.hn_heads) * V;
+                    const int lo = max(k0, a_lo * 32), hi = min(k0 + V, a_hi * 32);
+                    if (lo >= hi) continue;
+                    if (row >= sl.cnt) {
+                        for (int k = lo + lane; k < hi; k += 32) xs[(size_t)row * XS + k - a_lo * 32] = from_f<bf16>(0.f);
+                        continue;
+                    }
+                    const float* o = p.hn_o + (size_t)row * K;
+                    float ss = 0.f;
+                    if (V % 4 == 0) {
+#pragma unroll 4
+                        for (int k = k0 + 4 * lane; k < k0 + V; k += 128) {
+                            const float4 v = *reinterpret_cast<const float4*>(o + k);
+                            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                        }
+                    } else {
+                        for (int k = k0 + lane; k < k0 + V; k += 32) ss += o[k] * o[k];
+                    }
+                    const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
+                    const bf16* gt = reinterpret_cast<const bf16*>(p.hn_g) + (size_t)row * p.hn_ldg;
+#pragma unroll 4
+                    for (int k = lo + lane; k < hi; k += 32)
+                        xs[(size_t)row * XS + k - a_lo * 32] = from_f<bf16>(o[k] * inv * p.hn_w[k] * sigmoid_f(to_f(gt[k])));
                 }
-                __syncthreads();
-                for (int i = tid; i < 8 * (KP / 8); i += kThreads) {
-                    const int row = i / (KP / 8), c = i % (KP / 8);
+                for (int i = tid; i < 8 * 32; i += kThreads) {       // channels past K of the last chunk
+                    const int k = K + (i & 31);
+                    if (k < a_hi * 32) xs[(size_t)(i >> 5) * XS + k - a_lo * 32] = from_f<bf16>(0.f);
+                }
+            } else {
+                for (int i = tid; i < 8 * an * 4; i += kThreads) {
+                    const int row = i / (an * 4), c = i % (an * 4), k = a_lo * 32 + c * 8;
                     uint4 v = make_uint4(0, 0, 0, 0);
-                    if (row < nr && c * 8 < K) {
-                        const int e = sl.off + rb + row;
+                    if (row < sl.cnt && k < K) {
+                        const int e = sl.off + row;
                         const long long xr = p.entry_row ? p.entry_row[e] : e;
-                        v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.x) + xr * p.ldx + c * 8);
+                        v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(p.x) + xr * p.ldx + k);
                     }
                     *reinterpret_cast<uint4*>(xs + (size_t)row * XS + c * 8) = v;
                 }
-                __syncthreads();
             }
-            if (rb > 0) {
+            __syncthreads();
+        }
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)g * XS) + t;
+        for (int c0 = c_lo; c0 < c_hi; c0 += DEPTH) {
 #pragma unroll
-                for (int d = 0; d < kDmDepth; ++d) fetch(c_lo + d, d);
-            }
-            float acc[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)g * XS) + t;
-            for (int c0 = c_lo; c0 < c_hi; c0 += kDmDepth) {
-#pragma unroll
-                for (int d = 0; d < kDmDepth; ++d) {
-                    const int c = c0 + d;
-                    if (c < c_hi) {
-                        const uint4 a = qa[d], b = qb[d];
-                        fetch(c + kDmDepth, d);
-                        const uint4 xv = xb[c * 4];
-                        mma_bf16(acc, a.x, b.x, a.y, b.y, xv.x, xv.y);
-                        mma_bf16(acc, a.z, b.z, a.w, b.w, xv.z, xv.w);
-                    }
+            for (int d = 0; d < DEPTH; ++d) {
+                const int c = c0 + d;
+                if (c < c_hi) {
+                    const uint4 a = qa[d], b = qb[d];
+                    fetch(c + DEPTH, d);
+                    const uint4 xv = xb[(c - a_lo) * 4];
+                    mma_bf16(acc, a.x, b.x, a.y, b.y, xv.x, xv.y);
+                    mma_bf16(acc, a.z, b.z, a.w, b.w, xv.z, xv.w);
                 }
             }
-            if (s != 0) red[w * 32 + lane] = make_float4(acc[0], acc[1], acc[2], acc[3]);
-            __syncthreads();
-            if (s == 0 && live) {
-                for (int s2 = 1; s2 < SPLIT; ++s2) {
-                    const float4 v = red[(w + s2) * 32 + lane];
+        }
+        if (s != 0) red[w * 32 + lane] = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        __syncthreads();
+        if (s == 0) {
+            for (int s2 = 1; s2 < SPLIT; ++s2) {
+                const float4 v = red[(w + s2) * 32 + lane];
+                acc[0] += v.x;
+                acc[1] += v.y;
+                acc[2] += v.z;
+                acc[3] += v.w;
+            }
+        }
+        if (cs > 1) {                // SPLIT == 8, one tile per cluster
+            cluster_wait();
+            if (w == 0 && rank != 0) {
+                const uint32_t dst = cluster_addr(smem_u32(&s_part[rank][lane]), 0);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) st_cluster(dst + 4 * i, acc[i]);
+            }
+            cluster_arrive();
+            cluster_wait();
+            if (rank != 0) return;
+            if (w == 0)
+                for (int r = 1; r < cs; ++r) {
+                    const float4 v = s_part[r][lane];
                     acc[0] += v.x;
                     acc[1] += v.y;
                     acc[2] += v.z;
                     acc[3] += v.w;
                 }
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
-                    if (row < nr && n < p.N) dm_store<bf16>(p, sl.off + rb + row, n, p.alpha * act_dyn(p.act, acc[i]));
-                }
-            }
-            __syncthreads();
         }
+        if (s == 0 && live) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
+                if (row < sl.cnt && n < p.N) dm_store<bf16>(p, sl.off + row, n, p.alpha * act_dyn(p.act, acc[i]));
+            }
+        }
+        if (it + 1 < iters) __syncthreads();
     }
 }
 
@@ -222,7 +303,7 @@ __global__ void __launch_bounds__(256) dense_gather_kernel(const DmParams p, bf1
 // =====================================================================================================
 // tcgen05 kernel: 128 rows x TN features per tile
 // =====================================================================================================
-constexpr int kDtThreads = 192;        // warp 0: TMA, warp 1: MMA, warps 2..5: epilogue
+constexpr int kDtThreads = 320;        // warp 0: TMA, warp 1: MMA, warps 2..9: epilogue
 constexpr int kDtMaxSlots = 1024;
 
 template <int TN> struct DtCfg {
@@ -262,7 +343,7 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
         }
         for (int b = 0; b < 2; ++b) {
             mbar_init(afull + 8 * b, 1);
-            mbar_init(aempty + 8 * b, 4);
+            mbar_init(aempty + 8 * b, 8);
         }
         s_dead = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -376,7 +457,8 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
         }
         __syncwarp();
     } else {
-        const int q = warp & 3;      // tensor memory lanes 32 q .. 32 q + 31
+        const int q = warp & 3;              // tensor memory lanes 32 q .. 32 q + 31
+        const int half = (warp - 2) >> 2;    // left or right half of the tile's columns
         int buf = 0;
         uint32_t aph = 0;
         for (int tile = blockIdx.x; tile < total; tile += gridDim.x) {
@@ -390,7 +472,7 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
             const bool rin = r < sl.cnt;
             const size_t orow = (size_t)(sl.off + r);
 #pragma unroll 1
-            for (int c0 = 0; c0 < TN; c0 += 16) {
+            for (int c0 = half * (TN / 2); c0 < (half + 1) * (TN / 2); c0 += 16) {
                 const int n0 = ft * TN + c0;
                 if (n0 >= p.N) break;
                 uint32_t v[16];
@@ -490,7 +572,7 @@ extern "C" int glq_dense_debug_error(unsigned long long* out4, int clear) {
 static constexpr int kStreamRows = 8;
 
 extern "C" int glq_dense_matmul_path(const glq_dense_mm_t* a) {
-    if (a->dtype != GLQ_DT_BF16 || a->K % 8 || a->ldx % 8 || !al16(a->x) || !al16(a->W)) return 0;
+    if (a->dtype != GLQ_DT_BF16 || a->K % 8 || (!a->hn_o && (a->ldx % 8 || !al16(a->x))) || !al16(a->W)) return 0;
     const int rows = a->slot_index ? a->max_slot_rows : a->rows;
     if (rows <= kStreamRows && a->K <= 12288) return 1;
     if ((a->slot_index && a->max_slots > kDtMaxSlots) || (a->entry_row && !a->gather) || !encode_tiled()) return 0;
@@ -502,7 +584,7 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     if (a->dtype != GLQ_DT_BF16 && a->dtype != GLQ_DT_F32) return GLQ_ERR_ARG;
     if (a->rows == 0) return GLQ_OK;
     const bool grouped = a->slot_index != nullptr;
-    if (!a->x || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
+    if ((!a->x && !a->hn_o) || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
     if (grouped && (!a->n_slots || !a->slot_count || !a->slot_offset || a->max_slots <= 0 || a->max_slot_rows <= 0 || a->n_matrices <= 0))
         return GLQ_ERR_ARG;
     if (!grouped && a->entry_row) return GLQ_ERR_ARG;
@@ -529,14 +611,27 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     p.vec_y = a->y && al16(a->y) && a->ldy % 8 == 0;
     p.vec_y32 = a->y32 && al16(a->y32) && a->ldy32 % 4 == 0 && a->split % 4 == 0;
     const int path = glq_dense_matmul_path(a);
+    if (a->hn_o) {
+        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !a->hn_g || !a->hn_w || !al16(a->hn_o)) return GLQ_ERR_ARG;
+        p.hn_o = a->hn_o;
+        p.hn_g = a->hn_g;
+        p.hn_w = a->hn_w;
+        p.hn_ldg = a->hn_ldg;
+        p.hn_heads = a->hn_heads;
+        p.hn_eps = a->hn_eps;
+    }
     const int rows_max = grouped ? a->max_slot_rows : a->rows;
     if (path == 1) {
-        const size_t smem = (size_t)8 * ((a->K + 31) / 32 * 32 + 32) * 2 + (size_t)kWarpsPerCta * 32 * sizeof(float4);
-        const int tiles = cdiv_i(a->N, 16), want = 2 * dn_sms();
-        // few tiles: all eight warps of a CTA share one
-        if ((long)tiles * p.slots <= want * 2)
-            return dn_launch(dense_stream_kernel<8>, dim3(std::min(tiles, want), p.slots), kThreads, smem, stream, p);
-        return dn_launch(dense_stream_kernel<4>, dim3(std::min(cdiv_i(tiles, 2), want), p.slots), kThreads, smem, stream, p);
+        const int tiles = cdiv_i(a->N, 16), sms = dn_sms(), chunks = cdiv_i(a->K, 32);
+        p.cluster = 1;
+        const bool wide = (long)tiles * p.slots > 12L * sms;       // enough tiles: four warps each, CTAs walk over them
+        if (!wide)
+            while (p.cluster < kDmMaxCluster && (long)tiles * p.slots * p.cluster < 2L * sms && chunks >= 32 * p.cluster) p.cluster *= 2;
+        p.xs_max = (cdiv_i(chunks, p.cluster) + 1) * 32;
+        const size_t smem = (size_t)8 * p.xs_max * 2 + (size_t)kWarpsPerCta * 32 * sizeof(float4);
+        if (wide)
+            return dn_launch(dense_stream_kernel<4, 8, 2>, dim3(std::min(cdiv_i(tiles, 2), 2 * sms), p.slots), kThreads, smem, stream, p);
+        return dn_launch_cluster(dense_stream_kernel<8, GLQ_DM_DEPTH, GLQ_DM_CTAS>, dim3(tiles * p.cluster, p.slots), kThreads, smem, p.cluster, stream, p);
     }
     if (path == 2) {
         const void* xa = a->x;

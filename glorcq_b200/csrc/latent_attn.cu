@@ -1,6 +1,7 @@
 // Latent attention: keys and values of a position are projections of one latent vector (plus a rotated key part that
 // all heads share), and the cache holds only the latent and that part.
-//   * prep: norm of the new latents, rotation of the shared key part and of every head's rotated query part, cache write;
+//   * the norm of the new latents, the rotation of the shared key part and of every head's rotated query part, and the
+//     cache write are a launch of their own before the prompt form and part of the absorbed form's first launch;
 //   * absorbed form (decode steps, short portions): the query is taken through the key projection once
 //     (q' = W_uk^T q), scores and the weighted sum run over the cached latents of all heads at once on the tensor
 //     cores, and the value projection follows for the sum; positions are split over CTAs;
@@ -43,6 +44,27 @@ template <typename T> __device__ __forceinline__ void rotate_part(T* x, const fl
     }
 }
 
+// one new position: its latent normed, its key part turned, both into the cache
+template <typename T>
+__device__ __forceinline__ void cache_row(const LaParams& p, size_t row, long long pos, float* red) {
+    const int b = (int)(row / p.T), half = p.rot_dims / 2;
+    const float* c = p.ckr + row * p.ldk;
+    const float* kr = c + p.K;
+    T* dst = reinterpret_cast<T*>(p.cache) + ((size_t)b * p.max_len + pos) * p.ldc;
+    const float* cs = p.cos_t + (size_t)pos * half;
+    const float* sn = p.sin_t + (size_t)pos * half;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < p.K; i += blockDim.x) ss += c[i] * c[i];
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / p.K + p.eps);
+    for (int i = threadIdx.x; i < p.K; i += blockDim.x) dst[i] = from_f<T>(c[i] * inv * p.norm_w[i]);
+    for (int i = threadIdx.x; i < p.R; i += blockDim.x) {
+        float v = kr[i];
+        if (i < half) v = kr[i] * cs[i] - kr[i + half] * sn[i];
+        else if (i < 2 * half) v = kr[i] * cs[i - half] + kr[i - half] * sn[i - half];
+        dst[p.K + i] = from_f<T>(v);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(const LaParams p) {
     __shared__ float red[32];
@@ -50,27 +72,13 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LaParams p) {
     pdl_release();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const size_t row = blockIdx.x;
-    const int b = (int)(row / p.T), t = (int)(row % p.T);
-    const long long pos = *p.start + t;
+    const long long pos = *p.start + (long long)(row % p.T);
     if (pos < 0 || pos >= p.max_len) return;
-    const float* c = p.ckr + row * p.ldk;
-    T* dst = reinterpret_cast<T*>(p.cache) + ((size_t)b * p.max_len + pos) * p.ldc;
+    cache_row<T>(p, row, pos, red);
     const int half = p.rot_dims / 2;
-    const float* cs = p.cos_t + (size_t)pos * half;
-    const float* sn = p.sin_t + (size_t)pos * half;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < p.K; i += 128) ss += c[i] * c[i];
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / p.K + p.eps);
-    for (int i = threadIdx.x; i < p.K; i += 128) dst[i] = from_f<T>(c[i] * inv * p.norm_w[i]);
-    for (int i = threadIdx.x; i < p.R; i += 128) {
-        const float* kr = c + p.K;
-        float v = kr[i];
-        if (i < half) v = kr[i] * cs[i] - kr[i + half] * sn[i];
-        else if (i < 2 * half) v = kr[i] * cs[i - half] + kr[i - half] * sn[i - half];
-        dst[p.K + i] = from_f<T>(v);
-    }
     for (int h = warp; h < p.H; h += 4)
-        rotate_part(reinterpret_cast<T*>(p.q) + row * p.ldq + (size_t)h * (p.D + p.R) + p.D, cs, sn, half, lane);
+        rotate_part(reinterpret_cast<T*>(p.q) + row * p.ldq + (size_t)h * (p.D + p.R) + p.D, p.cos_t + (size_t)pos * half,
+                    p.sin_t + (size_t)pos * half, half, lane);
 }
 
 // 8 consecutive values from global memory
@@ -126,14 +134,24 @@ __device__ __forceinline__ void head_products(const T* __restrict__ W, int n_lo,
     }
 }
 
-// q' of a head: (K, D) times the unrotated query, then the rotated query, all times scale * log2(e)
+// q' of a head: (K, D) times the unrotated query, then the rotated query, all times scale * log2(e); the blocks behind
+// the last head write the cache rows of the new positions
 template <typename T, bool SPLIT>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const LaParams p) {
     extern __shared__ float xs[];
+    __shared__ float red[32];
     const int Dp = (p.D + 7) / 8 * 8;
     pdl_wait();
     pdl_release();
-    const int h = blockIdx.x, rows = p.B * p.T;
+    const int h = blockIdx.x, rows = p.B * p.T, half = p.rot_dims / 2;
+    const long long start = *p.start;
+    if (h == p.H) {
+        for (int row = blockIdx.z * gridDim.y + blockIdx.y; row < rows; row += gridDim.y * gridDim.z) {
+            const long long pos = start + row % p.T;
+            if (pos >= 0 && pos < p.max_len) cache_row<T>(p, row, pos, red);
+        }
+        return;
+    }
     const int per = (p.K + gridDim.y - 1) / gridDim.y, n_lo = blockIdx.y * per, n_hi = min(p.K, n_lo + per);
     const float sc = p.scale * 1.4426950408889634f;
     const int ld = SPLIT ? p.KRp : p.K + p.R;
@@ -163,8 +181,14 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LaParams p) {
             for (int i = threadIdx.x; i < nr * tail; i += 256) {
                 const int r = i / tail, j = i % tail;
                 float v = 0.f;
-                if (j < p.R) v = to_f(reinterpret_cast<const T*>(p.q)[(size_t)(r0 + r) * p.ldq + (size_t)h * (p.D + p.R) + p.D + j]) * sc;
-                put(r0 + r, p.K + j, v);
+                if (j < p.R) {
+                    const T* q = reinterpret_cast<const T*>(p.q) + (size_t)(r0 + r) * p.ldq + (size_t)h * (p.D + p.R) + p.D;
+                    const long long pos = min((long long)p.max_len - 1, max(0LL, start + (r0 + r) % p.T));
+                    v = to_f(q[j]);
+                    if (j < half) v = v * p.cos_t[pos * half + j] - to_f(q[j + half]) * p.sin_t[pos * half + j];
+                    else if (j < 2 * half) v = v * p.cos_t[pos * half + j - half] + to_f(q[j - half]) * p.sin_t[pos * half + j - half];
+                }
+                put(r0 + r, p.K + j, v * sc);
             }
         }
     }
@@ -187,24 +211,39 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LaParams p) {
             const int row = r0 + r, rr = (row % p.T) * p.H + h;
             return (((size_t)(row / p.T) * tiles + rr / 16) * p.splits + z) * 16 + rr % 16;
         };
-        if (threadIdx.x < nr) {
-            const int r = threadIdx.x;
-            float m = -INFINITY, l = 0.f;
-            for (int z = 0; z < p.splits; ++z) m = fmaxf(m, p.pm[part(r, z)]);
-            for (int z = 0; z < p.splits; ++z) {
-                const float w = exp2f(p.pm[part(r, z)] - m);
-                sw[r][z] = w;
-                l += w * p.pl[part(r, z)];
+        {
+            const int r = threadIdx.x >> 5, lane = threadIdx.x & 31;       // warp = row, lane = splits lane, lane + 32
+            if (r < nr) {
+                float mz[2], lz[2];
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    const int z = lane + 32 * u;
+                    mz[u] = z < p.splits ? p.pm[part(r, z)] : -INFINITY;
+                    lz[u] = z < p.splits ? p.pl[part(r, z)] : 0.f;
+                }
+                float m = fmaxf(mz[0], mz[1]);
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+                const float w0 = exp2f(mz[0] - m), w1 = exp2f(mz[1] - m);
+                const float inv = 1.f / warp_sum(w0 * lz[0] + w1 * lz[1]);
+                sw[r][lane] = w0 * inv;
+                sw[r][lane + 32] = w1 * inv;
             }
-            for (int z = 0; z < p.splits; ++z) sw[r][z] /= l;
         }
         __syncthreads();
         for (int i = threadIdx.x; i < nr * Kp; i += 256) {
             const int r = i / Kp, k = i % Kp;
             float v = 0.f;
-            if (k < p.K)
-                for (int z = 0; z < p.splits; ++z)
-                    if (sw[r][z] != 0.f) v += sw[r][z] * p.po[part(r, z) * p.K + k];
+            if (k < p.K) {
+                const float* po = p.po + part(r, 0) * p.K + k;
+                const size_t step = (size_t)16 * p.K;
+#pragma unroll 8
+                for (int z = 0; z < p.splits; ++z) {
+                    // a split without a visible position left its sums unwritten
+                    const float w = sw[r][z], x = w != 0.f ? po[z * step] : 0.f;
+                    v += w * x;
+                }
+            }
             xs[i] = v;
         }
         __syncthreads();
@@ -222,7 +261,7 @@ constexpr int kAbPos = 32;       // positions per stage
 
 // 16 rows (query position, head) against one split of the positions; NT: 8-column tiles of the latent per warp
 template <int NT>
-__global__ void __launch_bounds__(128) latent_absorbed_kernel(const LaParams p) {
+__global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) {
     extern __shared__ __align__(16) unsigned char la_raw[];
     const int KRp = p.KRp, LD = KRp + 8;
     bf16* qh = reinterpret_cast<bf16*>(la_raw);              // [16][LD]
@@ -230,7 +269,7 @@ __global__ void __launch_bounds__(128) latent_absorbed_kernel(const LaParams p) 
     bf16* cs = ql + 16 * LD;                                 // [2][kAbPos][LD]
     bf16* ph = cs + 2 * kAbPos * LD;                         // [16][kAbPos + 8]
     bf16* pl = ph + 16 * (kAbPos + 8);
-    __shared__ float sc[16][kAbPos + 1], s_m[16], s_l[16], s_f[16];
+    __shared__ float sc[2][16][kAbPos + 1], s_m[16], s_l[16], s_f[16];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     const int rt = blockIdx.x, z = blockIdx.y, b = blockIdx.z, tiles = gridDim.x;
     const int KR = p.K + p.R;
@@ -243,7 +282,7 @@ __global__ void __launch_bounds__(128) latent_absorbed_kernel(const LaParams p) 
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.max_len * p.ldc;
     auto load = [&](int c, int buf) {
         const int vec = KRp / 8;
-        for (int i = tid; i < kAbPos * vec; i += 128) {
+        for (int i = tid; i < kAbPos * vec; i += 256) {
             const int r = i / vec, cc = (i % vec) * 8, pos = c * kAbPos + r;
             const bool live = pos < total && cc < KR;
             cpa16(smem_u32(cs + ((size_t)buf * kAbPos + r) * LD + cc), live ? cache + (size_t)pos * p.ldc + cc : cache, live);
@@ -255,7 +294,7 @@ __global__ void __launch_bounds__(128) latent_absorbed_kernel(const LaParams p) 
         const bf16* src = reinterpret_cast<const bf16*>(p.qa) + ((size_t)b * p.rows16 + rt * 16) * KRp;
         const size_t plane = (size_t)p.B * p.rows16 * KRp;
         const int vec = KRp / 8;
-        for (int i = tid; i < 16 * vec; i += 128) {
+        for (int i = tid; i < 16 * vec; i += 256) {
             const int r = i / vec, cc = (i % vec) * 8;
             const bool live = rt * 16 + r < p.T * p.H;
             const uint4 zero = make_uint4(0, 0, 0, 0);
@@ -282,30 +321,36 @@ __global__ void __launch_bounds__(128) latent_absorbed_kernel(const LaParams p) 
         }
         __syncthreads();
         const bf16* ct = cs + (size_t)buf * kAbPos * LD;
-        // scores: warp = 8 positions
-        float s[4] = {0.f, 0.f, 0.f, 0.f};
-        for (int k0 = 0; k0 < KRp; k0 += 32) {
+        // scores: warp = 8 positions, half of the columns (every second step of 32)
+        float s[4][4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[u][e] = 0.f;
+        const int wp = warp & 3, wk = warp >> 2;
+        for (int k0 = 32 * wk; k0 < KRp; k0 += 64) {
             uint32_t b0, b1, b2, b3;
-            ldsm4(smem_u32(ct + (8 * warp + (lane & 7)) * LD + k0 + (lane >> 3) * 8), b0, b1, b2, b3);
+            ldsm4(smem_u32(ct + (8 * wp + (lane & 7)) * LD + k0 + (lane >> 3) * 8), b0, b1, b2, b3);
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
                 const int off = ((lane & 7) + ((lane >> 3) & 1) * 8) * LD + k0 + 16 * u + (lane >> 4) * 8;
                 uint32_t a0, a1, a2, a3;
                 ldsm4(smem_u32(qh + off), a0, a1, a2, a3);
-                mma_bf16(s, a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
+                mma_bf16(s[2 * u], a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
                 ldsm4(smem_u32(ql + off), a0, a1, a2, a3);
-                mma_bf16(s, a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
+                mma_bf16(s[2 * u + 1], a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
             }
         }
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[g + 8 * (e >> 1)][8 * warp + 2 * t4 + (e & 1)] = s[e];
+        for (int e = 0; e < 4; ++e)
+            sc[wk][g + 8 * (e >> 1)][8 * wp + 2 * t4 + (e & 1)] = (s[0][e] + s[2][e]) + (s[1][e] + s[3][e]);
         __syncthreads();
-        // softmax: warp = 4 rows, lane = position
+        // softmax: warp = 2 rows, lane = position
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int r = 4 * warp + i, row = rt * 16 + r, pos = c * kAbPos + lane;
+        for (int i = 0; i < 2; ++i) {
+            const int r = 2 * warp + i, row = rt * 16 + r, pos = c * kAbPos + lane;
             const bool seen = row < p.T * p.H && pos < total && pos <= start + row / p.H;
-            const float v = seen ? sc[r][lane] : -INFINITY;
+            const float v = seen ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY;
             float mx = v;
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -430,6 +475,13 @@ template <int DK, int DV> struct LpCfg {
     static constexpr size_t SMEM = (size_t)2 * STAGE * 2;
 };
 
+// 2^x by the special-function unit alone (2 ulp; -inf -> 0; results below the normal range flush to zero)
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 template <int DK, int DV>
 __global__ void __launch_bounds__(128) latent_prefill_kernel(const LaParams p) {
     using C = LpCfg<DK, DV>;
@@ -537,16 +589,16 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LaParams p) {
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
         const float n0 = fmaxf(m0, mx0), n1 = fmaxf(m1, mx1);
         const float f0 = n0 == -INFINITY ? 0.f : n0, f1 = n1 == -INFINITY ? 0.f : n1;
-        const float a0 = exp2f(m0 - f0), a1 = exp2f(m1 - f1);
+        const float a0 = ex2(m0 - f0), a1 = ex2(m1 - f1);
         m0 = n0;
         m1 = n1;
         float s0 = 0.f, s1 = 0.f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            s[j][0] = exp2f(s[j][0] - f0);
-            s[j][1] = exp2f(s[j][1] - f0);
-            s[j][2] = exp2f(s[j][2] - f1);
-            s[j][3] = exp2f(s[j][3] - f1);
+            s[j][0] = ex2(s[j][0] - f0);
+            s[j][1] = ex2(s[j][1] - f0);
+            s[j][2] = ex2(s[j][2] - f1);
+            s[j][3] = ex2(s[j][3] - f1);
             s0 += s[j][0] + s[j][1];
             s1 += s[j][2] + s[j][3];
         }
@@ -696,34 +748,36 @@ template <typename T> static int la_absorbed(const glq_latent_t* a, void* stream
     const bool tensor = la_tensor(a);
     const int rb = std::min(cdiv_i((long)a->B * a->T, kHmRows), 512);
     // output rows of a head are split over CTAs until the machine is covered
-    auto parts = [&](int n, int lanes_k) {
+    auto parts = [&](int n, int lanes_k, long want) {
         int gl = 1;
         while (gl < 32 && gl * 8 < lanes_k) gl <<= 1;
         const int step = 8 * (32 / gl);                      // output rows a CTA takes at a time
-        return std::max(1, std::min(cdiv_i(n, step), cdiv_i(2L * dn_sms(), (long)a->H * rb)));
+        return std::max(1, std::min(cdiv_i(n, step), cdiv_i(want, (long)a->H * rb)));
     };
     const size_t xa = (size_t)kHmRows * ((a->D + 7) / 8 * 8) * 4, xv = (size_t)kHmRows * ((a->K + 7) / 8 * 8) * 4;
     int st;
     if (tensor) {
-        st = dn_launch(latent_absorb_kernel<T, true>, dim3(a->H, parts(a->K, a->D), rb), 256, xa, stream, p);
+        st = dn_launch(latent_absorb_kernel<T, true>, dim3(a->H + 1, parts(a->K, a->D, 2L * dn_sms()), rb), 256, xa, stream, p);
         if (st != GLQ_OK) return st;
         const dim3 grid(p.rows16 / 16, p.splits, a->B);
         const size_t smem = la_absorbed_smem(p);
-        if (a->K <= 128) st = dn_launch(latent_absorbed_kernel<4>, grid, 128, smem, stream, p);
-        else if (a->K <= 256) st = dn_launch(latent_absorbed_kernel<8>, grid, 128, smem, stream, p);
-        else st = dn_launch(latent_absorbed_kernel<16>, grid, 128, smem, stream, p);
+        if (a->K <= 128) st = dn_launch(latent_absorbed_kernel<2>, grid, 256, smem, stream, p);
+        else if (a->K <= 256) st = dn_launch(latent_absorbed_kernel<4>, grid, 256, smem, stream, p);
+        else st = dn_launch(latent_absorbed_kernel<8>, grid, 256, smem, stream, p);
     } else {
-        st = dn_launch(latent_absorb_kernel<T, false>, dim3(a->H, parts(a->K, a->D), rb), 256, xa, stream, p);
+        st = dn_launch(latent_absorb_kernel<T, false>, dim3(a->H + 1, parts(a->K, a->D, 2L * dn_sms()), rb), 256, xa, stream, p);
         if (st != GLQ_OK) return st;
         const size_t smem = (size_t)(2 * a->K + a->R + 128) * 4;
         st = dn_launch(latent_absorbed_generic_kernel<T>, dim3(a->T * a->H, a->B), 128, smem, stream, p);
     }
     if (st != GLQ_OK) return st;
-    return dn_launch(latent_value_kernel<T>, dim3(a->H, parts(a->V, a->K), rb), 256, xv, stream, p);
+    return dn_launch(latent_value_kernel<T>, dim3(a->H, parts(a->V, a->K, dn_sms() / 2), rb), 256, xv, stream, p);
 }
 
 extern "C" int glq_latent_absorbed(const glq_latent_t* a, void* stream) {
-    if (!la_sizes_ok(a) || !a->q || !a->cache || !a->start || !a->ukt || !a->uv || !a->gate || !a->out || !a->workspace) return GLQ_ERR_ARG;
+    if (!la_sizes_ok(a) || !a->q || !a->ckr || !a->norm_w || !a->cache || !a->start || (a->rot_dims && (!a->cos_t || !a->sin_t)) || !a->ukt || !a->uv || !a->gate ||
+        !a->out || !a->workspace)
+        return GLQ_ERR_ARG;
     if (!al16(a->workspace) || !al16(a->ukt) || !al16(a->uv)) return GLQ_ERR_ALIGN;
     if (a->K > 4096 || a->D > 4096 || a->R > 4096 || a->B > 65535) return GLQ_ERR_UNSUPPORTED;
     if (a->T == 0) return GLQ_OK;

@@ -3,8 +3,9 @@
 //     m' = max(f + m, i);  S' = e^(f+m-m') S + e^(i-m') k v^T;  n' = e^(f+m-m') n + e^(i-m') k
 //     o = S'^T q / (max(|n'.q|, e^-m') + 1e-6)
 // Two forms of the same recurrence:
-//   * step: the recurrence itself, one position after the other.  A CTA owns 32 value columns of a head; the CTA of a
-//     head that arrives last applies the per-head norm and the output gate, so a decode step is one launch.
+//   * step: the recurrence itself, one position after the other; a CTA owns 32 value columns of a head.  The per-head
+//     norm and output gate that follow go into the staging of the output product of a decode step (dense_mm.cu), or are
+//     a launch of their own.
 //   * chunk: 64 positions at a time on the tensor cores.  With b the running sum of f inside a chunk, a_s = i_s - b_s
 //     and r_t = b_t - m_t, position s reaches position t of its chunk with weight e^(r_t + a_s) and the state at the
 //     chunk's start with e^(r_t + m_start); m_t = b_t + max(m_start, max_{s<=t} a_s) is the recurrence's own maximum.
@@ -29,15 +30,14 @@ struct MlParams {
     float* m;
     void* out;
     float* o;                      // (B * Tall, H * V)
-    int* counters;
     long long ldp, ldg;
     int B, T, H, D, V, slices;
     int state_idle;
     int t0, Tall;                  // this call's positions: t0 .. t0 + T - 1 of the Tall rows of a sequence
     float cap, eps, scale;
     // chunk form
-    float *r, *a, *mt, *min_, *nbuf;
-    bf16 *Shi, *Slo;
+    float *bs, *as, *cm, *tot, *m0, *min_, *nbuf;
+    uint32_t* Sb;
     int nc, Dp, Vp;
 };
 
@@ -56,12 +56,33 @@ __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, in
     const T* g = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)p.H * (2 * p.D + p.V) + (size_t)h * p.V;
     T* out = reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V;
     float ss = 0.f;
+    if (p.V % 4 == 0 && p.V <= 1024) {          // four values per lane and step, kept in registers
+        float4 x[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int v = (u * 32 + lane) * 4;
+            x[u] = v < p.V ? *reinterpret_cast<const float4*>(o + v) : make_float4(0, 0, 0, 0);
+            ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / p.V + p.eps);
+        const float* w = p.norm_w + (size_t)h * p.V;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const int v = (u * 32 + lane) * 4;
+            if (v < p.V) {
+                const float y[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) out[v + i] = from_f<T>(y[i] * inv * w[v + i] * sigmoid_f(to_f(g[v + i])));
+            }
+        }
+        return;
+    }
     for (int v = lane; v < p.V; v += 32) {
-        const float x = __ldcg(o + v);
+        const float x = o[v];
         ss += x * x;
     }
     const float inv = 1.f / sqrtf(warp_sum(ss) / p.V + p.eps);
-    for (int v = lane; v < p.V; v += 32) out[v] = from_f<T>(__ldcg(o + v) * inv * p.norm_w[h * p.V + v] * sigmoid_f(to_f(g[v])));
+    for (int v = lane; v < p.V; v += 32) out[v] = from_f<T>(o[v] * inv * p.norm_w[h * p.V + v] * sigmoid_f(to_f(g[v])));
 }
 
 template <typename T>
@@ -70,7 +91,6 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const MlParams p) {
     float* sq = ml_smem;                 // [D]
     float* sk = sq + p.D;                // [D]
     __shared__ float sv[kSl], part[8][kSl], dpart[8];
-    __shared__ int s_last;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int sl = blockIdx.x, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
     const int D = p.D, V = p.V, v0 = sl * kSl, vw = min(kSl, V - v0);
@@ -159,98 +179,72 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const MlParams p) {
                 num += part[w][tid];
                 dd += dpart[w];
             }
-            __stcg(p.o + row * p.H * V + (size_t)h * V + v0 + tid, num / (fmaxf(fabsf(dd), expf(-m)) + 1e-6f));
+            p.o[row * p.H * V + (size_t)h * V + v0 + tid] = num / (fmaxf(fabsf(dd), expf(-m)) + 1e-6f);
         }
     }
     if (tid == 0) *mp = m;
-    __threadfence();
-    __syncthreads();
-    if (tid == 0) {
-        const int old = atomicAdd(p.counters + bh, 1);
-        s_last = old == p.slices - 1;
-        if (s_last) p.counters[bh] = 0;
-    }
-    __syncthreads();
-    if (!s_last) return;
-    __threadfence();
-    for (int t = warp; t < p.T; t += 8) head_norm_gate<T>(p, (size_t)b * p.Tall + p.t0 + t, h, lane);
 }
 
 // ---- chunk form ------------------------------------------------------------------------------------------
-// gates of a head for all chunks: r, a, m of every position (positions past T weigh nothing), m at every chunk's start
-__global__ void __launch_bounds__(256) mlstm_gate_kernel(const MlParams p) {
-    extern __shared__ float ml_smem[];
-    float* ctot = ml_smem;               // [nc] sum of f
-    float* cmax = ctot + p.nc;           // [nc] max of a
-    float* cm = cmax + p.nc;             // [nc] m at the chunk's start
+// gates of the chunks, one warp each: running sum of f (bs), i - bs (as) and its running maximum (cm) for every position,
+// sum and maximum of the chunk (tot); positions past T weigh nothing
+__global__ void __launch_bounds__(128) mlstm_gate_kernel(const MlParams p) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int h = blockIdx.x % p.H, b = blockIdx.x / p.H;
-    const size_t bh = blockIdx.x, base = bh * (size_t)p.nc * kL;
+    const int c = blockIdx.x * 4 + warp, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
+    const size_t bh = blockIdx.y;
     pdl_wait();
     pdl_release();
-    for (int c = warp; c < p.nc; c += 8) {
-        float f[2], li[2];
+    if (c >= p.nc) return;
+    // the maximum the sequence starts from, before the state kernel replaces it
+    if (c == 0 && lane == 0) p.m0[bh] = p.m[bh * p.slices];
+    float f[2], li[2];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int t = c * kL + 2 * lane + e;
-            const size_t row = (size_t)b * p.Tall + p.t0 + t;
-            f[e] = t < p.T ? log_f(p, row, h) : 0.f;
-            li[e] = t < p.T ? log_i(p, row, h) : -INFINITY;
-        }
-        float sum = f[0] + f[1];
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const float u = __shfl_up_sync(0xffffffffu, sum, o);
-            if (lane >= o) sum += u;
-        }
-        const float b1 = sum, b0 = sum - f[1];
-        const float a0 = li[0] - b0, a1 = li[1] - b1;
-        float mx = fmaxf(a0, a1);
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const float u = __shfl_up_sync(0xffffffffu, mx, o);
-            if (lane >= o) mx = fmaxf(mx, u);
-        }
-        const float prev = __shfl_up_sync(0xffffffffu, mx, 1);
-        const size_t i = base + c * kL + 2 * lane;
-        p.a[i] = a0;
-        p.a[i + 1] = a1;
-        p.r[i] = b0;                     // b and the running maximum for now
-        p.r[i + 1] = b1;
-        p.mt[i] = lane ? fmaxf(prev, a0) : a0;
-        p.mt[i + 1] = mx;
-        if (lane == 31) {
-            ctot[c] = b1;
-            cmax[c] = mx;
-        }
+    for (int e = 0; e < 2; ++e) {
+        const int t = c * kL + 2 * lane + e;
+        const size_t row = (size_t)b * p.Tall + p.t0 + t;
+        f[e] = t < p.T ? log_f(p, row, h) : 0.f;
+        li[e] = t < p.T ? log_i(p, row, h) : -INFINITY;
     }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        float m = p.m[bh * p.slices];
-        for (int c = 0; c < p.nc; ++c) {
-            cm[c] = m;
-            p.min_[bh * p.nc + c] = m;
-            m = ctot[c] + fmaxf(m, cmax[c]);
-        }
-        for (int s = 0; s < p.slices; ++s) p.m[bh * p.slices + s] = m;
-    }
-    __syncthreads();
-    for (int c = warp; c < p.nc; c += 8) {
+    float sum = f[0] + f[1];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const size_t i = base + c * kL + 2 * lane + e;
-            const float bb = p.r[i], mm = bb + fmaxf(cm[c], p.mt[i]);
-            p.mt[i] = mm;
-            p.r[i] = bb - mm;
-        }
+    for (int o = 1; o < 32; o <<= 1) {
+        const float u = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += u;
     }
+    const float b1 = sum, b0 = sum - f[1];
+    const float a0 = li[0] - b0, a1 = li[1] - b1;
+    float mx = fmaxf(a0, a1);
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float u = __shfl_up_sync(0xffffffffu, mx, o);
+        if (lane >= o) mx = fmaxf(mx, u);
+    }
+    const float prev = __shfl_up_sync(0xffffffffu, mx, 1);
+    const size_t i = (bh * p.nc + c) * kL + 2 * lane;
+    *reinterpret_cast<float2*>(p.bs + i) = make_float2(b0, b1);
+    *reinterpret_cast<float2*>(p.as + i) = make_float2(a0, a1);
+    *reinterpret_cast<float2*>(p.cm + i) = make_float2(lane ? fmaxf(prev, a0) : a0, mx);
+    if (lane == 31) *reinterpret_cast<float2*>(p.tot + (bh * p.nc + c) * 2) = make_float2(b1, mx);
 }
 
 constexpr int kTd = 64, kLd = 72;        // tile width, row stride of a 64-wide shared-memory tile (bf16)
+constexpr int kStStages = 4;
+constexpr int kStStage = 2 * kL * kLd * 2 + kL * 4;      // bytes: keys, values, i - bs
 
-// state at every chunk's start (as two bf16 planes, and n) and after the last chunk; one CTA owns 64 x 64 of a head's S
+// 8x8 block of 16-bit values held row-wise across a warp -> column-wise
+__device__ __forceinline__ uint32_t transpose8(uint32_t v) {
+    uint32_t r;
+    asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+    return r;
+}
+
+// Scratch layout of a chunk's starting state: blocks of 16 rows (d) x 8 columns (v) as the fragments the output kernel's
+// products take, [d / 16][v / 8][lane] of uint4 = (first part rows 0-7, rows 8-15, second part rows 0-7, rows 8-15).
+
+// state at every chunk's start (as sums of two bf16 parts, and n) and after the last chunk; one CTA owns 64 x 64 of a
+// head's S: warp = 16 rows
 __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
-    __shared__ __align__(16) bf16 ks[2][kL * kLd], vs[2][kL * kLd];
+    extern __shared__ __align__(16) unsigned char ml_raw[];
     __shared__ float ws[kL];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.z % p.H, b = blockIdx.z / p.H;
@@ -258,13 +252,19 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
     const size_t bh = blockIdx.z;
     const bf16* kb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)p.H * p.D + (size_t)h * p.D;
     const bf16* vb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)2 * p.H * p.D + (size_t)h * p.V;
-    auto load = [&](int c, int buf) {
-        for (int i = tid; i < kL * 8; i += 128) {
-            const int s = i >> 3, cc = (i & 7) * 8, tt = c * kL + s;
-            const size_t row = ((size_t)b * p.Tall + p.t0 + (tt < p.T ? tt : 0)) * p.ldp;
-            const bool kl = tt < p.T && d0 + cc < p.D, vl = tt < p.T && v0 + cc < p.V;
-            cpa16(smem_u32(&ks[buf][s * kLd + cc]), kl ? kb + row + d0 + cc : kb, kl);
-            cpa16(smem_u32(&vs[buf][s * kLd + cc]), vl ? vb + row + v0 + cc : vb, vl);
+    auto load = [&](int c) {
+        unsigned char* st = ml_raw + (size_t)(c % kStStages) * kStStage;
+        if (c < p.nc) {
+            bf16* ks = reinterpret_cast<bf16*>(st);
+            bf16* vs = ks + kL * kLd;
+            for (int i = tid; i < kL * 8; i += 128) {
+                const int s = i >> 3, cc = (i & 7) * 8, tt = c * kL + s;
+                const size_t row = ((size_t)b * p.Tall + p.t0 + (tt < p.T ? tt : 0)) * p.ldp;
+                const bool kl = tt < p.T && d0 + cc < p.D, vl = tt < p.T && v0 + cc < p.V;
+                cpa16(smem_u32(ks + s * kLd + cc), kl ? kb + row + d0 + cc : kb, kl);
+                cpa16(smem_u32(vs + s * kLd + cc), vl ? vb + row + v0 + cc : vb, vl);
+            }
+            if (tid < kL / 4) cpa16(smem_u32(vs + kL * kLd) + 16 * tid, p.as + (bh * p.nc + c) * kL + 4 * tid, true);
         }
         cpa_commit();
     };
@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
     float acc[8][4], nacc[2];
     pdl_wait();
     pdl_release();
-    load(0, 0);
+    for (int c = 0; c < kStStages - 1; ++c) load(c);
     const size_t slb = bh * p.slices;
 #pragma unroll
     for (int j = 0; j < 8; ++j)
@@ -283,40 +283,43 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
         }
 #pragma unroll
     for (int e = 0; e < 2; ++e) nacc[e] = dr[e] < p.D ? p.n[(slb + v0 / kSl) * p.D + dr[e]] : 0.f;
+    float m = p.m0[bh];
+    float2 tot = *reinterpret_cast<const float2*>(p.tot + bh * p.nc * 2);
     for (int c = 0; c < p.nc; ++c) {
         const size_t bc = bh * p.nc + c;
-        if (c + 1 < p.nc) {
-            load(c + 1, (c + 1) & 1);
-            cpa_wait<1>();
-        } else {
-            cpa_wait<0>();
-        }
-        const float rl = p.r[bc * kL + kL - 1];
-        if (tid < kL) ws[tid] = expf(rl + p.a[bc * kL + tid]);
+        const float2 tot_next = c + 1 < p.nc ? *reinterpret_cast<const float2*>(p.tot + (bc + 1) * 2) : tot;
+        cpa_wait<kStStages - 2>();
+        __syncthreads();                 // chunk c has landed; nobody still reads the stage that is loaded next
+        load(c + kStStages - 1);
+        const unsigned char* st = ml_raw + (size_t)(c % kStStages) * kStStage;
+        const bf16* kt = reinterpret_cast<const bf16*>(st);
+        const bf16* vt = kt + kL * kLd;
+        const float* ac = reinterpret_cast<const float*>(vt + kL * kLd);
+        // the chunk's end: b_L = tot.x, m_L = b_L + max(m, tot.y)
+        const float m_end = tot.x + fmaxf(m, tot.y), rl = tot.x - m_end, keep = expf(rl + m);
+        if (tid < kL) ws[tid] = expf(rl + ac[tid]);
+        if (blockIdx.x == 0 && blockIdx.y == 0 && tid == 0) p.min_[bc] = m;
+        m = m_end;
+        tot = tot_next;
         // the state this chunk starts from
+        uint4* sb = reinterpret_cast<uint4*>(p.Sb) + ((bc * (p.Dp / 16) + d0 / 16 + warp) * (p.Vp / 8) + v0 / 8) * 32 + lane;
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                uint32_t hi, lo;
-                split_bf2(acc[j][2 * e], acc[j][2 * e + 1], hi, lo);
-                const size_t o = (bc * p.Dp + dr[e]) * p.Vp + v0 + 8 * j + 2 * t;
-                *reinterpret_cast<uint32_t*>(p.Shi + o) = hi;
-                *reinterpret_cast<uint32_t*>(p.Slo + o) = lo;
-            }
+        for (int j = 0; j < 8; ++j) {
+            uint32_t h0, l0, h1, l1;
+            split_bf2(acc[j][0], acc[j][1], h0, l0);
+            split_bf2(acc[j][2], acc[j][3], h1, l1);
+            sb[j * 32] = make_uint4(transpose8(h0), transpose8(h1), transpose8(l0), transpose8(l1));
+        }
         if (blockIdx.y == 0 && t == 0) {
             p.nbuf[bc * p.Dp + dr[0]] = nacc[0];
             p.nbuf[bc * p.Dp + dr[1]] = nacc[1];
         }
         __syncthreads();
-        const float keep = expf(rl + p.min_[bc]);
 #pragma unroll
         for (int j = 0; j < 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[j][e] *= keep;
         float ns[2] = {0.f, 0.f};
-        const bf16* kt = ks[c & 1];
-        const bf16* vt = vs[c & 1];
 #pragma unroll
         for (int kk = 0; kk < 4; ++kk) {
             uint32_t a[4], hi[4], lo[4];
@@ -344,8 +347,8 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
             ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 2);
             nacc[e] = keep * nacc[e] + ns[e];
         }
-        __syncthreads();
     }
+    cpa_wait<0>();
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -353,24 +356,32 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
             const int v = v0 + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
             if (d < p.D && v < p.V) p.S[((slb + v / kSl) * p.D + d) * kSl + v % kSl] = acc[j][e];
         }
-    if (t == 0)
-        for (int s = v0 / kSl; s < min(p.slices, (v0 + kTd) / kSl); ++s)
+    for (int s = v0 / kSl; s < min(p.slices, (v0 + kTd) / kSl); ++s) {
+        if (t == 0)
 #pragma unroll
             for (int e = 0; e < 2; ++e)
                 if (dr[e] < p.D) p.n[(slb + s) * p.D + dr[e]] = nacc[e];
+        if (blockIdx.x == 0 && tid == 0) p.m[slb + s] = m;
+    }
 }
 
-// outputs of a chunk: 64 positions x VT value columns of a head
+// outputs of a chunk: 64 positions x VT value columns of a head; the rows of the state come in steps of 32, two buffered
+template <int VT> struct MoCfg {
+    static constexpr int LV = VT + 8, NV = VT / 8, LQ = 40;
+    static constexpr int QK = kL * LQ * 2;                   // bytes of 64 x 32 queries (or keys)
+    static constexpr int SB = 2 * NV * 32 * 16;              // bytes of 32 rows of state fragments
+    static constexpr int STAGE = 2 * QK + SB;
+    static constexpr size_t SMEM = (size_t)2 * STAGE + (size_t)kL * LV * 2;
+};
+
 template <int VT>
-__global__ void __launch_bounds__(128) mlstm_out_kernel(const MlParams p) {
-    constexpr int LV = VT + 8, NV = VT / 8;
+__global__ void __launch_bounds__(128, 3) mlstm_out_kernel(const MlParams p) {
+    using C = MoCfg<VT>;
+    constexpr int LV = C::LV, NV = C::NV, LQ = C::LQ;
     extern __shared__ __align__(16) unsigned char ml_raw[];
-    bf16* qs = reinterpret_cast<bf16*>(ml_raw);          // [64][72]
-    bf16* ks = qs + kL * kLd;                            // [64][72]
-    bf16* sh = ks + kL * kLd;                            // [64][LV]
-    bf16* slo = sh + kTd * LV;                           // [64][LV]
-    bf16* vs = slo + kTd * LV;                           // [64][LV]
-    __shared__ float sa[kL], sr[kL], sm[kL], sqn[kL], sn[kTd];
+    bf16* vs = reinterpret_cast<bf16*>(ml_raw + 2 * C::STAGE);      // [64][LV]
+    __shared__ float sa[kL], sr[kL], sm[kL], sqn[kL];
+    __shared__ __align__(16) float sn[2][32];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.z % p.H, b = blockIdx.z / p.H, c = blockIdx.y, v0 = blockIdx.x * VT;
     const size_t bc = (size_t)blockIdx.z * p.nc + c;
@@ -378,15 +389,40 @@ __global__ void __launch_bounds__(128) mlstm_out_kernel(const MlParams p) {
     pdl_wait();
     pdl_release();
     auto row_of = [&](int s) { return ((size_t)b * p.Tall + p.t0 + c * kL + s) * p.ldp; };
+    auto load = [&](int k, int buf) {
+        unsigned char* st = ml_raw + (size_t)buf * C::STAGE;
+        bf16* qs = reinterpret_cast<bf16*>(st);
+        bf16* ks = qs + kL * LQ;
+        const int d0 = 32 * k;
+        for (int i = tid; i < kL * 4; i += 128) {
+            const int s = i >> 2, cc = (i & 3) * 8;
+            const bool live = c * kL + s < p.T && d0 + cc < p.D;
+            const bf16* src = live ? base + row_of(s) + (size_t)h * p.D + d0 + cc : base;
+            cpa16(smem_u32(qs + s * LQ + cc), src, live);
+            cpa16(smem_u32(ks + s * LQ + cc), live ? src + (size_t)p.H * p.D : base, live);
+        }
+        const uint4* sb = reinterpret_cast<const uint4*>(p.Sb) + (bc * (p.Dp / 16) + d0 / 16) * (size_t)(p.Vp / 8) * 32;
+        const uint32_t dst = smem_u32(st + 2 * C::QK);
+        for (int i = tid; i < 2 * NV * 32; i += 128) {
+            const int r = i / (NV * 32), j = i % (NV * 32);
+            const bool live = v0 / 8 + j / 32 < p.Vp / 8;
+            cpa16(dst + 16 * i, live ? sb + (size_t)r * (p.Vp / 8) * 32 + (size_t)(v0 / 8) * 32 + j : sb, live);
+        }
+        if (tid < 8) cpa16(smem_u32(&sn[buf][4 * tid]), p.nbuf + bc * p.Dp + d0 + 4 * tid, true);
+        cpa_commit();
+    };
     for (int i = tid; i < kL * (VT / 8); i += 128) {
         const int s = i / (VT / 8), cc = (i % (VT / 8)) * 8;
         const bool live = c * kL + s < p.T && v0 + cc < p.V;
         cpa16(smem_u32(vs + s * LV + cc), live ? base + row_of(s) + (size_t)2 * p.H * p.D + (size_t)h * p.V + v0 + cc : base, live);
     }
+    load(0, 0);
+    const float m0 = p.min_[bc];
     if (tid < kL) {
-        sa[tid] = p.a[bc * kL + tid];
-        sr[tid] = p.r[bc * kL + tid];
-        sm[tid] = p.mt[bc * kL + tid];
+        const float bb = p.bs[bc * kL + tid], mm = bb + fmaxf(m0, p.cm[bc * kL + tid]);
+        sa[tid] = p.as[bc * kL + tid];
+        sr[tid] = bb - mm;
+        sm[tid] = mm;
     }
     float qk[8][4], acc[NV][4];
 #pragma unroll
@@ -398,65 +434,53 @@ __global__ void __launch_bounds__(128) mlstm_out_kernel(const MlParams p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
     float qn = 0.f;                                      // row tid / 2, half tid % 2 of q . n
-    for (int d0 = 0; d0 < p.Dp; d0 += kTd) {
-        __syncthreads();
-        for (int i = tid; i < kL * 8; i += 128) {
-            const int s = i >> 3, cc = (i & 7) * 8;
-            const bool live = c * kL + s < p.T && d0 + cc < p.D;
-            const bf16* src = live ? base + row_of(s) + (size_t)h * p.D + d0 + cc : base;
-            cpa16(smem_u32(qs + s * kLd + cc), src, live);
-            cpa16(smem_u32(ks + s * kLd + cc), live ? src + (size_t)p.H * p.D : base, live);
+    const int nk = p.Dp / 32;
+    for (int k = 0; k < nk; ++k) {
+        if (k + 1 < nk) {
+            load(k + 1, (k + 1) & 1);
+            cpa_wait<1>();
+        } else {
+            cpa_wait<0>();
         }
-        for (int i = tid; i < kTd * (VT / 8); i += 128) {
-            const int d = i / (VT / 8), cc = (i % (VT / 8)) * 8;
-            const bool live = v0 + cc < p.Vp;
-            const size_t o = (bc * p.Dp + d0 + d) * p.Vp + v0 + cc;
-            cpa16(smem_u32(sh + d * LV + cc), p.Shi + (live ? o : 0), live);
-            cpa16(smem_u32(slo + d * LV + cc), p.Slo + (live ? o : 0), live);
-        }
-        cpa_commit();
-        if (tid < kTd) sn[tid] = p.nbuf[bc * p.Dp + d0 + tid];
-        cpa_wait<0>();
         __syncthreads();
+        const unsigned char* st = ml_raw + (size_t)(k & 1) * C::STAGE;
+        const bf16* qs = reinterpret_cast<const bf16*>(st);
+        const bf16* ks = qs + kL * LQ;
+        const uint32_t sb = smem_u32(st + 2 * C::QK);
         {
-            const bf16* qr = qs + (tid >> 1) * kLd + (tid & 1) * 32;
-            const float* nr = sn + (tid & 1) * 32;
+            const bf16* qr = qs + (tid >> 1) * LQ + (tid & 1) * 16;
+            const float* nr = sn[k & 1] + (tid & 1) * 16;
 #pragma unroll
-            for (int i = 0; i < 32; i += 2) {
+            for (int i = 0; i < 16; i += 2) {
                 const uint32_t w = *reinterpret_cast<const uint32_t*>(qr + i);
                 qn += bf_lo(w) * nr[i] + bf_hi(w) * nr[i + 1];
             }
         }
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
+        for (int kk = 0; kk < 2; ++kk) {
             uint32_t a0, a1, a2, a3;
-            ldsm4(smem_u32(qs + (16 * warp + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 16 * kk + (lane >> 4) * 8), a0, a1, a2, a3);
+            ldsm4(smem_u32(qs + (16 * warp + (lane & 7) + ((lane >> 3) & 1) * 8) * LQ + 16 * kk + (lane >> 4) * 8), a0, a1, a2, a3);
 #pragma unroll
             for (int jp = 0; jp < 4; ++jp) {
                 if (jp > warp) continue;                 // keys after every query of this warp
                 uint32_t b0, b1, b2, b3;
-                ldsm4(smem_u32(ks + (16 * jp + (lane & 7) + (lane >> 4) * 8) * kLd + 16 * kk + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
+                ldsm4(smem_u32(ks + (16 * jp + (lane & 7) + (lane >> 4) * 8) * LQ + 16 * kk + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
                 mma_bf16(qk[2 * jp], a0, a1, a2, a3, b0, b1);
                 mma_bf16(qk[2 * jp + 1], a0, a1, a2, a3, b2, b3);
             }
-            const int srow = 16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8;
 #pragma unroll
-            for (int jp = 0; jp < NV / 2; ++jp) {
-                uint32_t b0, b1, b2, b3;
-                ldsm4_t(smem_u32(sh + srow * LV + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
-                mma_bf16(acc[2 * jp], a0, a1, a2, a3, b0, b1);
-                mma_bf16(acc[2 * jp + 1], a0, a1, a2, a3, b2, b3);
-                ldsm4_t(smem_u32(slo + srow * LV + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
-                mma_bf16(acc[2 * jp], a0, a1, a2, a3, b0, b1);
-                mma_bf16(acc[2 * jp + 1], a0, a1, a2, a3, b2, b3);
+            for (int j = 0; j < NV; ++j) {
+                const uint4 f = lds128(sb + (uint32_t)((kk * NV + j) * 32 + lane) * 16);
+                mma_bf16(acc[j], a0, a1, a2, a3, f.x, f.y);
+                mma_bf16(acc[j], a0, a1, a2, a3, f.z, f.w);
             }
         }
+        __syncthreads();
     }
     qn += __shfl_xor_sync(0xffffffffu, qn, 1);
     if ((tid & 1) == 0) sqn[tid >> 1] = qn;
     __syncthreads();
     const int tr[2] = {16 * warp + g, 16 * warp + g + 8};
-    const float m0 = p.min_[bc];
     float den[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
@@ -515,6 +539,7 @@ __global__ void __launch_bounds__(128) mlstm_out_kernel(const MlParams p) {
 }
 
 // one warp per (row, head)
+template <typename T>
 __global__ void __launch_bounds__(256) mlstm_norm_kernel(const MlParams p) {
     pdl_wait();
     pdl_release();
@@ -522,7 +547,7 @@ __global__ void __launch_bounds__(256) mlstm_norm_kernel(const MlParams p) {
     if (i >= (long long)p.B * p.T * p.H) return;
     const int h = (int)(i % p.H);
     const long long bt = i / p.H;
-    head_norm_gate<bf16>(p, (size_t)(bt / p.T) * p.Tall + p.t0 + bt % p.T, h, threadIdx.x & 31);
+    head_norm_gate<T>(p, (size_t)(bt / p.T) * p.Tall + p.t0 + bt % p.T, h, threadIdx.x & 31);
 }
 
 }  // namespace glq
@@ -535,9 +560,9 @@ static inline size_t up256d(size_t v) { return (v + 255) / 256 * 256; }
 static constexpr int kSegment = 4096;      // positions the chunk form takes at a time (bounds its workspace)
 
 struct MlWs {
-    size_t o, r, a, mt, min_, nbuf, hi, lo, total;
+    size_t bs, as, cm, tot, m0, min_, nbuf, sb, total;
 };
-static MlWs ml_ws(const glq_mlstm_t* a, bool chunked) {
+static MlWs ml_ws(const glq_mlstm_t* a) {
     MlWs w{};
     size_t at = 0;
     auto take = [&](size_t bytes) {
@@ -545,31 +570,26 @@ static MlWs ml_ws(const glq_mlstm_t* a, bool chunked) {
         at += up256d(bytes);
         return v;
     };
-    w.o = take((size_t)a->B * a->T * a->H * a->V * 4);
-    if (chunked) {
-        const size_t bh = (size_t)a->B * a->H, nc = cdiv_i(std::min(a->T, kSegment), kL), Dp = (a->D + 63) / 64 * 64, Vp = (a->V + 63) / 64 * 64;
-        w.r = take(bh * nc * kL * 4);
-        w.a = take(bh * nc * kL * 4);
-        w.mt = take(bh * nc * kL * 4);
-        w.min_ = take(bh * nc * 4);
-        w.nbuf = take(bh * nc * Dp * 4);
-        w.hi = take(bh * nc * Dp * Vp * 2);
-        w.lo = take(bh * nc * Dp * Vp * 2);
-    }
+    const size_t bh = (size_t)a->B * a->H, nc = cdiv_i(std::min(a->T, kSegment), kL), Dp = (a->D + 63) / 64 * 64, Vp = (a->V + 63) / 64 * 64;
+    w.bs = take(bh * nc * kL * 4);
+    w.as = take(bh * nc * kL * 4);
+    w.cm = take(bh * nc * kL * 4);
+    w.tot = take(bh * nc * 8);
+    w.m0 = take(bh * 4);
+    w.min_ = take(bh * nc * 4);
+    w.nbuf = take(bh * nc * Dp * 4);
+    w.sb = take(bh * nc * Dp * Vp * 4);
     w.total = at;
     return w;
 }
-extern "C" size_t glq_mlstm_workspace_bytes(const glq_mlstm_t* a, int chunked) { return ml_ws(a, chunked != 0).total; }
+extern "C" size_t glq_mlstm_workspace_bytes(const glq_mlstm_t* a) { return ml_ws(a).total; }
 
-static int ml_params(const glq_mlstm_t* a, MlParams& p, bool chunked) {
+static int ml_params(const glq_mlstm_t* a, MlParams& p) {
     if (!a || a->B <= 0 || a->T < 0 || a->H <= 0 || a->D <= 0 || a->V <= 0 || !(a->gate_cap > 0.f)) return GLQ_ERR_ARG;
-    if (!a->qkvg || !a->gates || !a->bias_i || !a->bias_f || !a->norm_w || !a->S || !a->n || !a->m || !a->out || !a->workspace || !a->counters)
-        return GLQ_ERR_ARG;
-    if (!al16(a->S) || !al16(a->workspace)) return GLQ_ERR_ALIGN;
-    const MlWs w = ml_ws(a, chunked);
-    if (a->workspace_bytes < w.total) return GLQ_ERR_WORKSPACE;
+    if (!a->qkvg || !a->gates || !a->bias_i || !a->bias_f || !a->norm_w || !a->S || !a->n || !a->m || !a->o) return GLQ_ERR_ARG;
+    if (a->dtype != GLQ_DT_BF16 && a->dtype != GLQ_DT_F32) return GLQ_ERR_ARG;
+    if (!al16(a->S) || !al16(a->o)) return GLQ_ERR_ALIGN;
     if (a->D > 8192 || (long)a->B * a->H > 65535) return GLQ_ERR_UNSUPPORTED;
-    char* ws = reinterpret_cast<char*>(a->workspace);
     p.qkvg = a->qkvg;
     p.gates = a->gates;
     p.bias_i = a->bias_i;
@@ -578,9 +598,8 @@ static int ml_params(const glq_mlstm_t* a, MlParams& p, bool chunked) {
     p.S = a->S;
     p.n = a->n;
     p.m = a->m;
+    p.o = a->o;
     p.out = a->out;
-    p.o = reinterpret_cast<float*>(ws + w.o);
-    p.counters = a->counters;
     p.ldp = a->ldp;
     p.ldg = a->ldg;
     p.B = a->B;
@@ -593,52 +612,58 @@ static int ml_params(const glq_mlstm_t* a, MlParams& p, bool chunked) {
     p.cap = a->gate_cap;
     p.eps = a->eps;
     p.scale = (float)(1.0 / sqrt((double)a->D));
-    if (chunked) {
-        p.r = reinterpret_cast<float*>(ws + w.r);
-        p.a = reinterpret_cast<float*>(ws + w.a);
-        p.mt = reinterpret_cast<float*>(ws + w.mt);
-        p.min_ = reinterpret_cast<float*>(ws + w.min_);
-        p.nbuf = reinterpret_cast<float*>(ws + w.nbuf);
-        p.Shi = reinterpret_cast<bf16*>(ws + w.hi);
-        p.Slo = reinterpret_cast<bf16*>(ws + w.lo);
-        p.Dp = (a->D + 63) / 64 * 64;
-        p.Vp = (a->V + 63) / 64 * 64;
-    }
     return GLQ_OK;
+}
+static int ml_norm(const MlParams& p, int dtype, void* stream) {
+    const dim3 grid(cdiv_i((long)p.B * p.T * p.H, 8));
+    if (dtype == GLQ_DT_BF16) return dn_launch(mlstm_norm_kernel<bf16>, grid, 256, 0, stream, p);
+    return dn_launch(mlstm_norm_kernel<float>, grid, 256, 0, stream, p);
 }
 
 extern "C" int glq_mlstm_step(const glq_mlstm_t* a, void* stream) {
     MlParams p{};
-    const int st = ml_params(a, p, false);
+    int st = ml_params(a, p);
     if (st != GLQ_OK) return st;
     if (p.T == 0) return GLQ_OK;
     const dim3 grid(p.slices, p.B * p.H);
     const size_t smem = (size_t)2 * p.D * 4;
-    if (a->dtype == GLQ_DT_BF16) return dn_launch(mlstm_step_kernel<bf16>, grid, 256, smem, stream, p);
-    if (a->dtype == GLQ_DT_F32) return dn_launch(mlstm_step_kernel<float>, grid, 256, smem, stream, p);
-    return GLQ_ERR_ARG;
+    if (a->dtype == GLQ_DT_BF16) st = dn_launch(mlstm_step_kernel<bf16>, grid, 256, smem, stream, p);
+    else st = dn_launch(mlstm_step_kernel<float>, grid, 256, smem, stream, p);
+    if (st != GLQ_OK || !p.out) return st;
+    return ml_norm(p, a->dtype, stream);
 }
 
 extern "C" int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream) {
     if (!a || a->dtype != GLQ_DT_BF16) return GLQ_ERR_ARG;
     if (a->D % 8 || a->V % 8 || a->ldp % 8) return GLQ_ERR_UNSUPPORTED;
     MlParams p{};
-    int st = ml_params(a, p, true);
+    int st = ml_params(a, p);
     if (st != GLQ_OK) return st;
-    if (!al16(a->qkvg)) return GLQ_ERR_ALIGN;
+    const MlWs w = ml_ws(a);
+    if (!a->out || !a->workspace) return GLQ_ERR_ARG;
+    if (a->workspace_bytes < w.total) return GLQ_ERR_WORKSPACE;
+    if (!al16(a->qkvg) || !al16(a->workspace)) return GLQ_ERR_ALIGN;
+    char* ws = reinterpret_cast<char*>(a->workspace);
+    p.bs = reinterpret_cast<float*>(ws + w.bs);
+    p.as = reinterpret_cast<float*>(ws + w.as);
+    p.cm = reinterpret_cast<float*>(ws + w.cm);
+    p.tot = reinterpret_cast<float*>(ws + w.tot);
+    p.m0 = reinterpret_cast<float*>(ws + w.m0);
+    p.min_ = reinterpret_cast<float*>(ws + w.min_);
+    p.nbuf = reinterpret_cast<float*>(ws + w.nbuf);
+    p.Sb = reinterpret_cast<uint32_t*>(ws + w.sb);
+    p.Dp = (a->D + 63) / 64 * 64;
+    p.Vp = (a->V + 63) / 64 * 64;
     const int bh = p.B * p.H;
     for (p.t0 = 0; p.t0 < p.Tall; p.t0 += kSegment) {
         p.T = std::min(kSegment, p.Tall - p.t0);
         p.nc = cdiv_i(p.T, kL);
-        if ((st = dn_launch(mlstm_gate_kernel, dim3(bh), 256, (size_t)3 * p.nc * 4, stream, p)) != GLQ_OK) return st;
-        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 128, 0, stream, p)) != GLQ_OK) return st;
-        constexpr size_t fixed = (size_t)2 * kL * kLd * 2;
-        if (p.V > 64)
-            st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, fixed + (size_t)3 * 64 * 136 * 2, stream, p);
-        else
-            st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, fixed + (size_t)3 * 64 * 72 * 2, stream, p);
+        if ((st = dn_launch(mlstm_gate_kernel, dim3(cdiv_i(p.nc, 4), bh), 128, 0, stream, p)) != GLQ_OK) return st;
+        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 128, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
+        if (p.V > 64) st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, MoCfg<128>::SMEM, stream, p);
+        else st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, MoCfg<64>::SMEM, stream, p);
         if (st != GLQ_OK) return st;
-        if ((st = dn_launch(mlstm_norm_kernel, dim3(cdiv_i((long)p.B * p.T * p.H, 8)), 256, 0, stream, p)) != GLQ_OK) return st;
+        if ((st = ml_norm(p, a->dtype, stream)) != GLQ_OK) return st;
     }
     return GLQ_OK;
 }

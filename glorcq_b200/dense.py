@@ -123,21 +123,42 @@ def route(logits, correction, experts, identity, top):
     return p
 
 
-def mlstm(qkvg, gates, B, T, heads, dim, vdim, cap, eps, bias_i, bias_f, norm_w, state, chunked, state_idle=False):
-    """Matrix-memory recurrence with per-head norm and output gate over T positions; ``state`` is advanced."""
+def mlstm(qkvg, gates, B, T, heads, dim, vdim, cap, eps, bias_i, bias_f, norm_w, state, chunked, state_idle=False, raw=False):
+    """Matrix-memory recurrence over T positions with per-head norm and output gate, or with ``raw`` (one-by-one form
+    only) its float output before them; ``state`` is advanced."""
     _need(qkvg, "qkvg")
     L, dev = _lib.dense(), qkvg.device
-    out = torch.empty(B * T, heads * vdim, dtype=qkvg.dtype, device=dev)
+    o = torch.empty(B * T, heads * vdim, dtype=torch.float32, device=dev)
+    out = None if raw and not chunked else torch.empty(B * T, heads * vdim, dtype=qkvg.dtype, device=dev)
     a = _lib.MLstm(dtype=DTYPES[qkvg.dtype], B=B, T=T, H=heads, D=dim, V=vdim, state_idle=int(state_idle), gate_cap=cap, eps=eps,
                    qkvg=qkvg.data_ptr(), ldp=qkvg.stride(0), gates=gates.data_ptr(), ldg=gates.stride(0), bias_i=bias_i.data_ptr(),
                    bias_f=bias_f.data_ptr(), norm_w=norm_w.data_ptr(), S=state.S.data_ptr(), n=state.n.data_ptr(),
-                   m=state.m.data_ptr(), out=out.data_ptr(), counters=state.counters.data_ptr())
-    ws = torch.empty(L.glq_mlstm_workspace_bytes(C.byref(a), int(chunked)), dtype=torch.uint8, device=dev)
-    a.workspace, a.workspace_bytes = ws.data_ptr(), ws.numel()
+                   m=state.m.data_ptr(), o=o.data_ptr(), out=None if out is None else out.data_ptr())
+    ws = None
+    if chunked:
+        ws = torch.empty(L.glq_mlstm_workspace_bytes(C.byref(a)), dtype=torch.uint8, device=dev)
+        a.workspace, a.workspace_bytes = ws.data_ptr(), ws.numel()
     with torch.cuda.device(dev):
         fn = L.glq_mlstm_chunk if chunked else L.glq_mlstm_step
         _lib.check_dense(fn(C.byref(a), _stream_ptr(dev)), "mlstm")
-    return out
+    return o if out is None else out
+
+
+def head_norm_matmul_supported(o, W):
+    return W.dtype == torch.bfloat16 and o.shape[0] <= 8 and W.shape[1] % 8 == 0 and W.shape[1] <= 12288
+
+
+def head_norm_matmul(o, gate, norm_w, heads, eps, W):
+    """(rms_norm of each head of o, times norm_w, times sigmoid(gate)) . W^T in float: the end of a recurrent mixer's
+    decode step in one launch."""
+    N, K = W.shape
+    y32 = torch.empty(o.shape[0], ceil_to(N, 4), dtype=torch.float32, device=o.device)
+    a = _lib.DenseMM(dtype=DTYPES[W.dtype], N=N, K=K, rows=o.shape[0], n_matrices=1, split=0, alpha=1.0, W=W.data_ptr(),
+                     y32=y32.data_ptr(), ldy32=y32.stride(0), hn_o=o.data_ptr(), hn_g=gate.data_ptr(), hn_ldg=gate.stride(0),
+                     hn_w=norm_w.data_ptr(), hn_heads=heads, hn_eps=eps)
+    with torch.cuda.device(o.device):
+        _lib.check_dense(_lib.dense().glq_dense_matmul(C.byref(a), _stream_ptr(o.device)), "head_norm_matmul")
+    return y32[:, :N]
 
 
 class Latent:
@@ -157,6 +178,7 @@ class Latent:
             _lib.check_dense(fn(C.byref(self.a), _stream_ptr(self.dev)), what)
 
     def prep(self):
+        """Rotates q in place and writes the cache rows: comes before ``prefill``; ``absorbed`` does both by itself."""
         self._call(_lib.dense().glq_latent_prep, "latent_prep")
 
     def prefill_supported(self):

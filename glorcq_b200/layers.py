@@ -50,8 +50,12 @@ class MatrixMemoryMixer(nn.Module):
     def forward(self, h, B, T, start, kv_len, state):
         qkvg, gates = dense.matmul(h, self.w_in, split=self.split)
         chunked = T > SHORT_PASS and h.dtype == torch.bfloat16 and self.dim % 8 == 0 and self.vdim % 8 == 0
+        fused = not chunked and dense.head_norm_matmul_supported(qkvg, self.w_out)
         o = dense.mlstm(qkvg, gates, B, T, self.heads, self.dim, self.vdim, self.cap, self.eps, self.bias_i, self.bias_f,
-                        self.norm_w, state, chunked, state_idle=True)
+                        self.norm_w, state, chunked, state_idle=True, raw=fused)
+        if fused:
+            gate = qkvg[:, 2 * self.heads * self.dim + self.heads * self.vdim:]
+            return dense.head_norm_matmul(o, gate, self.norm_w, self.heads, self.eps, self.w_out)
         return dense.matmul(o, self.w_out, split=0)[1]
 
 
@@ -95,10 +99,10 @@ class LatentAttentionMixer(nn.Module):
         y = torch.empty(B * T, self.heads * self.vdim, dtype=h.dtype, device=h.device)
         call = dense.Latent(q, rest, rest[:, self.kv_rank + self.rot_dim:], start, B, T, self.heads, self.dim, self.rot_dim,
                             self.vdim, self.kv_rank, self.rot_dims, self.scale, self.eps, self.norm_w, cos, sin, state, y)
-        call.prep()
         if T <= SHORT_PASS or kv_len is None or not call.prefill_supported():
             call.absorbed(self.ukt, self.uv)
         else:
+            call.prep()
             kv = torch.empty(B, kv_len, self.w_kv.shape[0], dtype=h.dtype, device=h.device) if B > 1 else None
             for b in range(B):
                 one = dense.matmul(state.rows[b], self.w_kv, rows=kv_len)[0]

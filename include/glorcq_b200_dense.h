@@ -54,6 +54,14 @@ typedef struct glq_dense_mm {
     float* y32;
     int64_t ldy32;
     void* gather;          /* (rows, K) scratch for entry_row on the tensor-core path, or NULL when entry_row is */
+    /* up to 8 rows, bf16, instead of x: row = rms_norm over each of hn_heads equal parts of hn_o (rows, K) float, times
+     * hn_w (K), times sigmoid(hn_g (rows, K) bf16, row stride hn_ldg) */
+    const float* hn_o;
+    const void* hn_g;
+    int64_t hn_ldg;
+    const float* hn_w;
+    int32_t hn_heads;
+    float hn_eps;
 } glq_dense_mm_t;
 int glq_dense_matmul(const glq_dense_mm_t* a, void* stream);
 /* 0: generic kernel, 1: streaming kernel (few rows), 2: tcgen05 kernel */
@@ -72,7 +80,7 @@ int glq_dense_add_norm(int dtype, const float* y, const float* w, const float* f
  *   S = e^(f + m - m') S + e^(i - m') k v^T (n alike), o = S^T q / (max(|n.q|, e^-m') + 1e-6), q scaled by D^-1/2
  *   out = rms_norm_per_head(o) * norm_w * sigmoid(g)
  * qkvg (B*T, ldp): q (H*D) | k (H*D) | v (H*V) | g (H*V) of `dtype`; gates (B*T, ldg) float: i (H) | f (H).
- * State: S (B, H, D, V), n (B, H, slices, D), m (B, H, slices) float, slices = glq_mlstm_slices(V).             */
+ * State: S (B, H, slices, D, 32), n (B, H, slices, D), m (B, H, slices) float, slices = glq_mlstm_slices(V).             */
 typedef struct glq_mlstm {
     int32_t dtype, B, T, H, D, V;
     int32_t state_idle;    /* step: 1 when the launch right before this one on the stream does not touch this state */
@@ -87,21 +95,21 @@ typedef struct glq_mlstm {
     float* S;
     float* n;
     float* m;
-    void* out;             /* (B*T, H*V) of dtype */
-    void* workspace;
+    float* o;              /* (B*T, H*V) float: the recurrence's output before norm and gate */
+    void* out;             /* (B*T, H*V) of dtype; step: NULL leaves norm and gate to the caller (glq_dense_matmul, hn_o) */
+    void* workspace;       /* chunk */
     size_t workspace_bytes;
-    int32_t* counters;     /* B*H, zero before the first call, left zero */
 } glq_mlstm_t;
 int glq_mlstm_slices(int V);
-size_t glq_mlstm_workspace_bytes(const glq_mlstm_t* a, int chunked);
+size_t glq_mlstm_workspace_bytes(const glq_mlstm_t* a);
 int glq_mlstm_step(const glq_mlstm_t* a, void* stream);    /* recurrent form, any T */
 int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream);   /* chunkwise form on the tensor cores, bf16 */
 
 /* Latent attention.  Cache row of a position: latent (K) | rotated key part (R), `dtype`, row stride ldc.
- * prep: latents of the new positions are RMS-normed (weight norm_w), the shared key part and every head's rotated
- *   query part (in place in q) are turned, and the cache rows start .. start + T - 1 are written.
+ * prep (before prefill): latents of the new positions are RMS-normed (weight norm_w), the shared key part and every
+ *   head's rotated query part (in place in q) are turned, and the cache rows start .. start + T - 1 are written.
  *   q (B*T, ldq): head by head D | R.  ckr (B*T, ldk) float: K | R.  cos/sin (max_len, rot_dims / 2) float.
- * absorbed (decode, short portions, any T in float32): scores against the cached latents themselves with
+ * absorbed (decode, short portions, any T in float32; turns q and writes the cache rows itself): scores against the cached latents themselves with
  *   q' = uk^T q, then the value projection uv of the weighted latent, times sigmoid of the head's gate.
  *   ukt (H, K, D), uv (H, V, K) of dtype, gate (B*T, ldk) float at column offset given by the pointer.
  * prefill (bf16): keys and values already projected, kv (B*S, ldkv): H*D keys | H*V values for positions 0..S-1,
