@@ -282,7 +282,7 @@ __global__ void __launch_bounds__(256) dense_route_kernel(const RtParams p) {
 
 // few entries: routing and lists in one CTA
 constexpr int kRouteOneCta = 1024;
-__global__ void __launch_bounds__(256) dense_route_plan_kernel(const RtParams p) {
+__global__ void __launch_bounds__(1024) dense_route_plan_kernel(const RtParams p) {
     extern __shared__ float rt_sc[];
     __shared__ int s_sel[kRouteOneCta];
     __shared__ float s_wts[kRouteOneCta];
@@ -290,7 +290,8 @@ __global__ void __launch_bounds__(256) dense_route_plan_kernel(const RtParams p)
     pdl_wait();
     pdl_release();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int t = warp; t < p.n; t += 8) route_corrected(p, t, lane, rt_sc + (size_t)warp * 2 * p.A, s_sel, s_wts);
+    if (warp < 8)       // the lists take all warps
+        for (int t = warp; t < p.n; t += 8) route_corrected(p, t, lane, rt_sc + (size_t)warp * 2 * p.A, s_sel, s_wts);
     __syncthreads();
     const int ms = p.max_slots;
     plan_entries<float>(cnt, p.n, p.E, p.top, p.chunk, 0, 1, s_sel, s_wts, p.active, p.n_active, p.slot_count, p.slot_offset,
@@ -388,7 +389,7 @@ extern "C" int glq_route(const glq_route_t* a, void* stream) {
     p.max_slots = a->max_slots;
     const int nk = a->n * a->top;
     const size_t sc = (size_t)16 * p.A * 4;
-    if (nk <= kRouteOneCta && a->n <= 128) return dn_launch(dense_route_plan_kernel, dim3(1), 256, sc + (size_t)2 * p.E * 4, stream, p);
+    if (nk <= kRouteOneCta && a->n <= 128) return dn_launch(dense_route_plan_kernel, dim3(1), 1024, sc + (size_t)2 * p.E * 4, stream, p);
     if (!a->block_counts) return GLQ_ERR_ARG;
     int st = dn_launch(dense_route_kernel, dim3(cdiv_i(a->n, 8)), 256, sc, stream, p);
     if (st != GLQ_OK) return st;

@@ -3,6 +3,8 @@
 
 #include <cuda_bf16.h>
 
+#include <cstdlib>
+
 #include "../../include/glorcq_b200_dense.h"
 #include "tc_mm.cuh"
 
@@ -110,27 +112,21 @@ inline int dn_sms() {
 // Launch that may start while its predecessor drains: every kernel here calls pdl_wait() before it touches anything a
 // predecessor wrote.
 template <typename... KArgs, typename... Args>
-inline int dn_launch_cluster(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, int cluster, void* stream, Args... args) {
+inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+    static const bool pdl = std::getenv("GLQ_NO_PDL") == nullptr;
     if (smem > 48 * 1024) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(block);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
-    cudaLaunchAttribute attr[2]{};
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
-    attr[1].id = cudaLaunchAttributeClusterDimension;
-    attr[1].val.clusterDim.x = cluster;
-    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
-    cfg.attrs = attr;
-    cfg.numAttrs = cluster > 1 ? 2 : 1;
+    cudaLaunchAttribute attr{};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = pdl ? 1 : 0;
     DN_CUDA(cudaLaunchKernelEx(&cfg, kern, KArgs(args)...));
     return GLQ_OK;
-}
-template <typename... KArgs, typename... Args>
-inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
-    return dn_launch_cluster(kern, grid, block, smem, 1, stream, args...);
 }
 
 }  // namespace glq

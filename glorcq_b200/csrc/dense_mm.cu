@@ -31,7 +31,6 @@ struct DmParams {
     int N, K, rows, slots, split, act;
     float alpha;
     int vec_y, vec_y32;
-    int cluster, xs_max;             // streaming kernel: CTAs that share a tile's k range; activation row stride
     const float* hn_o;               // streaming kernel: rows made from a recurrence's output (see glq_dense_mm_t)
     const void* hn_g;
     const float* hn_w;
@@ -59,51 +58,24 @@ template <typename T> __device__ __forceinline__ void dm_store(const DmParams& p
 // =====================================================================================================
 __device__ __forceinline__ uint4 dm_ldg(const uint4* p) {
     uint4 v;
-    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];"
+    asm volatile("ld.global.nc.L1::no_allocate.L2::256B.v4.u32 {%0,%1,%2,%3}, [%4];"
                  : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
                  : "l"(p));
     return v;
 }
-__device__ __forceinline__ uint32_t cluster_rank() {
-    uint32_t r;
-    asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
-    return r;
-}
-__device__ __forceinline__ uint32_t cluster_addr(uint32_t saddr, uint32_t rank) {
-    uint32_t a;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(saddr), "r"(rank));
-    return a;
-}
-__device__ __forceinline__ void st_cluster(uint32_t addr, float v) {
-    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory");
-}
-__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
-__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
-constexpr int kDmMaxCluster = 4;
-#ifndef GLQ_DM_DEPTH
-#define GLQ_DM_DEPTH 4
-#define GLQ_DM_CTAS 3
-#endif
-
-// SPLIT warps share one 16-row tile; with p.cluster > 1 the CTAs of a cluster share its k range as well, and the first of
-// them adds the others' sums (in rank order).  DEPTH 16-byte loads per lane and row are in flight.
-template <int SPLIT, int DEPTH, int CTAS>
-__global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmParams p) {
-    constexpr int TILES = kWarpsPerCta / SPLIT;
+// WARPS warps a CTA, SPLIT of them share one 16-row tile; DEPTH 16-byte loads per lane and row are in flight.
+template <int WARPS, int SPLIT, int DEPTH, int CTAS>
+__global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const DmParams p) {
+    constexpr int TILES = WARPS / SPLIT, THREADS = WARPS * 32;
     extern __shared__ __align__(16) unsigned char dm_smem[];
-    __shared__ float4 s_part[kDmMaxCluster][32];
     const int K = p.K, tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
     const int g = lane >> 2, t = lane & 3;
     const int tw = w / SPLIT, s = w % SPLIT;
-    const int cs = p.cluster, rank = cs > 1 ? (int)cluster_rank() : 0;
-    const int bx = (int)blockIdx.x / cs, nbx = (int)gridDim.x / cs;
-    // 32-channel chunks of this CTA, and of this warp inside it
-    const int chunks = (K + 31) / 32;
-    const int a_lo = (int)((long)rank * chunks / cs), a_hi = (int)((long)(rank + 1) * chunks / cs), an = a_hi - a_lo;
-    const int c_lo = a_lo + (int)((long)s * an / SPLIT), c_hi = a_lo + (int)((long)(s + 1) * an / SPLIT);
-    const int XS = (an + 1) * 32;                                  // padded activation rows: distinct banks
+    const int chunks = (K + 31) / 32;                              // of 32 channels
+    const int c_lo = (int)((long)s * chunks / SPLIT), c_hi = (int)((long)(s + 1) * chunks / SPLIT);
+    const int XS = (chunks + 1) * 32;                              // padded activation rows: distinct banks
     bf16* xs = reinterpret_cast<bf16*>(dm_smem);
-    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * p.xs_max * 2);
+    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * XS * 2);
     const int ntiles = (p.N + 15) / 16;
     const bool plain = p.slot_index == nullptr;
     DmSlot sl{0, 0, p.rows};
@@ -111,13 +83,12 @@ __global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmPa
         pdl_wait();
         pdl_release();
         sl = dm_slot(p, blockIdx.y);
-        if (sl.cnt == 0) return;                                   // the whole cluster: its CTAs share blockIdx.y
+        if (sl.cnt == 0) return;
     }
-    if (cs > 1) cluster_arrive();                                  // "this CTA runs": waited for before its memory is written
     const bf16* Wm = reinterpret_cast<const bf16*>(p.W) + (size_t)sl.mat * p.N * K;
-    const int iters = (ntiles + TILES * nbx - 1) / (TILES * nbx);
+    const int iters = (ntiles + TILES * (int)gridDim.x - 1) / (TILES * (int)gridDim.x);
     for (int it = 0; it < iters; ++it) {
-        const int tile = (it * nbx + bx) * TILES + tw;
+        const int tile = (it * (int)gridDim.x + (int)blockIdx.x) * TILES + tw;
         const bool live = tile < ntiles;
         const int r0 = min(tile * 16 + g, p.N - 1), r1 = min(tile * 16 + g + 8, p.N - 1);
         const bf16* w0 = Wm + (size_t)r0 * K + t * 8;
@@ -139,12 +110,10 @@ __global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmPa
             if (p.hn_o) {
                 // rows = per-head RMS norm of hn_o, times its weight, times the sigmoid of the gate; warp = (row, head)
                 const int V = K / p.hn_heads;
-                for (int i = w; i < 8 * p.hn_heads; i += kWarpsPerCta) {
+                for (int i = w; i < 8 * p.hn_heads; i += WARPS) {
                     const int row = i / p.hn_heads, k0 = (i % p.hn_heads) * V;
-                    const int lo = max(k0, a_lo * 32), hi = min(k0 + V, a_hi * 32);
-                    if (lo >= hi) continue;
                     if (row >= sl.cnt) {
-                        for (int k = lo + lane; k < hi; k += 32) xs[(size_t)row * XS + k - a_lo * 32] = from_f<bf16>(0.f);
+                        for (int k = k0 + lane; k < k0 + V; k += 32) xs[(size_t)row * XS + k] = from_f<bf16>(0.f);
                         continue;
                     }
                     const float* o = p.hn_o + (size_t)row * K;
@@ -161,16 +130,16 @@ __global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmPa
                     const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
                     const bf16* gt = reinterpret_cast<const bf16*>(p.hn_g) + (size_t)row * p.hn_ldg;
 #pragma unroll 4
-                    for (int k = lo + lane; k < hi; k += 32)
-                        xs[(size_t)row * XS + k - a_lo * 32] = from_f<bf16>(o[k] * inv * p.hn_w[k] * sigmoid_f(to_f(gt[k])));
+                    for (int k = k0 + lane; k < k0 + V; k += 32)
+                        xs[(size_t)row * XS + k] = from_f<bf16>(o[k] * inv * p.hn_w[k] * sigmoid_f(to_f(gt[k])));
                 }
-                for (int i = tid; i < 8 * 32; i += kThreads) {       // channels past K of the last chunk
+                for (int i = tid; i < 8 * 32; i += THREADS) {        // channels past K of the last chunk
                     const int k = K + (i & 31);
-                    if (k < a_hi * 32) xs[(size_t)(i >> 5) * XS + k - a_lo * 32] = from_f<bf16>(0.f);
+                    if (k < chunks * 32) xs[(size_t)(i >> 5) * XS + k] = from_f<bf16>(0.f);
                 }
             } else {
-                for (int i = tid; i < 8 * an * 4; i += kThreads) {
-                    const int row = i / (an * 4), c = i % (an * 4), k = a_lo * 32 + c * 8;
+                for (int i = tid; i < 8 * chunks * 4; i += THREADS) {
+                    const int row = i / (chunks * 4), c = i % (chunks * 4), k = c * 8;
                     uint4 v = make_uint4(0, 0, 0, 0);
                     if (row < sl.cnt && k < K) {
                         const int e = sl.off + row;
@@ -191,7 +160,7 @@ __global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmPa
                 if (c < c_hi) {
                     const uint4 a = qa[d], b = qb[d];
                     fetch(c + DEPTH, d);
-                    const uint4 xv = xb[(c - a_lo) * 4];
+                    const uint4 xv = xb[c * 4];
                     mma_bf16(acc, a.x, b.x, a.y, b.y, xv.x, xv.y);
                     mma_bf16(acc, a.z, b.z, a.w, b.w, xv.z, xv.w);
                 }
@@ -207,25 +176,6 @@ __global__ void __launch_bounds__(kThreads, CTAS) dense_stream_kernel(const DmPa
                 acc[2] += v.z;
                 acc[3] += v.w;
             }
-        }
-        if (cs > 1) {                // SPLIT == 8, one tile per cluster
-            cluster_wait();
-            if (w == 0 && rank != 0) {
-                const uint32_t dst = cluster_addr(smem_u32(&s_part[rank][lane]), 0);
-#pragma unroll
-                for (int i = 0; i < 4; ++i) st_cluster(dst + 4 * i, acc[i]);
-            }
-            cluster_arrive();
-            cluster_wait();
-            if (rank != 0) return;
-            if (w == 0)
-                for (int r = 1; r < cs; ++r) {
-                    const float4 v = s_part[r][lane];
-                    acc[0] += v.x;
-                    acc[1] += v.y;
-                    acc[2] += v.z;
-                    acc[3] += v.w;
-                }
         }
         if (s == 0 && live) {
 #pragma unroll
@@ -622,16 +572,19 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     }
     const int rows_max = grouped ? a->max_slot_rows : a->rows;
     if (path == 1) {
-        const int tiles = cdiv_i(a->N, 16), sms = dn_sms(), chunks = cdiv_i(a->K, 32);
-        p.cluster = 1;
-        const bool wide = (long)tiles * p.slots > 12L * sms;       // enough tiles: four warps each, CTAs walk over them
-        if (!wide)
-            while (p.cluster < kDmMaxCluster && (long)tiles * p.slots * p.cluster < 2L * sms && chunks >= 32 * p.cluster) p.cluster *= 2;
-        p.xs_max = (cdiv_i(chunks, p.cluster) + 1) * 32;
-        const size_t smem = (size_t)8 * p.xs_max * 2 + (size_t)kWarpsPerCta * 32 * sizeof(float4);
-        if (wide)
-            return dn_launch(dense_stream_kernel<4, 8, 2>, dim3(std::min(cdiv_i(tiles, 2), 2 * sms), p.slots), kThreads, smem, stream, p);
-        return dn_launch_cluster(dense_stream_kernel<8, GLQ_DM_DEPTH, GLQ_DM_CTAS>, dim3(tiles * p.cluster, p.slots), kThreads, smem, p.cluster, stream, p);
+        const int tiles = cdiv_i(a->N, 16), sms = dn_sms();
+        auto go = [&](auto kern, int warps, int grid) {
+            const size_t smem = (size_t)8 * (cdiv_i(a->K, 32) + 1) * 32 * 2 + (size_t)warps * 32 * sizeof(float4);
+            return dn_launch(kern, dim3(grid, p.slots), warps * 32, smem, stream, p);
+        };
+        // measured on 1 x N x K products of 6 to 25 MB: many tiles walk over resident CTAs; a few per SM fit one wave of
+        // small CTAs; less than one per SM takes deep loads, with sixteen warps on a tile when rows are long
+        const long work = (long)tiles * p.slots;
+        if (work > 12L * sms) return go(dense_stream_kernel<8, 4, 8, 2>, 8, std::min(cdiv_i(tiles, 2), 2 * sms));
+        if (work > 3L * sms) return go(dense_stream_kernel<4, 4, 8, 4>, 4, tiles);
+        if (work > sms) return go(dense_stream_kernel<8, 8, 4, 3>, 8, tiles);
+        if (a->K >= 4096) return go(dense_stream_kernel<16, 16, 8, 1>, 16, tiles);
+        return go(dense_stream_kernel<8, 8, 8, 2>, 8, tiles);
     }
     if (path == 2) {
         const void* xa = a->x;

@@ -33,6 +33,7 @@ struct LaParams {
     float* po;           // (B, tiles, splits, 16, K)
     float* pm;           // (B, tiles, splits, 16)
     float* pl;
+    float* ol;           // (B * T, H, K) weighted latents
     int KRp, rows16, splits;
 };
 
@@ -194,57 +195,67 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LaParams p) {
     }
 }
 
-// combine the splits of a row, project the weighted latent with the head's value matrix, apply the head's gate
+constexpr int kMaxSplits = 128;
+
+// weighted latent of a (row, head): the splits' sums combined; grid (rows, heads, column parts)
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LaParams p) {
+    __shared__ float sw[kMaxSplits];
+    pdl_wait();
+    pdl_release();
+    const int row = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
+    const int rr = (row % p.T) * p.H + h;
+    const size_t first = (((size_t)(row / p.T) * (p.rows16 / 16) + rr / 16) * p.splits) * 16 + rr % 16;     // split z: + 16 z
+    if (threadIdx.x < 32) {
+        float mz[kMaxSplits / 32], lz[kMaxSplits / 32], m = -INFINITY;
+#pragma unroll
+        for (int u = 0; u < kMaxSplits / 32; ++u) {
+            const int z = lane + 32 * u;
+            mz[u] = z < p.splits ? p.pm[first + 16 * z] : -INFINITY;
+            lz[u] = z < p.splits ? p.pl[first + 16 * z] : 0.f;
+            m = fmaxf(m, mz[u]);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        float l = 0.f;
+#pragma unroll
+        for (int u = 0; u < kMaxSplits / 32; ++u) {
+            mz[u] = exp2f(mz[u] - m);
+            l += mz[u] * lz[u];
+        }
+        const float inv = 1.f / warp_sum(l);
+#pragma unroll
+        for (int u = 0; u < kMaxSplits / 32; ++u) sw[lane + 32 * u] = mz[u] * inv;
+    }
+    __syncthreads();
+    const int per = (p.K + gridDim.z - 1) / gridDim.z, k_hi = min(p.K, (int)(blockIdx.z + 1) * per);
+    for (int k = blockIdx.z * per + threadIdx.x; k < k_hi; k += 128) {
+        const float* po = p.po + first * p.K + k;
+        float v = 0.f;
+#pragma unroll 16
+        for (int z = 0; z < p.splits; ++z) {
+            // a split without a visible position left its sums unwritten
+            const float w = sw[z], x = w != 0.f ? po[(size_t)16 * z * p.K] : 0.f;
+            v += w * x;
+        }
+        p.ol[((size_t)row * p.H + h) * p.K + k] = v;
+    }
+}
+
+// the head's value matrix times the weighted latent, times the head's gate
 template <typename T>
 __global__ void __launch_bounds__(256) latent_value_kernel(const LaParams p) {
     extern __shared__ float xs[];
-    __shared__ float sw[kHmRows][64];
     const int Kp = (p.K + 7) / 8 * 8;
     pdl_wait();
     pdl_release();
-    const int h = blockIdx.x, rows = p.B * p.T, tiles = p.rows16 / 16;
+    const int h = blockIdx.x, rows = p.B * p.T;
     const int per = (p.V + gridDim.y - 1) / gridDim.y, n_lo = blockIdx.y * per, n_hi = min(p.V, n_lo + per);
     for (int r0 = blockIdx.z * kHmRows; r0 < rows; r0 += gridDim.z * kHmRows) {
         const int nr = min(kHmRows, rows - r0);
         __syncthreads();
-        auto part = [&](int r, int z) {              // index of (row, split) among the partial sums
-            const int row = r0 + r, rr = (row % p.T) * p.H + h;
-            return (((size_t)(row / p.T) * tiles + rr / 16) * p.splits + z) * 16 + rr % 16;
-        };
-        {
-            const int r = threadIdx.x >> 5, lane = threadIdx.x & 31;       // warp = row, lane = splits lane, lane + 32
-            if (r < nr) {
-                float mz[2], lz[2];
-#pragma unroll
-                for (int u = 0; u < 2; ++u) {
-                    const int z = lane + 32 * u;
-                    mz[u] = z < p.splits ? p.pm[part(r, z)] : -INFINITY;
-                    lz[u] = z < p.splits ? p.pl[part(r, z)] : 0.f;
-                }
-                float m = fmaxf(mz[0], mz[1]);
-#pragma unroll
-                for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-                const float w0 = exp2f(mz[0] - m), w1 = exp2f(mz[1] - m);
-                const float inv = 1.f / warp_sum(w0 * lz[0] + w1 * lz[1]);
-                sw[r][lane] = w0 * inv;
-                sw[r][lane + 32] = w1 * inv;
-            }
-        }
-        __syncthreads();
         for (int i = threadIdx.x; i < nr * Kp; i += 256) {
             const int r = i / Kp, k = i % Kp;
-            float v = 0.f;
-            if (k < p.K) {
-                const float* po = p.po + part(r, 0) * p.K + k;
-                const size_t step = (size_t)16 * p.K;
-#pragma unroll 8
-                for (int z = 0; z < p.splits; ++z) {
-                    // a split without a visible position left its sums unwritten
-                    const float w = sw[r][z], x = w != 0.f ? po[z * step] : 0.f;
-                    v += w * x;
-                }
-            }
-            xs[i] = v;
+            xs[i] = k < p.K ? p.ol[((size_t)(r0 + r) * p.H + h) * p.K + k] : 0.f;
         }
         __syncthreads();
         head_products(reinterpret_cast<const T*>(p.uv) + (size_t)h * p.V * p.K, n_lo, n_hi, p.K, p.K % 8 == 0, xs, Kp, nr,
@@ -703,12 +714,12 @@ static bool la_tensor(const glq_latent_t* a) {
 static int la_splits(const glq_latent_t* a) {
     if (!la_tensor(a)) return 1;
     const long ctas = (long)a->B * ((a->T * a->H + 15) / 16);
-    const long want = std::max<long>(1, 2L * dn_sms() / ctas), tiles = cdiv_i(a->max_len, kAbPos);
-    const long cap = a->max_splits > 0 ? std::min(a->max_splits, 64) : 64;
+    const long want = std::max<long>(1, dn_sms() / ctas), tiles = cdiv_i(a->max_len, kAbPos);
+    const long cap = a->max_splits > 0 ? std::min(a->max_splits, kMaxSplits) : kMaxSplits;
     return (int)std::min(std::min(want, tiles), cap);
 }
 struct LaWs {
-    size_t qa, po, pm, pl, total;
+    size_t qa, po, pm, pl, ol, total;
 };
 static LaWs la_ws(const glq_latent_t* a) {
     const LaParams p = la_params(a);
@@ -719,7 +730,8 @@ static LaWs la_ws(const glq_latent_t* a) {
     w.po = up(la_tensor(a) ? rows * p.KRp * 4 : rows * (a->K + a->R) * 4);
     w.pm = w.po + up(parts * a->K * 4);
     w.pl = w.pm + up(parts * 4);
-    w.total = w.pl + up(parts * 4);
+    w.ol = w.pl + up(parts * 4);
+    w.total = w.ol + up((size_t)a->B * a->T * a->H * a->K * 4);
     return w;
 }
 
@@ -744,6 +756,7 @@ template <typename T> static int la_absorbed(const glq_latent_t* a, void* stream
     p.po = reinterpret_cast<float*>(ws + w.po);
     p.pm = reinterpret_cast<float*>(ws + w.pm);
     p.pl = reinterpret_cast<float*>(ws + w.pl);
+    p.ol = reinterpret_cast<float*>(ws + w.ol);
     p.splits = la_splits(a);
     const bool tensor = la_tensor(a);
     const int rb = std::min(cdiv_i((long)a->B * a->T, kHmRows), 512);
@@ -757,7 +770,7 @@ template <typename T> static int la_absorbed(const glq_latent_t* a, void* stream
     const size_t xa = (size_t)kHmRows * ((a->D + 7) / 8 * 8) * 4, xv = (size_t)kHmRows * ((a->K + 7) / 8 * 8) * 4;
     int st;
     if (tensor) {
-        st = dn_launch(latent_absorb_kernel<T, true>, dim3(a->H + 1, parts(a->K, a->D, 2L * dn_sms()), rb), 256, xa, stream, p);
+        st = dn_launch(latent_absorb_kernel<T, true>, dim3(a->H + 1, parts(a->K, a->D, 4L * dn_sms()), rb), 256, xa, stream, p);
         if (st != GLQ_OK) return st;
         const dim3 grid(p.rows16 / 16, p.splits, a->B);
         const size_t smem = la_absorbed_smem(p);
@@ -765,13 +778,17 @@ template <typename T> static int la_absorbed(const glq_latent_t* a, void* stream
         else if (a->K <= 256) st = dn_launch(latent_absorbed_kernel<4>, grid, 256, smem, stream, p);
         else st = dn_launch(latent_absorbed_kernel<8>, grid, 256, smem, stream, p);
     } else {
-        st = dn_launch(latent_absorb_kernel<T, false>, dim3(a->H + 1, parts(a->K, a->D, 2L * dn_sms()), rb), 256, xa, stream, p);
+        st = dn_launch(latent_absorb_kernel<T, false>, dim3(a->H + 1, parts(a->K, a->D, 4L * dn_sms()), rb), 256, xa, stream, p);
         if (st != GLQ_OK) return st;
         const size_t smem = (size_t)(2 * a->K + a->R + 128) * 4;
         st = dn_launch(latent_absorbed_generic_kernel<T>, dim3(a->T * a->H, a->B), 128, smem, stream, p);
     }
     if (st != GLQ_OK) return st;
-    return dn_launch(latent_value_kernel<T>, dim3(a->H, parts(a->V, a->K, dn_sms() / 2), rb), 256, xv, stream, p);
+    const long rh = (long)a->B * a->T * a->H;
+    const int kp = (int)std::max<long>(1, std::min<long>(cdiv_i(a->K, 128), cdiv_i(2L * dn_sms(), rh)));
+    st = dn_launch(latent_combine_kernel, dim3(a->B * a->T, a->H, kp), 128, 0, stream, p);
+    if (st != GLQ_OK) return st;
+    return dn_launch(latent_value_kernel<T>, dim3(a->H, parts(a->V, a->K, 2L * dn_sms()), rb), 256, xv, stream, p);
 }
 
 extern "C" int glq_latent_absorbed(const glq_latent_t* a, void* stream) {
@@ -779,7 +796,7 @@ extern "C" int glq_latent_absorbed(const glq_latent_t* a, void* stream) {
         !a->out || !a->workspace)
         return GLQ_ERR_ARG;
     if (!al16(a->workspace) || !al16(a->ukt) || !al16(a->uv)) return GLQ_ERR_ALIGN;
-    if (a->K > 4096 || a->D > 4096 || a->R > 4096 || a->B > 65535) return GLQ_ERR_UNSUPPORTED;
+    if (a->K > 4096 || a->D > 4096 || a->R > 4096 || a->B > 65535 || a->H > 65534) return GLQ_ERR_UNSUPPORTED;
     if (a->T == 0) return GLQ_OK;
     return a->dtype == GLQ_DT_BF16 ? la_absorbed<bf16>(a, stream) : la_absorbed<float>(a, stream);
 }

@@ -32,7 +32,7 @@ struct MlParams {
     float* o;                      // (B * Tall, H * V)
     long long ldp, ldg;
     int B, T, H, D, V, slices;
-    int state_idle;
+    int state_idle, vec4;          // vec4: gates, norm weights and outputs allow reads of four values
     int t0, Tall;                  // this call's positions: t0 .. t0 + T - 1 of the Tall rows of a sequence
     float cap, eps, scale;
     // chunk form
@@ -49,14 +49,27 @@ __device__ __forceinline__ float log_f(const MlParams& p, size_t row, int h) {
     return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
 }
 
-// rows row0 .. of head h: out = rms_norm(o) * w * sigmoid(g); one warp per row
+__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
+}
+__device__ __forceinline__ void ld4(const bf16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v[0] = bf_lo(a.x), v[1] = bf_hi(a.x), v[2] = bf_lo(a.y), v[3] = bf_hi(a.y);
+}
+__device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void st4(bf16* p, float a, float b, float c, float d) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(a, b), pack_bf2(c, d));
+}
+
+// one row of head h: out = rms_norm(o) * w * sigmoid(g); one warp
 template <typename T>
 __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, int h, int lane) {
     const float* o = p.o + row * p.H * p.V + (size_t)h * p.V;
     const T* g = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)p.H * (2 * p.D + p.V) + (size_t)h * p.V;
     T* out = reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V;
     float ss = 0.f;
-    if (p.V % 4 == 0 && p.V <= 1024) {          // four values per lane and step, kept in registers
+    if (p.V % 4 == 0 && p.V <= 1024 && p.vec4) {          // four values per lane and step, kept in registers
         float4 x[8];
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
@@ -70,9 +83,11 @@ __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, in
         for (int u = 0; u < 8; ++u) {
             const int v = (u * 32 + lane) * 4;
             if (v < p.V) {
-                const float y[4] = {x[u].x, x[u].y, x[u].z, x[u].w};
-#pragma unroll
-                for (int i = 0; i < 4; ++i) out[v + i] = from_f<T>(y[i] * inv * w[v + i] * sigmoid_f(to_f(g[v + i])));
+                float gv[4];
+                ld4(g + v, gv);
+                const float4 wv = *reinterpret_cast<const float4*>(w + v);
+                st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[0]), x[u].y * inv * wv.y * sigmoid_f(gv[1]),
+                    x[u].z * inv * wv.z * sigmoid_f(gv[2]), x[u].w * inv * wv.w * sigmoid_f(gv[3]));
             }
         }
         return;
@@ -242,11 +257,11 @@ __device__ __forceinline__ uint32_t transpose8(uint32_t v) {
 // products take, [d / 16][v / 8][lane] of uint4 = (first part rows 0-7, rows 8-15, second part rows 0-7, rows 8-15).
 
 // state at every chunk's start (as sums of two bf16 parts, and n) and after the last chunk; one CTA owns 64 x 64 of a
-// head's S: warp = 16 rows
-__global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
+// head's S: warp = 16 rows x 32 columns
+__global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
     extern __shared__ __align__(16) unsigned char ml_raw[];
     __shared__ float ws[kL];
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+    const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, wv = tid >> 7, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.z % p.H, b = blockIdx.z / p.H;
     const int d0 = blockIdx.x * kTd, v0 = blockIdx.y * kTd;
     const size_t bh = blockIdx.z;
@@ -257,7 +272,7 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
         if (c < p.nc) {
             bf16* ks = reinterpret_cast<bf16*>(st);
             bf16* vs = ks + kL * kLd;
-            for (int i = tid; i < kL * 8; i += 128) {
+            for (int i = tid; i < kL * 8; i += 256) {
                 const int s = i >> 3, cc = (i & 7) * 8, tt = c * kL + s;
                 const size_t row = ((size_t)b * p.Tall + p.t0 + (tt < p.T ? tt : 0)) * p.ldp;
                 const bool kl = tt < p.T && d0 + cc < p.D, vl = tt < p.T && v0 + cc < p.V;
@@ -269,16 +284,16 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
         cpa_commit();
     };
     const int dr[2] = {d0 + 16 * warp + g, d0 + 16 * warp + g + 8};
-    float acc[8][4], nacc[2];
+    float acc[4][4], nacc[2];
     pdl_wait();
     pdl_release();
     for (int c = 0; c < kStStages - 1; ++c) load(c);
     const size_t slb = bh * p.slices;
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int v = v0 + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
+            const int v = v0 + 32 * wv + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
             acc[j][e] = d < p.D && v < p.V ? p.S[((slb + v / kSl) * p.D + d) * kSl + v % kSl] : 0.f;
         }
 #pragma unroll
@@ -302,21 +317,21 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
         m = m_end;
         tot = tot_next;
         // the state this chunk starts from
-        uint4* sb = reinterpret_cast<uint4*>(p.Sb) + ((bc * (p.Dp / 16) + d0 / 16 + warp) * (p.Vp / 8) + v0 / 8) * 32 + lane;
+        uint4* sb = reinterpret_cast<uint4*>(p.Sb) + ((bc * (p.Dp / 16) + d0 / 16 + warp) * (p.Vp / 8) + v0 / 8 + 4 * wv) * 32 + lane;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
+        for (int j = 0; j < 4; ++j) {
             uint32_t h0, l0, h1, l1;
             split_bf2(acc[j][0], acc[j][1], h0, l0);
             split_bf2(acc[j][2], acc[j][3], h1, l1);
             sb[j * 32] = make_uint4(transpose8(h0), transpose8(h1), transpose8(l0), transpose8(l1));
         }
-        if (blockIdx.y == 0 && t == 0) {
+        if (blockIdx.y == 0 && wv == 0 && t == 0) {
             p.nbuf[bc * p.Dp + dr[0]] = nacc[0];
             p.nbuf[bc * p.Dp + dr[1]] = nacc[1];
         }
         __syncthreads();
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+        for (int j = 0; j < 4; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[j][e] *= keep;
         float ns[2] = {0.f, 0.f};
@@ -331,15 +346,15 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
                 ns[i & 1] += x + y;
                 split_bf2(x, y, hi[i], lo[i]);
             }
+            uint32_t vb_[2][4];
 #pragma unroll
-            for (int jp = 0; jp < 4; ++jp) {
-                uint32_t b0, b1, b2, b3;
-                ldsm4_t(smem_u32(vt + (16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 16 * jp + (lane >> 4) * 8), b0, b1, b2, b3);
-                mma_bf16(acc[2 * jp], hi[0], hi[1], hi[2], hi[3], b0, b1);
-                mma_bf16(acc[2 * jp], lo[0], lo[1], lo[2], lo[3], b0, b1);
-                mma_bf16(acc[2 * jp + 1], hi[0], hi[1], hi[2], hi[3], b2, b3);
-                mma_bf16(acc[2 * jp + 1], lo[0], lo[1], lo[2], lo[3], b2, b3);
-            }
+            for (int jp = 0; jp < 2; ++jp)
+                ldsm4_t(smem_u32(vt + (16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 32 * wv + 16 * jp + (lane >> 4) * 8), vb_[jp][0],
+                        vb_[jp][1], vb_[jp][2], vb_[jp][3]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) mma_bf16(acc[j], hi[0], hi[1], hi[2], hi[3], vb_[j >> 1][2 * (j & 1)], vb_[j >> 1][2 * (j & 1) + 1]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) mma_bf16(acc[j], lo[0], lo[1], lo[2], lo[3], vb_[j >> 1][2 * (j & 1)], vb_[j >> 1][2 * (j & 1) + 1]);
         }
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
@@ -350,14 +365,14 @@ __global__ void __launch_bounds__(128) mlstm_state_kernel(const MlParams p) {
     }
     cpa_wait<0>();
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int v = v0 + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
+            const int v = v0 + 32 * wv + 8 * j + 2 * t + (e & 1), d = dr[e >> 1];
             if (d < p.D && v < p.V) p.S[((slb + v / kSl) * p.D + d) * kSl + v % kSl] = acc[j][e];
         }
     for (int s = v0 / kSl; s < min(p.slices, (v0 + kTd) / kSl); ++s) {
-        if (t == 0)
+        if (t == 0 && wv == 0)
 #pragma unroll
             for (int e = 0; e < 2; ++e)
                 if (dr[e] < p.D) p.n[(slb + s) * p.D + dr[e]] = nacc[e];
@@ -609,6 +624,7 @@ static int ml_params(const glq_mlstm_t* a, MlParams& p) {
     p.V = a->V;
     p.slices = glq_mlstm_slices(a->V);
     p.state_idle = a->state_idle;
+    p.vec4 = al16(a->qkvg) && al16(a->out) && al16(a->norm_w) && a->ldp % 4 == 0 && a->H * (2 * a->D + a->V) % 4 == 0;
     p.cap = a->gate_cap;
     p.eps = a->eps;
     p.scale = (float)(1.0 / sqrt((double)a->D));
@@ -659,7 +675,7 @@ extern "C" int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream) {
         p.T = std::min(kSegment, p.Tall - p.t0);
         p.nc = cdiv_i(p.T, kL);
         if ((st = dn_launch(mlstm_gate_kernel, dim3(cdiv_i(p.nc, 4), bh), 128, 0, stream, p)) != GLQ_OK) return st;
-        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 128, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
+        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 256, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
         if (p.V > 64) st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, MoCfg<128>::SMEM, stream, p);
         else st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, MoCfg<64>::SMEM, stream, p);
         if (st != GLQ_OK) return st;
