@@ -131,7 +131,7 @@ class DenseMM(C.Structure):
     """glq_dense_mm_t"""
     _fields_ = [(f, C.c_int32) for f in ("dtype", "act", "N", "K", "rows", "n_matrices", "max_slots", "max_slot_rows", "split")] + \
                [("alpha", C.c_float)] + [(f, vp) for f in ("slot_index", "n_slots", "slot_count", "slot_offset", "entry_row", "x")] + \
-               [("ldx", C.c_int64), ("W", vp), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp),
+               [("ldx", C.c_int64), ("W", vp), ("ldw", C.c_int64), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp),
                 ("hn_o", vp), ("hn_g", vp), ("hn_ldg", C.c_int64), ("hn_w", vp), ("hn_heads", C.c_int32), ("hn_eps", C.c_float)]
 
 
@@ -149,7 +149,7 @@ class Latent(C.Structure):
                [("scale", C.c_float), ("eps", C.c_float), ("start", vp), ("q", vp), ("ldq", C.c_int64), ("ckr", vp),
                 ("ldk", C.c_int64)] + [(f, vp) for f in ("gate", "norm_w", "cos_t", "sin_t", "cache")] + \
                [("ldc", C.c_int64)] + [(f, vp) for f in ("ukt", "uv", "out", "kv")] + \
-               [("ldkv", C.c_int64), ("S", C.c_int32), ("max_splits", C.c_int32), ("workspace", vp), ("workspace_bytes", C.c_size_t)]
+               [("ldkv", C.c_int64), ("vt", vp), ("ldvt", C.c_int64), ("S", C.c_int32), ("max_splits", C.c_int32), ("workspace", vp), ("workspace_bytes", C.c_size_t)]
 
 
 class Route(C.Structure):
@@ -176,7 +176,7 @@ _DENSE_SIGS = {
     "glq_latent_prep": (_i, [C.POINTER(Latent), vp]),
     "glq_latent_absorbed_workspace_bytes": (_z, [C.POINTER(Latent)]),
     "glq_latent_absorbed": (_i, [C.POINTER(Latent), vp]),
-    "glq_latent_prefill_supported": (_i, [C.POINTER(Latent)]),
+    "glq_latent_prefill_form": (_i, [C.POINTER(Latent)]),
     "glq_latent_prefill": (_i, [C.POINTER(Latent), vp]),
     "glq_route_max_slots": (_i, [_i, _i, _i, _i]),
     "glq_route": (_i, [C.POINTER(Route), vp]),

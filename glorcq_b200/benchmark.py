@@ -226,7 +226,10 @@ def prompt_kernels(t, size, T):
 
     def call():
         return dense.Latent(q, rest, rest[:, k + r:], start, 1, T, hh, d, r, v, k, r, (d + r) ** -0.5, 1e-5, nw, cos, sin, c, y)
-    sec = graph_time([lambda: call().prefill(kv, T)] * 4)
+    vt = torch.randn(hh * v, dense.ceil_to(T, 8), device=dev).to(bf)
+    two = call().prefill_form() == 2
+    keys = kv[:, :hh * d].contiguous() if two else kv
+    sec = graph_time([lambda: call().prefill(keys, T, vt if two else None)] * 4)
     t.add(f"latent attention, prompt ({T} positions, {hh} heads, {d + r} / {v})", sec, T * hh * (2 * d + r + 2 * v) * 2,
           float(T) * T * hh * (d + r + v), "prompt attention")
     sec = graph_time([lambda: call().prep()] * 4)

@@ -7,12 +7,7 @@
 //     accumulator is double-buffered in tensor memory so that the epilogue of a tile overlaps the next tile's products;
 //   * float32, or rows that are no multiple of 16 bytes: a tiled kernel on the CUDA cores.
 // Rows sums are taken in a fixed order in all three: results do not depend on what else is in the batch.
-#include <cuda.h>
-
-#include <cstdlib>
-#include <mutex>
-
-#include "dense_common.cuh"
+#include "tma.cuh"
 
 namespace glq {
 thread_local int g_dense_cuda_error = 0;
@@ -27,7 +22,7 @@ struct DmParams {
     const int* slot_count;
     const int* slot_offset;
     const int* entry_row;
-    long long ldx, ldy, ldy32;
+    long long ldx, ldy, ldy32, ldw;
     int N, K, rows, slots, split, act;
     float alpha;
     int vec_y, vec_y32;
@@ -85,14 +80,14 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
         sl = dm_slot(p, blockIdx.y);
         if (sl.cnt == 0) return;
     }
-    const bf16* Wm = reinterpret_cast<const bf16*>(p.W) + (size_t)sl.mat * p.N * K;
+    const bf16* Wm = reinterpret_cast<const bf16*>(p.W) + (size_t)sl.mat * p.N * p.ldw;
     const int iters = (ntiles + TILES * (int)gridDim.x - 1) / (TILES * (int)gridDim.x);
     for (int it = 0; it < iters; ++it) {
         const int tile = (it * (int)gridDim.x + (int)blockIdx.x) * TILES + tw;
         const bool live = tile < ntiles;
         const int r0 = min(tile * 16 + g, p.N - 1), r1 = min(tile * 16 + g + 8, p.N - 1);
-        const bf16* w0 = Wm + (size_t)r0 * K + t * 8;
-        const bf16* w1 = Wm + (size_t)r1 * K + t * 8;
+        const bf16* w0 = Wm + (size_t)r0 * p.ldw + t * 8;
+        const bf16* w1 = Wm + (size_t)r1 * p.ldw + t * 8;
         const int lim = K - 8 - t * 8;      // this lane's 8 channels of chunk c exist when 32 c <= lim
         uint4 qa[DEPTH], qb[DEPTH];
         auto fetch = [&](int c, int d) {
@@ -198,7 +193,7 @@ __global__ void __launch_bounds__(256) dense_generic_kernel(const DmParams p) {
     pdl_release();
     const DmSlot sl = dm_slot(p, blockIdx.z);
     const int n0 = blockIdx.x * 64;
-    const T* Wm = reinterpret_cast<const T*>(p.W) + (size_t)sl.mat * p.N * p.K;
+    const T* Wm = reinterpret_cast<const T*>(p.W) + (size_t)sl.mat * p.N * p.ldw;
     const T* X = reinterpret_cast<const T*>(p.x);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     for (int m0 = blockIdx.y * 64; m0 < sl.cnt; m0 += gridDim.y * 64) {
@@ -214,7 +209,7 @@ __global__ void __launch_bounds__(256) dense_generic_kernel(const DmParams p) {
                     const long long xr = p.entry_row ? p.entry_row[e] : e;
                     xv = to_f(X[xr * p.ldx + k0 + kk]);
                 }
-                if (kin && n0 + r < p.N) wv = to_f(Wm[(size_t)(n0 + r) * p.K + k0 + kk]);
+                if (kin && n0 + r < p.N) wv = to_f(Wm[(size_t)(n0 + r) * p.ldw + k0 + kk]);
                 xs[kk][r] = xv;
                 ws[kk][r] = wv;
             }
@@ -261,16 +256,6 @@ template <int TN> struct DtCfg {
     static constexpr int S = (208 * 1024) / STAGE > 6 ? 6 : (208 * 1024) / STAGE;
     static constexpr size_t SMEM = (size_t)S * STAGE + 1024;
 };
-
-// both operands bf16, K-major, fp32 accumulator, M = 128
-__host__ __device__ constexpr uint32_t dt_idesc(int n) { return tc_idesc(n) | (1u << 7) | (1u << 10); }
-
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst),
-        "l"(map), "r"(x), "r"(y), "r"(bar)
-        : "memory");
-}
 
 template <int TN>
 __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_constant__ CUtensorMap ma,
@@ -415,8 +400,7 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
             int slot, mt, ft;
             locate(tile, slot, mt, ft);
             const DmSlot sl = dm_slot(p, slot);
-            if (!tc_wait(afull + 8 * buf, aph, dead, 113)) break;
-            __syncwarp();
+            if (!tc_wait_warp(afull + 8 * buf, aph, dead, 113)) break;
             tc_fence_after();
             const int r = mt * 128 + q * 32 + lane;
             const bool rin = r < sl.cnt;
@@ -462,33 +446,10 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
 }
 
 // ---- host ---------------------------------------------------------------------------------------------
-typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-static EncodeTiled encode_tiled() {
-    static EncodeTiled fn = [] {
-        void* p = nullptr;
-        cudaDriverEntryPointQueryResult st;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &st) != cudaSuccess ||
-            st != cudaDriverEntryPointSuccess)
-            p = nullptr;
-        return reinterpret_cast<EncodeTiled>(p);
-    }();
-    return fn;
-}
-// (rows, K) bf16 with row stride ld elements; boxes of 64 columns x box_rows, 128-byte swizzle, zeros outside
-static bool make_map(CUtensorMap* m, const void* base, long rows, long K, long ld, int box_rows) {
-    const cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
-    const cuuint32_t box[2] = {64, (cuuint32_t)box_rows}, es[2] = {1, 1};
-    return encode_tiled()(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, es,
-                          CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 template <int TN>
 static int launch_dt(const DmParams& p, const void* xa, long xrows, long ldx, long nmat, long tiles, void* stream) {
     CUtensorMap ma, mb;
-    if (!make_map(&ma, xa, xrows, p.K, ldx, 128) || !make_map(&mb, p.W, nmat * p.N, p.K, p.K, TN)) return GLQ_ERR_UNSUPPORTED;
+    if (!make_map(&ma, xa, xrows, p.K, ldx, 128) || !make_map(&mb, p.W, nmat * p.N, p.K, p.ldw, TN)) return GLQ_ERR_UNSUPPORTED;
     const int grid = (int)std::max<long>(1, std::min<long>(tiles, dn_sms()));
     return dn_launch(dense_tc_kernel<TN>, dim3(grid), kDtThreads, DtCfg<TN>::SMEM, stream, ma, mb, p);
 }
@@ -522,7 +483,7 @@ extern "C" int glq_dense_debug_error(unsigned long long* out4, int clear) {
 static constexpr int kStreamRows = 8;
 
 extern "C" int glq_dense_matmul_path(const glq_dense_mm_t* a) {
-    if (a->dtype != GLQ_DT_BF16 || a->K % 8 || (!a->hn_o && (a->ldx % 8 || !al16(a->x))) || !al16(a->W)) return 0;
+    if (a->dtype != GLQ_DT_BF16 || a->K % 8 || a->ldw % 8 || (!a->hn_o && (a->ldx % 8 || !al16(a->x))) || !al16(a->W)) return 0;
     const int rows = a->slot_index ? a->max_slot_rows : a->rows;
     if (rows <= kStreamRows && a->K <= 12288) return 1;
     if ((a->slot_index && a->max_slots > kDtMaxSlots) || (a->entry_row && !a->gather) || !encode_tiled()) return 0;
@@ -532,6 +493,7 @@ extern "C" int glq_dense_matmul_path(const glq_dense_mm_t* a) {
 extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     if (!a || a->N <= 0 || a->K <= 0 || a->rows < 0 || a->split < 0 || a->split > a->N) return GLQ_ERR_ARG;
     if (a->dtype != GLQ_DT_BF16 && a->dtype != GLQ_DT_F32) return GLQ_ERR_ARG;
+    if (a->ldw && a->ldw < a->K) return GLQ_ERR_ARG;
     if (a->rows == 0) return GLQ_OK;
     const bool grouped = a->slot_index != nullptr;
     if ((!a->x && !a->hn_o) || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
@@ -549,6 +511,7 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     p.slot_offset = a->slot_offset;
     p.entry_row = a->entry_row;
     p.ldx = a->ldx;
+    p.ldw = a->ldw ? a->ldw : a->K;
     p.ldy = a->ldy;
     p.ldy32 = a->ldy32;
     p.N = a->N;

@@ -18,6 +18,7 @@ namespace glq {
 
 constexpr int kSl = 32;            // value columns of a slice
 constexpr int kL = 64;             // positions of a chunk
+constexpr int kSegment = 4096;     // positions the chunk form takes at a time (bounds its workspace)
 
 struct MlParams {
     const void* qkvg;
@@ -261,6 +262,7 @@ __device__ __forceinline__ uint32_t transpose8(uint32_t v) {
 __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
     extern __shared__ __align__(16) unsigned char ml_raw[];
     __shared__ float ws[kL];
+    __shared__ float2 s_tot[kSegment / kL];
     const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, wv = tid >> 7, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.z % p.H, b = blockIdx.z / p.H;
     const int d0 = blockIdx.x * kTd, v0 = blockIdx.y * kTd;
@@ -299,10 +301,9 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
 #pragma unroll
     for (int e = 0; e < 2; ++e) nacc[e] = dr[e] < p.D ? p.n[(slb + v0 / kSl) * p.D + dr[e]] : 0.f;
     float m = p.m0[bh];
-    float2 tot = *reinterpret_cast<const float2*>(p.tot + bh * p.nc * 2);
+    for (int c = tid; c < p.nc; c += 256) s_tot[c] = *reinterpret_cast<const float2*>(p.tot + (bh * p.nc + c) * 2);
     for (int c = 0; c < p.nc; ++c) {
         const size_t bc = bh * p.nc + c;
-        const float2 tot_next = c + 1 < p.nc ? *reinterpret_cast<const float2*>(p.tot + (bc + 1) * 2) : tot;
         cpa_wait<kStStages - 2>();
         __syncthreads();                 // chunk c has landed; nobody still reads the stage that is loaded next
         load(c + kStStages - 1);
@@ -311,11 +312,11 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
         const bf16* vt = kt + kL * kLd;
         const float* ac = reinterpret_cast<const float*>(vt + kL * kLd);
         // the chunk's end: b_L = tot.x, m_L = b_L + max(m, tot.y)
+        const float2 tot = s_tot[c];
         const float m_end = tot.x + fmaxf(m, tot.y), rl = tot.x - m_end, keep = expf(rl + m);
         if (tid < kL) ws[tid] = expf(rl + ac[tid]);
         if (blockIdx.x == 0 && blockIdx.y == 0 && tid == 0) p.min_[bc] = m;
         m = m_end;
-        tot = tot_next;
         // the state this chunk starts from
         uint4* sb = reinterpret_cast<uint4*>(p.Sb) + ((bc * (p.Dp / 16) + d0 / 16 + warp) * (p.Vp / 8) + v0 / 8 + 4 * wv) * 32 + lane;
 #pragma unroll
@@ -572,7 +573,6 @@ using namespace glq;
 extern "C" int glq_mlstm_slices(int V) { return (V + kSl - 1) / kSl; }
 
 static inline size_t up256d(size_t v) { return (v + 255) / 256 * 256; }
-static constexpr int kSegment = 4096;      // positions the chunk form takes at a time (bounds its workspace)
 
 struct MlWs {
     size_t bs, as, cm, tot, m0, min_, nbuf, sb, total;

@@ -31,19 +31,20 @@ def debug_error(clear=True):
     return None if out[0] == 0 else [int(v) for v in out]
 
 
-def matmul(x, W, split=None, act=ACT_NONE, alpha=1.0, ldx=None, rows=None, plan=None, gathered=True):
+def matmul(x, W, split=None, act=ACT_NONE, alpha=1.0, ldx=None, rows=None, plan=None, gathered=True, out=None):
     """alpha * act(x . W^T) with the first ``split`` columns in x's type and the others in float: (y or None, y32 or
     None), each (rows, columns) with a padded row stride.  ``plan`` (``route``): W is (experts, N, K) and every entry
-    goes through its expert's matrix, reading its token's row of x (``gathered``) or its own."""
+    goes through its expert's matrix, reading its token's row of x (``gathered``) or its own.  ``out``: where y goes."""
     _need(x, "x")
     N, K = W.shape[-2], W.shape[-1]
     split = N if split is None else split
     rows = (plan.entries if plan is not None else x.shape[0]) if rows is None else rows
     dev = x.device
-    y = torch.empty(rows, ceil_to(split, 8), dtype=x.dtype, device=dev) if split else None
+    y = out if out is not None else torch.empty(rows, ceil_to(split, 8), dtype=x.dtype, device=dev) if split else None
     y32 = torch.empty(rows, ceil_to(N - split, 4), dtype=torch.float32, device=dev) if split < N else None
     a = _lib.DenseMM(dtype=DTYPES[x.dtype], act=act, N=N, K=K, rows=rows, n_matrices=1, split=split, alpha=alpha,
-                     x=x.data_ptr(), ldx=x.stride(0) if ldx is None else ldx, W=W.data_ptr())
+                     x=x.data_ptr(), ldx=x.stride(0) if ldx is None else ldx, W=W.data_ptr(),
+                     ldw=W.stride(-2))
     if y is not None:
         a.y, a.ldy = y.data_ptr(), y.stride(0)
     if y32 is not None:
@@ -181,8 +182,9 @@ class Latent:
         """Rotates q in place and writes the cache rows: comes before ``prefill``; ``absorbed`` does both by itself."""
         self._call(_lib.dense().glq_latent_prep, "latent_prep")
 
-    def prefill_supported(self):
-        return bool(_lib.dense().glq_latent_prefill_supported(C.byref(self.a)))
+    def prefill_form(self):
+        """0: only ``absorbed`` covers these sizes; 1: ``prefill`` takes keys | values; 2: keys and transposed values."""
+        return _lib.dense().glq_latent_prefill_form(C.byref(self.a))
 
     def absorbed(self, ukt, uv):
         L = _lib.dense()
@@ -191,8 +193,10 @@ class Latent:
         self.a.workspace, self.a.workspace_bytes = ws.data_ptr(), ws.numel()
         self._call(L.glq_latent_absorbed, "latent_absorbed")
 
-    def prefill(self, kv, S):
+    def prefill(self, kv, S, vt=None):
         self.a.kv, self.a.ldkv, self.a.S = kv.data_ptr(), kv.stride(-2), S
+        if vt is not None:
+            self.a.vt, self.a.ldvt = vt.data_ptr(), vt.stride(-2)
         self._call(_lib.dense().glq_latent_prefill, "latent_prefill")
 
 

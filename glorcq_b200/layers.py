@@ -93,24 +93,35 @@ class LatentAttentionMixer(nn.Module):
             self._tables = rotation_tables(self.rot_dims, max_len, self.rot_base, device)
         return self._tables
 
+    def expand(self, state, B, S, form):
+        """Keys and values of positions 0..S-1 as the prompt form of the attention takes them."""
+        n_k, n_v = self.heads * self.dim, self.heads * self.vdim
+
+        def new(rows, cols):
+            return torch.empty(B, rows, dense.ceil_to(cols, 8), dtype=state.rows.dtype, device=state.rows.device)
+        if form == 1:
+            kv = new(S, n_k + n_v)
+            for b in range(B):
+                dense.matmul(state.rows[b], self.w_kv, rows=S, out=kv[b])
+            return kv, S
+        k, vt = new(S, n_k), new(n_v, S)
+        for b in range(B):
+            dense.matmul(state.rows[b], self.w_kv[:n_k], rows=S, out=k[b])
+            dense.matmul(self.uv, state.rows[b, :S, :self.kv_rank], out=vt[b])
+        return k, S, vt
+
     def forward(self, h, B, T, start, kv_len, state):
         q, rest = dense.matmul(h, self.w_in, split=self.split)
         cos, sin = self.tables(state.rows.shape[1], h.device)
         y = torch.empty(B * T, self.heads * self.vdim, dtype=h.dtype, device=h.device)
         call = dense.Latent(q, rest, rest[:, self.kv_rank + self.rot_dim:], start, B, T, self.heads, self.dim, self.rot_dim,
                             self.vdim, self.kv_rank, self.rot_dims, self.scale, self.eps, self.norm_w, cos, sin, state, y)
-        if T <= SHORT_PASS or kv_len is None or not call.prefill_supported():
+        form = 0 if T <= SHORT_PASS or kv_len is None else call.prefill_form()
+        if form == 0:
             call.absorbed(self.ukt, self.uv)
         else:
             call.prep()
-            kv = torch.empty(B, kv_len, self.w_kv.shape[0], dtype=h.dtype, device=h.device) if B > 1 else None
-            for b in range(B):
-                one = dense.matmul(state.rows[b], self.w_kv, rows=kv_len)[0]
-                if kv is None:
-                    kv = one
-                else:
-                    kv[b].copy_(one)
-            call.prefill(kv, kv_len)
+            call.prefill(*self.expand(state, B, kv_len, form))
         return dense.matmul(y, self.w_out, split=0)[1]
 
 

@@ -49,6 +49,7 @@ typedef struct glq_dense_mm {
     const void* x;
     int64_t ldx;
     const void* W;
+    int64_t ldw;           /* row stride of W, 0: K */
     void* y;
     int64_t ldy;
     float* y32;
@@ -134,6 +135,8 @@ typedef struct glq_latent {
     void* out;             /* (B*T, H*V) of dtype */
     const void* kv;
     int64_t ldkv;
+    const void* vt;        /* prefill on tcgen05: values transposed, (B, H*V, ldvt); kv then holds keys only */
+    int64_t ldvt;
     int32_t S;             /* prefill: positions in kv */
     int32_t max_splits;    /* absorbed: upper bound of the position splits */
     void* workspace;
@@ -142,7 +145,8 @@ typedef struct glq_latent {
 int glq_latent_prep(const glq_latent_t* a, void* stream);
 size_t glq_latent_absorbed_workspace_bytes(const glq_latent_t* a);
 int glq_latent_absorbed(const glq_latent_t* a, void* stream);
-int glq_latent_prefill_supported(const glq_latent_t* a);
+/* 0: not covered, 1: mma form (kv = keys | values), 2: tcgen05 form (kv = keys, vt = values transposed) */
+int glq_latent_prefill_form(const glq_latent_t* a);
 int glq_latent_prefill(const glq_latent_t* a, void* stream);
 
 /* Routing: s = softmax(logits) over E experts and `identity` pass-through experts, the `top` largest of
