@@ -37,8 +37,8 @@ struct MlParams {
     int t0, Tall;                  // this call's positions: t0 .. t0 + T - 1 of the Tall rows of a sequence
     float cap, eps, scale;
     // chunk form
-    float *bs, *as, *cm, *tot, *m0, *min_, *nbuf;
-    uint32_t* Sb;
+    float *bs, *as, *cm, *tot, *m0, *min_, *nbuf, *ksum;
+    uint32_t *Sb, *Kb;
     int nc, Dp, Vp;
 };
 
@@ -202,50 +202,99 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const MlParams p) {
 }
 
 // ---- chunk form ------------------------------------------------------------------------------------------
-// gates of the chunks, one warp each: running sum of f (bs), i - bs (as) and its running maximum (cm) for every position,
-// sum and maximum of the chunk (tot); positions past T weigh nothing
-__global__ void __launch_bounds__(128) mlstm_gate_kernel(const MlParams p) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int c = blockIdx.x * 4 + warp, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
-    const size_t bh = blockIdx.y;
+// Per chunk and head, one CTA.  Gates: running sum of f (bs), i - bs (as) and its running maximum (cm) for every position,
+// sum and maximum of the chunk (tot); positions past T weigh nothing.  Keys: k e^(as - maximum) as the left operand of the
+// state's products, [d / 16][16 positions][part][lane] of uint4 (part: the two bf16 parts), and their sum over the chunk.
+constexpr int kGd = 128;                 // keys of 128 channels at a time: warp = 16 of them
+__global__ void __launch_bounds__(256) mlstm_gate_kernel(const MlParams p) {
+    __shared__ __align__(16) bf16 ks[kL * (kGd + 8)];
+    __shared__ float ws[kL];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, t4 = lane & 3;
+    const int c = blockIdx.x, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
+    const size_t bh = blockIdx.y, bc = bh * p.nc + c;
+    const bf16* kb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)p.H * p.D + (size_t)h * p.D;
     pdl_wait();
     pdl_release();
-    if (c >= p.nc) return;
-    // the maximum the sequence starts from, before the state kernel replaces it
-    if (c == 0 && lane == 0) p.m0[bh] = p.m[bh * p.slices];
-    float f[2], li[2];
+    auto load = [&](int d0) {
+        for (int i = tid; i < kL * (kGd / 8); i += 256) {
+            const int s = i / (kGd / 8), cc = (i % (kGd / 8)) * 8, tt = c * kL + s;
+            const bool live = tt < p.T && d0 + cc < p.D;
+            cpa16(smem_u32(ks + s * (kGd + 8) + cc), live ? kb + ((size_t)b * p.Tall + p.t0 + tt) * p.ldp + d0 + cc : kb, live);
+        }
+        cpa_commit();
+    };
+    load(0);
+    if (warp == 0) {
+        // the maximum the sequence starts from, before the state kernel replaces it
+        if (c == 0 && lane == 0) p.m0[bh] = p.m[bh * p.slices];
+        float f[2], li[2];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-        const int t = c * kL + 2 * lane + e;
-        const size_t row = (size_t)b * p.Tall + p.t0 + t;
-        f[e] = t < p.T ? log_f(p, row, h) : 0.f;
-        li[e] = t < p.T ? log_i(p, row, h) : -INFINITY;
-    }
-    float sum = f[0] + f[1];
+        for (int e = 0; e < 2; ++e) {
+            const int t = c * kL + 2 * lane + e;
+            const size_t row = (size_t)b * p.Tall + p.t0 + t;
+            f[e] = t < p.T ? log_f(p, row, h) : 0.f;
+            li[e] = t < p.T ? log_i(p, row, h) : -INFINITY;
+        }
+        float sum = f[0] + f[1];
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-        const float u = __shfl_up_sync(0xffffffffu, sum, o);
-        if (lane >= o) sum += u;
-    }
-    const float b1 = sum, b0 = sum - f[1];
-    const float a0 = li[0] - b0, a1 = li[1] - b1;
-    float mx = fmaxf(a0, a1);
+        for (int o = 1; o < 32; o <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += u;
+        }
+        const float b1 = sum, b0 = sum - f[1];
+        const float a0 = li[0] - b0, a1 = li[1] - b1;
+        float mx = fmaxf(a0, a1);
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-        const float u = __shfl_up_sync(0xffffffffu, mx, o);
-        if (lane >= o) mx = fmaxf(mx, u);
+        for (int o = 1; o < 32; o <<= 1) {
+            const float u = __shfl_up_sync(0xffffffffu, mx, o);
+            if (lane >= o) mx = fmaxf(mx, u);
+        }
+        const float prev = __shfl_up_sync(0xffffffffu, mx, 1), top = __shfl_sync(0xffffffffu, mx, 31);
+        const size_t i = bc * kL + 2 * lane;
+        *reinterpret_cast<float2*>(p.bs + i) = make_float2(b0, b1);
+        *reinterpret_cast<float2*>(p.as + i) = make_float2(a0, a1);
+        *reinterpret_cast<float2*>(p.cm + i) = make_float2(lane ? fmaxf(prev, a0) : a0, mx);
+        if (lane == 31) *reinterpret_cast<float2*>(p.tot + bc * 2) = make_float2(b1, mx);
+        ws[2 * lane] = expf(a0 - top);
+        ws[2 * lane + 1] = expf(a1 - top);
     }
-    const float prev = __shfl_up_sync(0xffffffffu, mx, 1);
-    const size_t i = (bh * p.nc + c) * kL + 2 * lane;
-    *reinterpret_cast<float2*>(p.bs + i) = make_float2(b0, b1);
-    *reinterpret_cast<float2*>(p.as + i) = make_float2(a0, a1);
-    *reinterpret_cast<float2*>(p.cm + i) = make_float2(lane ? fmaxf(prev, a0) : a0, mx);
-    if (lane == 31) *reinterpret_cast<float2*>(p.tot + (bh * p.nc + c) * 2) = make_float2(b1, mx);
+    for (int d0 = 0; d0 < p.Dp; d0 += kGd) {
+        cpa_wait<0>();
+        __syncthreads();
+        if (d0 + 16 * warp < p.Dp) {
+            uint4* dst = reinterpret_cast<uint4*>(p.Kb) + (bc * (p.Dp / 16) + d0 / 16 + warp) * 256 + lane;
+            float ns[2] = {0.f, 0.f};
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                uint32_t a[4], hi[4], lo[4];
+                ldsm4_t(smem_u32(ks + (16 * kk + (lane >> 4) * 8 + (lane & 7)) * (kGd + 8) + 16 * warp + ((lane >> 3) & 1) * 8), a[0], a[1],
+                        a[2], a[3]);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int s = 16 * kk + 2 * t4 + 8 * (i >> 1);
+                    const float x = bf_lo(a[i]) * ws[s], y = bf_hi(a[i]) * ws[s + 1];
+                    ns[i & 1] += x + y;
+                    split_bf2(x, y, hi[i], lo[i]);
+                }
+                dst[kk * 64] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                dst[kk * 64 + 32] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 1);
+                ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 2);
+                if (t4 == 0) p.ksum[bc * p.Dp + d0 + 16 * warp + (lane >> 2) + 8 * e] = ns[e];
+            }
+        }
+        __syncthreads();
+        if (d0 + kGd < p.Dp) load(d0 + kGd);
+    }
 }
 
 constexpr int kTd = 64, kLd = 72;        // tile width, row stride of a 64-wide shared-memory tile (bf16)
+constexpr int kKb = 4 * 4 * 64 * 16;     // bytes of a chunk's key operand for 64 channels
 constexpr int kStStages = 4;
-constexpr int kStStage = 2 * kL * kLd * 2 + kL * 4;      // bytes: keys, values, i - bs
+constexpr int kStStage = kKb + kL * kLd * 2 + kTd * 4;   // bytes: key operand, values, key sums
 
 // 8x8 block of 16-bit values held row-wise across a warp -> column-wise
 __device__ __forceinline__ uint32_t transpose8(uint32_t v) {
@@ -261,27 +310,25 @@ __device__ __forceinline__ uint32_t transpose8(uint32_t v) {
 // head's S: warp = 16 rows x 32 columns
 __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
     extern __shared__ __align__(16) unsigned char ml_raw[];
-    __shared__ float ws[kL];
     __shared__ float2 s_tot[kSegment / kL];
     const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, wv = tid >> 7, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.z % p.H, b = blockIdx.z / p.H;
     const int d0 = blockIdx.x * kTd, v0 = blockIdx.y * kTd;
     const size_t bh = blockIdx.z;
-    const bf16* kb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)p.H * p.D + (size_t)h * p.D;
     const bf16* vb = reinterpret_cast<const bf16*>(p.qkvg) + (size_t)2 * p.H * p.D + (size_t)h * p.V;
     auto load = [&](int c) {
-        unsigned char* st = ml_raw + (size_t)(c % kStStages) * kStStage;
         if (c < p.nc) {
-            bf16* ks = reinterpret_cast<bf16*>(st);
-            bf16* vs = ks + kL * kLd;
-            for (int i = tid; i < kL * 8; i += 256) {
-                const int s = i >> 3, cc = (i & 7) * 8, tt = c * kL + s;
-                const size_t row = ((size_t)b * p.Tall + p.t0 + (tt < p.T ? tt : 0)) * p.ldp;
-                const bool kl = tt < p.T && d0 + cc < p.D, vl = tt < p.T && v0 + cc < p.V;
-                cpa16(smem_u32(ks + s * kLd + cc), kl ? kb + row + d0 + cc : kb, kl);
-                cpa16(smem_u32(vs + s * kLd + cc), vl ? vb + row + v0 + cc : vb, vl);
+            const uint32_t st = smem_u32(ml_raw) + (uint32_t)(c % kStStages) * kStStage;
+            const unsigned char* ka = reinterpret_cast<const unsigned char*>(p.Kb) + ((bh * p.nc + c) * (p.Dp / 16) + d0 / 16) * 4096;
+#pragma unroll
+            for (int i = 0; i < kKb / 16 / 256; ++i) cpa16(st + 16 * (tid + 256 * i), ka + 16 * (tid + 256 * i), true);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int s = (tid >> 3) + 32 * i, cc = (tid & 7) * 8, tt = c * kL + s;
+                const bool vl = tt < p.T && v0 + cc < p.V;
+                cpa16(st + kKb + (s * kLd + cc) * 2, vl ? vb + ((size_t)b * p.Tall + p.t0 + tt) * p.ldp + v0 + cc : vb, vl);
             }
-            if (tid < kL / 4) cpa16(smem_u32(vs + kL * kLd) + 16 * tid, p.as + (bh * p.nc + c) * kL + 4 * tid, true);
+            if (tid < kTd / 4) cpa16(st + kKb + kL * kLd * 2 + 16 * tid, p.ksum + (bh * p.nc + c) * p.Dp + d0 + 4 * tid, true);
         }
         cpa_commit();
     };
@@ -308,15 +355,34 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
         __syncthreads();                 // chunk c has landed; nobody still reads the stage that is loaded next
         load(c + kStStages - 1);
         const unsigned char* st = ml_raw + (size_t)(c % kStStages) * kStStage;
-        const bf16* kt = reinterpret_cast<const bf16*>(st);
-        const bf16* vt = kt + kL * kLd;
-        const float* ac = reinterpret_cast<const float*>(vt + kL * kLd);
-        // the chunk's end: b_L = tot.x, m_L = b_L + max(m, tot.y)
+        const uint32_t ka = smem_u32(st) + (uint32_t)(warp * 256 + lane) * 16, va = smem_u32(st) + kKb;
+        const float* ksum = reinterpret_cast<const float*>(st + kKb + kL * kLd * 2);
+        // the chunk's end: b_L = tot.x, m_L = b_L + max(m, tot.y); keys carry e^(as - tot.y)
         const float2 tot = s_tot[c];
-        const float m_end = tot.x + fmaxf(m, tot.y), rl = tot.x - m_end, keep = expf(rl + m);
-        if (tid < kL) ws[tid] = expf(rl + ac[tid]);
+        const float m_end = tot.x + fmaxf(m, tot.y), rl = tot.x - m_end, keep = expf(rl + m), fac = expf(rl + tot.y);
         if (blockIdx.x == 0 && blockIdx.y == 0 && tid == 0) p.min_[bc] = m;
         m = m_end;
+        float add[2][4][4];
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) add[u][j][e] = 0.f;
+#pragma unroll
+        for (int kk = 0; kk < 4; ++kk) {
+            const uint4 hi = lds128(ka + kk * 1024), lo = lds128(ka + kk * 1024 + 512);
+            uint32_t vf[2][4];
+#pragma unroll
+            for (int jp = 0; jp < 2; ++jp)
+                ldsm4_t(va + ((16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 32 * wv + 16 * jp + (lane >> 4) * 8) * 2, vf[jp][0], vf[jp][1],
+                        vf[jp][2], vf[jp][3]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                mma_bf16(add[0][j], hi.x, hi.y, hi.z, hi.w, vf[j >> 1][2 * (j & 1)], vf[j >> 1][2 * (j & 1) + 1]);
+                mma_bf16(add[1][j], lo.x, lo.y, lo.z, lo.w, vf[j >> 1][2 * (j & 1)], vf[j >> 1][2 * (j & 1) + 1]);
+            }
+        }
         // the state this chunk starts from
         uint4* sb = reinterpret_cast<uint4*>(p.Sb) + ((bc * (p.Dp / 16) + d0 / 16 + warp) * (p.Vp / 8) + v0 / 8 + 4 * wv) * 32 + lane;
 #pragma unroll
@@ -330,39 +396,12 @@ __global__ void __launch_bounds__(256) mlstm_state_kernel(const MlParams p) {
             p.nbuf[bc * p.Dp + dr[0]] = nacc[0];
             p.nbuf[bc * p.Dp + dr[1]] = nacc[1];
         }
-        __syncthreads();
 #pragma unroll
         for (int j = 0; j < 4; ++j)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) acc[j][e] *= keep;
-        float ns[2] = {0.f, 0.f};
+            for (int e = 0; e < 4; ++e) acc[j][e] = keep * acc[j][e] + fac * (add[0][j][e] + add[1][j][e]);
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
-            uint32_t a[4], hi[4], lo[4];
-            ldsm4_t(smem_u32(kt + (16 * kk + (lane >> 4) * 8 + (lane & 7)) * kLd + 16 * warp + ((lane >> 3) & 1) * 8), a[0], a[1], a[2], a[3]);
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int s = 16 * kk + 2 * t + 8 * (i >> 1);
-                const float x = bf_lo(a[i]) * ws[s], y = bf_hi(a[i]) * ws[s + 1];
-                ns[i & 1] += x + y;
-                split_bf2(x, y, hi[i], lo[i]);
-            }
-            uint32_t vb_[2][4];
-#pragma unroll
-            for (int jp = 0; jp < 2; ++jp)
-                ldsm4_t(smem_u32(vt + (16 * kk + (lane & 7) + ((lane >> 3) & 1) * 8) * kLd + 32 * wv + 16 * jp + (lane >> 4) * 8), vb_[jp][0],
-                        vb_[jp][1], vb_[jp][2], vb_[jp][3]);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) mma_bf16(acc[j], hi[0], hi[1], hi[2], hi[3], vb_[j >> 1][2 * (j & 1)], vb_[j >> 1][2 * (j & 1) + 1]);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) mma_bf16(acc[j], lo[0], lo[1], lo[2], lo[3], vb_[j >> 1][2 * (j & 1)], vb_[j >> 1][2 * (j & 1) + 1]);
-        }
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 1);
-            ns[e] += __shfl_xor_sync(0xffffffffu, ns[e], 2);
-            nacc[e] = keep * nacc[e] + ns[e];
-        }
+        for (int e = 0; e < 2; ++e) nacc[e] = keep * nacc[e] + fac * ksum[16 * warp + g + 8 * e];
     }
     cpa_wait<0>();
 #pragma unroll
@@ -575,7 +614,7 @@ extern "C" int glq_mlstm_slices(int V) { return (V + kSl - 1) / kSl; }
 static inline size_t up256d(size_t v) { return (v + 255) / 256 * 256; }
 
 struct MlWs {
-    size_t bs, as, cm, tot, m0, min_, nbuf, sb, total;
+    size_t bs, as, cm, tot, m0, min_, nbuf, ksum, sb, kb, total;
 };
 static MlWs ml_ws(const glq_mlstm_t* a) {
     MlWs w{};
@@ -593,7 +632,9 @@ static MlWs ml_ws(const glq_mlstm_t* a) {
     w.m0 = take(bh * 4);
     w.min_ = take(bh * nc * 4);
     w.nbuf = take(bh * nc * Dp * 4);
+    w.ksum = take(bh * nc * Dp * 4);
     w.sb = take(bh * nc * Dp * Vp * 4);
+    w.kb = take(bh * nc * Dp * kL * 4);
     w.total = at;
     return w;
 }
@@ -667,14 +708,16 @@ extern "C" int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream) {
     p.m0 = reinterpret_cast<float*>(ws + w.m0);
     p.min_ = reinterpret_cast<float*>(ws + w.min_);
     p.nbuf = reinterpret_cast<float*>(ws + w.nbuf);
+    p.ksum = reinterpret_cast<float*>(ws + w.ksum);
     p.Sb = reinterpret_cast<uint32_t*>(ws + w.sb);
+    p.Kb = reinterpret_cast<uint32_t*>(ws + w.kb);
     p.Dp = (a->D + 63) / 64 * 64;
     p.Vp = (a->V + 63) / 64 * 64;
     const int bh = p.B * p.H;
     for (p.t0 = 0; p.t0 < p.Tall; p.t0 += kSegment) {
         p.T = std::min(kSegment, p.Tall - p.t0);
         p.nc = cdiv_i(p.T, kL);
-        if ((st = dn_launch(mlstm_gate_kernel, dim3(cdiv_i(p.nc, 4), bh), 128, 0, stream, p)) != GLQ_OK) return st;
+        if ((st = dn_launch(mlstm_gate_kernel, dim3(p.nc, bh), 256, 0, stream, p)) != GLQ_OK) return st;
         if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 256, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
         if (p.V > 64) st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, MoCfg<128>::SMEM, stream, p);
         else st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, MoCfg<64>::SMEM, stream, p);
