@@ -329,6 +329,8 @@ extern "C" int glq_dense_add_norm(int dtype, const float* y, const float* w, con
         const bool vec = C % 8 == 0 && al16(y) && al16(w) && al16(x) && al16(h) && al16(final_w);
         if (vec && C <= 8 * kRowThreads)
             return dn_launch(dense_add_norm_kernel<T, 1>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
+        if (vec && C <= 16 * kRowThreads)
+            return dn_launch(dense_add_norm_kernel<T, 2>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
         if (vec && C <= 32 * kRowThreads)
             return dn_launch(dense_add_norm_kernel<T, 4>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
         return dn_launch(dense_add_norm_kernel<T, 0>, dim3(rows), kRowThreads, (size_t)C * 4, stream, y, w, final_w, eps, C, x, (T*)h);
@@ -349,6 +351,7 @@ extern "C" int glq_dense_combine_norm(int dtype, const void* entry_out, int64_t 
                              final_w, eps, C, x, (T*)h);
         };
         if (vec && C <= 8 * kRowThreads) return go(dense_combine_norm_kernel<T, 1>, 0);
+        if (vec && C <= 16 * kRowThreads) return go(dense_combine_norm_kernel<T, 2>, 0);
         if (vec && C <= 32 * kRowThreads) return go(dense_combine_norm_kernel<T, 4>, 0);
         return go(dense_combine_norm_kernel<T, 0>, (size_t)C * 4);
     });

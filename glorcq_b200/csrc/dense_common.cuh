@@ -111,8 +111,9 @@ inline int dn_sms() {
 
 // Launch that may start while its predecessor drains: every kernel here calls pdl_wait() before it touches anything a
 // predecessor wrote.
+// (early = false: an ordinary launch, for a kernel whose waiting CTAs would only take room from its predecessor)
 template <typename... KArgs, typename... Args>
-inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+inline int dn_launch_if(bool early, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
     static const bool pdl = std::getenv("GLQ_NO_PDL") == nullptr;
     if (smem > 48 * 1024) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     cudaLaunchConfig_t cfg{};
@@ -124,9 +125,13 @@ inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, 
     attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
-    cfg.numAttrs = pdl ? 1 : 0;
+    cfg.numAttrs = pdl && early ? 1 : 0;
     DN_CUDA(cudaLaunchKernelEx(&cfg, kern, KArgs(args)...));
     return GLQ_OK;
+}
+template <typename... KArgs, typename... Args>
+inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+    return dn_launch_if(true, kern, grid, block, smem, stream, args...);
 }
 
 }  // namespace glq

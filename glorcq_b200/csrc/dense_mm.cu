@@ -26,6 +26,7 @@ struct DmParams {
     int N, K, rows, slots, split, act;
     float alpha;
     int vec_y, vec_y32;
+    int xrows;                       // streaming kernel: activation rows staged, one of zeros behind fewer than eight
     const float* hn_o;               // streaming kernel: rows made from a recurrence's output (see glq_dense_mm_t)
     const void* hn_g;
     const float* hn_w;
@@ -70,7 +71,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
     const int c_lo = (int)((long)s * chunks / SPLIT), c_hi = (int)((long)(s + 1) * chunks / SPLIT);
     const int XS = (chunks + 1) * 32;                              // padded activation rows: distinct banks
     bf16* xs = reinterpret_cast<bf16*>(dm_smem);
-    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)8 * XS * 2);
+    float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)p.xrows * XS * 2);
     const int ntiles = (p.N + 15) / 16;
     const bool plain = p.slot_index == nullptr;
     DmSlot sl{0, 0, p.rows};
@@ -105,7 +106,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
             if (p.hn_o) {
                 // rows = per-head RMS norm of hn_o, times its weight, times the sigmoid of the gate; warp = (row, head)
                 const int V = K / p.hn_heads;
-                for (int i = w; i < 8 * p.hn_heads; i += WARPS) {
+                for (int i = w; i < p.xrows * p.hn_heads; i += WARPS) {
                     const int row = i / p.hn_heads, k0 = (i % p.hn_heads) * V;
                     if (row >= sl.cnt) {
                         for (int k = k0 + lane; k < k0 + V; k += 32) xs[(size_t)row * XS + k] = from_f<bf16>(0.f);
@@ -128,12 +129,12 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                     for (int k = k0 + lane; k < k0 + V; k += 32)
                         xs[(size_t)row * XS + k] = from_f<bf16>(o[k] * inv * p.hn_w[k] * sigmoid_f(to_f(gt[k])));
                 }
-                for (int i = tid; i < 8 * 32; i += THREADS) {        // channels past K of the last chunk
+                for (int i = tid; i < p.xrows * 32; i += THREADS) {  // channels past K of the last chunk
                     const int k = K + (i & 31);
                     if (k < chunks * 32) xs[(size_t)(i >> 5) * XS + k] = from_f<bf16>(0.f);
                 }
             } else {
-                for (int i = tid; i < 8 * chunks * 4; i += THREADS) {
+                for (int i = tid; i < p.xrows * chunks * 4; i += THREADS) {
                     const int row = i / (chunks * 4), c = i % (chunks * 4), k = c * 8;
                     uint4 v = make_uint4(0, 0, 0, 0);
                     if (row < sl.cnt && k < K) {
@@ -147,7 +148,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
             __syncthreads();
         }
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
-        const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)g * XS) + t;
+        const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)min(g, p.xrows - 1) * XS) + t;   // past the rows: zeros
         for (int c0 = c_lo; c0 < c_hi; c0 += DEPTH) {
 #pragma unroll
             for (int d = 0; d < DEPTH; ++d) {
@@ -481,11 +482,13 @@ extern "C" int glq_dense_debug_error(unsigned long long* out4, int clear) {
 
 // rows per problem up to which the streaming kernel runs (weights are read once per 8 rows)
 static constexpr int kStreamRows = 8;
+static size_t stream_row_bytes(int K) { return (size_t)(cdiv_i(K, 32) + 1) * 64; }
+static int stream_rows(const glq_dense_mm_t* a) { return std::min(8, (a->slot_index ? a->max_slot_rows : a->rows) + 1); }
 
 extern "C" int glq_dense_matmul_path(const glq_dense_mm_t* a) {
     if (a->dtype != GLQ_DT_BF16 || a->K % 8 || a->ldw % 8 || (!a->hn_o && (a->ldx % 8 || !al16(a->x))) || !al16(a->W)) return 0;
     const int rows = a->slot_index ? a->max_slot_rows : a->rows;
-    if (rows <= kStreamRows && a->K <= 12288) return 1;
+    if (rows <= kStreamRows && stream_row_bytes(a->K) * stream_rows(a) <= 200 * 1024) return 1;
     if ((a->slot_index && a->max_slots > kDtMaxSlots) || (a->entry_row && !a->gather) || !encode_tiled()) return 0;
     return 2;
 }
@@ -536,15 +539,16 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     const int rows_max = grouped ? a->max_slot_rows : a->rows;
     if (path == 1) {
         const int tiles = cdiv_i(a->N, 16), sms = dn_sms();
+        p.xrows = stream_rows(a);
         auto go = [&](auto kern, int warps, int grid) {
-            const size_t smem = (size_t)8 * (cdiv_i(a->K, 32) + 1) * 32 * 2 + (size_t)warps * 32 * sizeof(float4);
+            const size_t smem = stream_row_bytes(a->K) * p.xrows + (size_t)warps * 32 * sizeof(float4);
             return dn_launch(kern, dim3(grid, p.slots), warps * 32, smem, stream, p);
         };
         // measured on 1 x N x K products of 6 to 25 MB: many tiles walk over resident CTAs; a few per SM fit one wave of
         // small CTAs; less than one per SM takes deep loads, with sixteen warps on a tile when rows are long
         const long work = (long)tiles * p.slots;
         if (work > 12L * sms) return go(dense_stream_kernel<8, 4, 8, 2>, 8, std::min(cdiv_i(tiles, 2), 2 * sms));
-        if (work > 3L * sms) return go(dense_stream_kernel<4, 4, 8, 4>, 4, tiles);
+        if (work > 3L * sms && a->K < 4096) return go(dense_stream_kernel<4, 4, 8, 4>, 4, tiles);
         if (work > sms) return go(dense_stream_kernel<8, 8, 4, 3>, 8, tiles);
         if (a->K >= 4096) return go(dense_stream_kernel<16, 16, 8, 1>, 16, tiles);
         return go(dense_stream_kernel<8, 8, 8, 2>, 8, tiles);

@@ -197,6 +197,16 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LaParams p) {
 }
 
 constexpr int kMaxSplits = 128;
+constexpr int kAbPos = 32;       // positions per stage of the absorbed form
+
+// stages of split z for `total` positions, and how many splits have any
+struct SplitRange {
+    int lo, hi, used;
+};
+__device__ __forceinline__ SplitRange split_range(const LaParams& p, int z, int total) {
+    const int ntile = (total + kAbPos - 1) / kAbPos, per = (ntile + p.splits - 1) / p.splits;
+    return {z * per, min(ntile, (z + 1) * per), (ntile + per - 1) / per};
+}
 
 // weighted latent of a (row, head): the splits' sums combined; grid (rows, heads, column parts)
 __global__ void __launch_bounds__(512) latent_combine_kernel(const LaParams p) {
@@ -205,6 +215,8 @@ __global__ void __launch_bounds__(512) latent_combine_kernel(const LaParams p) {
     pdl_release();
     const int row = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
     const int rr = (row % p.T) * p.H + h;
+    // splits behind the last position left their sums unwritten
+    const int used = p.splits > 1 ? split_range(p, 0, (int)min((long long)p.max_len, *p.start + p.T)).used : 1;
     const size_t first = (((size_t)(row / p.T) * (p.rows16 / 16) + rr / 16) * p.splits) * 16 + rr % 16;     // split z: + 16 z
     if (threadIdx.x < 32) {
         float mz[kMaxSplits / 32], lz[kMaxSplits / 32], m = -INFINITY;
@@ -230,7 +242,7 @@ __global__ void __launch_bounds__(512) latent_combine_kernel(const LaParams p) {
     __syncthreads();
     // 128 columns at a time, four groups of threads over the splits
     const int per = (p.K + gridDim.z - 1) / gridDim.z, k_hi = min(p.K, (int)(blockIdx.z + 1) * per);
-    const int zq = (p.splits + 3) / 4, grp = threadIdx.x >> 7, z0 = grp * zq, z1 = min(p.splits, z0 + zq);
+    const int zq = (used + 3) / 4, grp = threadIdx.x >> 7, z0 = grp * zq, z1 = min(used, z0 + zq);
     for (int kb = blockIdx.z * per; kb < k_hi; kb += 128) {
         const int k = kb + (threadIdx.x & 127);
         float v = 0.f;
@@ -238,9 +250,7 @@ __global__ void __launch_bounds__(512) latent_combine_kernel(const LaParams p) {
             const float* po = p.po + first * p.K + k;
 #pragma unroll 16
             for (int z = z0; z < z1; ++z) {
-                // a split without a visible position left its sums unwritten
-                const float w = sw[z], x = w != 0.f ? po[(size_t)16 * z * p.K] : 0.f;
-                v += w * x;
+                v += sw[z] * po[(size_t)16 * z * p.K];
             }
         }
         part[grp][threadIdx.x & 127] = v;
@@ -279,7 +289,6 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LaParams p) {
 }
 
 // ---- attention over the cached latents, tensor cores ----------------------------------------------------
-constexpr int kAbPos = 32;       // positions per stage
 
 // 16 rows (query position, head) against one split of the positions; NT: 8-column tiles of the latent per warp
 template <int NT>
@@ -299,8 +308,8 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
     pdl_release();
     const long long start = *p.start;
     const int total = (int)min((long long)p.max_len, start + p.T);
-    const int ntile = (total + kAbPos - 1) / kAbPos, per = (ntile + p.splits - 1) / p.splits;
-    const int c_lo = z * per, c_hi = min(ntile, c_lo + per);
+    const SplitRange sr = split_range(p, z, total);
+    const int c_lo = sr.lo, c_hi = sr.hi;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.max_len * p.ldc;
     auto load = [&](int c, int buf) {
         const int vec = KRp / 8;
@@ -311,18 +320,18 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
         }
         cpa_commit();
     };
-    if (c_lo < c_hi) load(c_lo, 0);
-    {
+    if (c_lo < c_hi) {      // the queries' copies join the first stage's group
         const bf16* src = reinterpret_cast<const bf16*>(p.qa) + ((size_t)b * p.rows16 + rt * 16) * KRp;
         const size_t plane = (size_t)p.B * p.rows16 * KRp;
         const int vec = KRp / 8;
         for (int i = tid; i < 16 * vec; i += 256) {
             const int r = i / vec, cc = (i % vec) * 8;
             const bool live = rt * 16 + r < p.T * p.H;
-            const uint4 zero = make_uint4(0, 0, 0, 0);
-            *reinterpret_cast<uint4*>(qh + r * LD + cc) = live ? *reinterpret_cast<const uint4*>(src + (size_t)r * KRp + cc) : zero;
-            *reinterpret_cast<uint4*>(ql + r * LD + cc) = live ? *reinterpret_cast<const uint4*>(src + plane + (size_t)r * KRp + cc) : zero;
+            const bf16* q = live ? src + (size_t)r * KRp + cc : src;
+            cpa16(smem_u32(qh + r * LD + cc), q, live);
+            cpa16(smem_u32(ql + r * LD + cc), q + plane, live);
         }
+        load(c_lo, 0);
     }
     if (tid < 16) {
         s_m[tid] = -INFINITY;

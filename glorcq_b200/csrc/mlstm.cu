@@ -72,9 +72,11 @@ __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, in
     float ss = 0.f;
     if (p.V % 4 == 0 && p.V <= 1024 && p.vec4) {          // four values per lane and step, kept in registers
         float4 x[8];
+        float gv[8][4];                          // requested together with the row, ahead of its sum
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
             const int v = (u * 32 + lane) * 4;
+            if (v < p.V) ld4(g + v, gv[u]);
             x[u] = v < p.V ? *reinterpret_cast<const float4*>(o + v) : make_float4(0, 0, 0, 0);
             ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
         }
@@ -84,11 +86,9 @@ __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, in
         for (int u = 0; u < 8; ++u) {
             const int v = (u * 32 + lane) * 4;
             if (v < p.V) {
-                float gv[4];
-                ld4(g + v, gv);
                 const float4 wv = *reinterpret_cast<const float4*>(w + v);
-                st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[0]), x[u].y * inv * wv.y * sigmoid_f(gv[1]),
-                    x[u].z * inv * wv.z * sigmoid_f(gv[2]), x[u].w * inv * wv.w * sigmoid_f(gv[3]));
+                st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[u][0]), x[u].y * inv * wv.y * sigmoid_f(gv[u][1]),
+                    x[u].z * inv * wv.z * sigmoid_f(gv[u][2]), x[u].w * inv * wv.w * sigmoid_f(gv[u][3]));
             }
         }
         return;
@@ -718,9 +718,9 @@ extern "C" int glq_mlstm_chunk(const glq_mlstm_t* a, void* stream) {
         p.T = std::min(kSegment, p.Tall - p.t0);
         p.nc = cdiv_i(p.T, kL);
         if ((st = dn_launch(mlstm_gate_kernel, dim3(p.nc, bh), 256, 0, stream, p)) != GLQ_OK) return st;
-        if ((st = dn_launch(mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 256, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
-        if (p.V > 64) st = dn_launch(mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, MoCfg<128>::SMEM, stream, p);
-        else st = dn_launch(mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, MoCfg<64>::SMEM, stream, p);
+        if ((st = dn_launch_if(false, mlstm_state_kernel, dim3(p.Dp / 64, p.Vp / 64, bh), 256, (size_t)kStStages * kStStage, stream, p)) != GLQ_OK) return st;
+        if (p.V > 64) st = dn_launch_if(false, mlstm_out_kernel<128>, dim3(cdiv_i(p.V, 128), p.nc, bh), 128, MoCfg<128>::SMEM, stream, p);
+        else st = dn_launch_if(false, mlstm_out_kernel<64>, dim3(1, p.nc, bh), 128, MoCfg<64>::SMEM, stream, p);
         if (st != GLQ_OK) return st;
         if ((st = ml_norm(p, a->dtype, stream)) != GLQ_OK) return st;
     }

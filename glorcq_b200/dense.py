@@ -146,7 +146,7 @@ def mlstm(qkvg, gates, B, T, heads, dim, vdim, cap, eps, bias_i, bias_f, norm_w,
 
 
 def head_norm_matmul_supported(o, W):
-    return W.dtype == torch.bfloat16 and o.shape[0] <= 8 and W.shape[1] % 8 == 0 and W.shape[1] <= 12288
+    return W.dtype == torch.bfloat16 and o.shape[0] <= 8 and W.shape[1] % 8 == 0 and min(8, o.shape[0] + 1) * (W.shape[1] + 64) * 2 <= 200 * 1024
 
 
 def head_norm_matmul(o, gate, norm_w, heads, eps, W):
