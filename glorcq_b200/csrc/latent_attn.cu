@@ -197,7 +197,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const LaParams p) {
 }
 
 constexpr int kMaxSplits = 128;
-constexpr int kAbPos = 32;       // positions per stage of the absorbed form
+constexpr int kAbPos = 64;       // positions per stage of the absorbed form
 
 // stages of split z for `total` positions, and how many splits have any
 struct SplitRange {
@@ -311,12 +311,13 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
     const SplitRange sr = split_range(p, z, total);
     const int c_lo = sr.lo, c_hi = sr.hi;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.max_len * p.ldc;
-    auto load = [&](int c, int buf) {
-        const int vec = KRp / 8;
-        for (int i = tid; i < kAbPos * vec; i += 256) {
-            const int r = i / vec, cc = (i % vec) * 8, pos = c * kAbPos + r;
-            const bool live = pos < total && cc < KR;
-            cpa16(smem_u32(cs + ((size_t)buf * kAbPos + r) * LD + cc), live ? cache + (size_t)pos * p.ldc + cc : cache, live);
+    auto load = [&](int c, int buf) {        // warp = rows warp, warp + 8, ..
+        const uint32_t dst = smem_u32(cs + (size_t)buf * kAbPos * LD);
+#pragma unroll 4
+        for (int r = warp; r < kAbPos; r += 8) {
+            const int pos = c * kAbPos + r;
+            const bf16* src = cache + (size_t)(pos < total ? pos : 0) * p.ldc;
+            for (int cc = 8 * lane; cc < KRp; cc += 256) cpa16(dst + (r * LD + cc) * 2, cc < KR ? src + cc : src, pos < total && cc < KR);
         }
         cpa_commit();
     };
@@ -352,45 +353,59 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
         }
         __syncthreads();
         const bf16* ct = cs + (size_t)buf * kAbPos * LD;
-        // scores: warp = 8 positions, half of the columns (every second step of 32)
-        float s[4][4];
+        // scores: warp = 16 positions, half of the columns (every second step of 32)
+        float s[4][4];                       // query part x 8-position tile
 #pragma unroll
         for (int u = 0; u < 4; ++u)
 #pragma unroll
             for (int e = 0; e < 4; ++e) s[u][e] = 0.f;
         const int wp = warp & 3, wk = warp >> 2;
+        const uint32_t ba = smem_u32(ct + (16 * wp + (lane & 7) + (lane >> 4) * 8) * LD + ((lane >> 3) & 1) * 8);
+        const uint32_t qo = (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
+        const uint32_t qha = smem_u32(qh) + qo, qla = smem_u32(ql) + qo;
+#pragma unroll 2
         for (int k0 = 32 * wk; k0 < KRp; k0 += 64) {
-            uint32_t b0, b1, b2, b3;
-            ldsm4(smem_u32(ct + (8 * wp + (lane & 7)) * LD + k0 + (lane >> 3) * 8), b0, b1, b2, b3);
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-                const int off = ((lane & 7) + ((lane >> 3) & 1) * 8) * LD + k0 + 16 * u + (lane >> 4) * 8;
-                uint32_t a0, a1, a2, a3;
-                ldsm4(smem_u32(qh + off), a0, a1, a2, a3);
-                mma_bf16(s[2 * u], a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
-                ldsm4(smem_u32(ql + off), a0, a1, a2, a3);
-                mma_bf16(s[2 * u + 1], a0, a1, a2, a3, u ? b2 : b0, u ? b3 : b1);
+                const uint32_t o = (uint32_t)(k0 + 16 * u) * 2;
+                uint32_t b0, b1, b2, b3, a0, a1, a2, a3;
+                ldsm4(ba + o, b0, b1, b2, b3);
+                ldsm4(qha + o, a0, a1, a2, a3);
+                mma_bf16(s[0], a0, a1, a2, a3, b0, b1);
+                mma_bf16(s[1], a0, a1, a2, a3, b2, b3);
+                ldsm4(qla + o, a0, a1, a2, a3);
+                mma_bf16(s[2], a0, a1, a2, a3, b0, b1);
+                mma_bf16(s[3], a0, a1, a2, a3, b2, b3);
             }
         }
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-            sc[wk][g + 8 * (e >> 1)][8 * wp + 2 * t4 + (e & 1)] = (s[0][e] + s[2][e]) + (s[1][e] + s[3][e]);
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sc[wk][g + 8 * (e >> 1)][16 * wp + 8 * n + 2 * t4 + (e & 1)] = s[n][e] + s[2 + n][e];
         __syncthreads();
-        // softmax: warp = 2 rows, lane = position
+        // softmax: warp = 2 rows, lane = positions lane and lane + 32
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            const int r = 2 * warp + i, row = rt * 16 + r, pos = c * kAbPos + lane;
-            const bool seen = row < p.T * p.H && pos < total && pos <= start + row / p.H;
-            const float v = seen ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY;
-            float mx = v;
+            const int r = 2 * warp + i, row = rt * 16 + r;
+            const long long lim = row < p.T * p.H ? min((long long)total - 1, start + row / p.H) - c * kAbPos : -1;   // last position seen
+            float v[2];
+#pragma unroll
+            for (int u = 0; u < 2; ++u) v[u] = lane + 32 * u <= lim ? sc[0][r][lane + 32 * u] + sc[1][r][lane + 32 * u] : -INFINITY;
+            float mx = fmaxf(v[0], v[1]);
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             const float mo = s_m[r], mn = fmaxf(mo, mx);
-            const float pv = seen ? exp2f(v - mn) : 0.f, f = mn == -INFINITY ? 1.f : exp2f(mo - mn);
-            const float sum = warp_sum(pv);
-            const bf16 hi = __float2bfloat16_rn(pv);
-            ph[r * (kAbPos + 8) + lane] = hi;
-            pl[r * (kAbPos + 8) + lane] = __float2bfloat16_rn(pv - __bfloat162float(hi));
+            const float f = mn == -INFINITY ? 1.f : exp2f(mo - mn);
+            float sum = 0.f;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const float pv = lane + 32 * u <= lim ? exp2f(v[u] - mn) : 0.f;
+                sum += pv;
+                const bf16 hi = __float2bfloat16_rn(pv);
+                ph[r * (kAbPos + 8) + lane + 32 * u] = hi;
+                pl[r * (kAbPos + 8) + lane + 32 * u] = __float2bfloat16_rn(pv - __bfloat162float(hi));
+            }
+            sum = warp_sum(sum);
             __syncwarp();
             if (lane == 0) {
                 s_m[r] = mn;
