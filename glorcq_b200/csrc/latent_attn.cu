@@ -290,9 +290,11 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const LaParams p) {
 
 // ---- attention over the cached latents, tensor cores ----------------------------------------------------
 
+constexpr int kAbThreads = 512;
+
 // 16 rows (query position, head) against one split of the positions; NT: 8-column tiles of the latent per warp
 template <int NT>
-__global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) {
+__global__ void __launch_bounds__(kAbThreads) latent_absorbed_kernel(const LaParams p) {
     extern __shared__ __align__(16) unsigned char la_raw[];
     const int KRp = p.KRp, LD = KRp + 8;
     bf16* qh = reinterpret_cast<bf16*>(la_raw);              // [16][LD]
@@ -300,7 +302,7 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
     bf16* cs = ql + 16 * LD;                                 // [2][kAbPos][LD]
     bf16* ph = cs + 2 * kAbPos * LD;                         // [16][kAbPos + 8]
     bf16* pl = ph + 16 * (kAbPos + 8);
-    __shared__ float sc[2][16][kAbPos + 1], s_m[16], s_l[16], s_f[16];
+    __shared__ float sc[4][16][kAbPos + 1], s_m[16], s_l[16], s_f[16];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     const int rt = blockIdx.x, z = blockIdx.y, b = blockIdx.z, tiles = gridDim.x;
     const int KR = p.K + p.R;
@@ -311,10 +313,10 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
     const SplitRange sr = split_range(p, z, total);
     const int c_lo = sr.lo, c_hi = sr.hi;
     const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.max_len * p.ldc;
-    auto load = [&](int c, int buf) {        // warp = rows warp, warp + 8, ..
+    auto load = [&](int c, int buf) {        // warp = rows warp, warp + 16, ..
         const uint32_t dst = smem_u32(cs + (size_t)buf * kAbPos * LD);
 #pragma unroll 4
-        for (int r = warp; r < kAbPos; r += 8) {
+        for (int r = warp; r < kAbPos; r += kAbThreads / 32) {
             const int pos = c * kAbPos + r;
             const bf16* src = cache + (size_t)(pos < total ? pos : 0) * p.ldc;
             for (int cc = 8 * lane; cc < KRp; cc += 256) cpa16(dst + (r * LD + cc) * 2, cc < KR ? src + cc : src, pos < total && cc < KR);
@@ -325,7 +327,7 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
         const bf16* src = reinterpret_cast<const bf16*>(p.qa) + ((size_t)b * p.rows16 + rt * 16) * KRp;
         const size_t plane = (size_t)p.B * p.rows16 * KRp;
         const int vec = KRp / 8;
-        for (int i = tid; i < 16 * vec; i += 256) {
+        for (int i = tid; i < 16 * vec; i += kAbThreads) {
             const int r = i / vec, cc = (i % vec) * 8;
             const bool live = rt * 16 + r < p.T * p.H;
             const bf16* q = live ? src + (size_t)r * KRp + cc : src;
@@ -353,7 +355,7 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
         }
         __syncthreads();
         const bf16* ct = cs + (size_t)buf * kAbPos * LD;
-        // scores: warp = 16 positions, half of the columns (every second step of 32)
+        // scores: warp = 16 positions, a quarter of the columns (every fourth step of 32)
         float s[4][4];                       // query part x 8-position tile
 #pragma unroll
         for (int u = 0; u < 4; ++u)
@@ -364,7 +366,7 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
         const uint32_t qo = (uint32_t)(((lane & 7) + ((lane >> 3) & 1) * 8) * LD + (lane >> 4) * 8) * 2;
         const uint32_t qha = smem_u32(qh) + qo, qla = smem_u32(ql) + qo;
 #pragma unroll 2
-        for (int k0 = 32 * wk; k0 < KRp; k0 += 64) {
+        for (int k0 = 32 * wk; k0 < KRp; k0 += 128) {
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
                 const uint32_t o = (uint32_t)(k0 + 16 * u) * 2;
@@ -383,14 +385,14 @@ __global__ void __launch_bounds__(256) latent_absorbed_kernel(const LaParams p) 
 #pragma unroll
             for (int e = 0; e < 4; ++e) sc[wk][g + 8 * (e >> 1)][16 * wp + 8 * n + 2 * t4 + (e & 1)] = s[n][e] + s[2 + n][e];
         __syncthreads();
-        // softmax: warp = 2 rows, lane = positions lane and lane + 32
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int r = 2 * warp + i, row = rt * 16 + r;
+        // softmax: warp = a row, lane = positions lane and lane + 32
+        {
+            const int r = warp, row = rt * 16 + r;
             const long long lim = row < p.T * p.H ? min((long long)total - 1, start + row / p.H) - c * kAbPos : -1;   // last position seen
             float v[2];
 #pragma unroll
-            for (int u = 0; u < 2; ++u) v[u] = lane + 32 * u <= lim ? sc[0][r][lane + 32 * u] + sc[1][r][lane + 32 * u] : -INFINITY;
+            for (int u = 0; u < 2; ++u) v[u] = lane + 32 * u <= lim ? (sc[0][r][lane + 32 * u] + sc[1][r][lane + 32 * u]) + (sc[2][r][lane + 32 * u] + sc[3][r][lane + 32 * u])
+                                                                          : -INFINITY;
             float mx = fmaxf(v[0], v[1]);
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -1007,7 +1009,7 @@ static size_t la_absorbed_smem(const LaParams& p) {
 // tensor-core form of the absorbed attention: 16-byte rows, latents of up to 512 columns
 static bool la_tensor(const glq_latent_t* a) {
     return a->dtype == GLQ_DT_BF16 && a->K % 16 == 0 && a->K <= 512 && a->R % 8 == 0 && a->ldc % 8 == 0 && al16(a->cache) &&
-           la_absorbed_smem(la_params(a)) <= 220 * 1024;
+           la_absorbed_smem(la_params(a)) <= 208 * 1024;
 }
 static int la_splits(const glq_latent_t* a) {
     if (!la_tensor(a)) return 1;
@@ -1072,9 +1074,8 @@ template <typename T> static int la_absorbed(const glq_latent_t* a, void* stream
         if (st != GLQ_OK) return st;
         const dim3 grid(p.rows16 / 16, p.splits, a->B);
         const size_t smem = la_absorbed_smem(p);
-        if (a->K <= 128) st = dn_launch(latent_absorbed_kernel<2>, grid, 256, smem, stream, p);
-        else if (a->K <= 256) st = dn_launch(latent_absorbed_kernel<4>, grid, 256, smem, stream, p);
-        else st = dn_launch(latent_absorbed_kernel<8>, grid, 256, smem, stream, p);
+        if (a->K <= 256) st = dn_launch(latent_absorbed_kernel<2>, grid, kAbThreads, smem, stream, p);
+        else st = dn_launch(latent_absorbed_kernel<4>, grid, kAbThreads, smem, stream, p);
     } else {
         st = dn_launch(latent_absorb_kernel<T, false>, dim3(a->H + 1, parts(a->K, a->D, 4L * dn_sms()), rb), 256, xa, stream, p);
         if (st != GLQ_OK) return st;
