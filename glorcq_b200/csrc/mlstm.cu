@@ -63,36 +63,40 @@ __device__ __forceinline__ void st4(bf16* p, float a, float b, float c, float d)
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(a, b), pack_bf2(c, d));
 }
 
+// one warp: out = rms_norm(o) * w * sigmoid(g) for V <= 128 U values, four per lane and step, all requested before the sum
+template <typename T, int U>
+__device__ __forceinline__ void norm_gate_row(const float* __restrict__ o, const T* __restrict__ g, const float* __restrict__ w,
+                                              T* __restrict__ out, int V, float eps, int lane) {
+    float4 x[U];
+    float gv[U][4], ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int v = (u * 32 + lane) * 4;
+        x[u] = v < V ? *reinterpret_cast<const float4*>(o + v) : make_float4(0, 0, 0, 0);
+        if (v < V) ld4(g + v, gv[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
+    const float inv = 1.f / sqrtf(warp_sum(ss) / V + eps);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const int v = (u * 32 + lane) * 4;
+        if (v < V) {
+            const float4 wv = *reinterpret_cast<const float4*>(w + v);
+            st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[u][0]), x[u].y * inv * wv.y * sigmoid_f(gv[u][1]),
+                x[u].z * inv * wv.z * sigmoid_f(gv[u][2]), x[u].w * inv * wv.w * sigmoid_f(gv[u][3]));
+        }
+    }
+}
+
 // one row of head h: out = rms_norm(o) * w * sigmoid(g); one warp
 template <typename T>
 __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, int h, int lane) {
     const float* o = p.o + row * p.H * p.V + (size_t)h * p.V;
     const T* g = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)p.H * (2 * p.D + p.V) + (size_t)h * p.V;
     T* out = reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V;
+    if (p.V % 4 == 0 && p.V <= 512 && p.vec4) return norm_gate_row<T, 4>(o, g, p.norm_w + (size_t)h * p.V, out, p.V, p.eps, lane);
     float ss = 0.f;
-    if (p.V % 4 == 0 && p.V <= 1024 && p.vec4) {          // four values per lane and step, kept in registers
-        float4 x[8];
-        float gv[8][4];                          // requested together with the row, ahead of its sum
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const int v = (u * 32 + lane) * 4;
-            if (v < p.V) ld4(g + v, gv[u]);
-            x[u] = v < p.V ? *reinterpret_cast<const float4*>(o + v) : make_float4(0, 0, 0, 0);
-            ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
-        }
-        const float inv = 1.f / sqrtf(warp_sum(ss) / p.V + p.eps);
-        const float* w = p.norm_w + (size_t)h * p.V;
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const int v = (u * 32 + lane) * 4;
-            if (v < p.V) {
-                const float4 wv = *reinterpret_cast<const float4*>(w + v);
-                st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[u][0]), x[u].y * inv * wv.y * sigmoid_f(gv[u][1]),
-                    x[u].z * inv * wv.z * sigmoid_f(gv[u][2]), x[u].w * inv * wv.w * sigmoid_f(gv[u][3]));
-            }
-        }
-        return;
-    }
     for (int v = lane; v < p.V; v += 32) {
         const float x = o[v];
         ss += x * x;
