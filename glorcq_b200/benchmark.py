@@ -35,7 +35,7 @@ def zokunex_config(size, n_layers=8):
         mlp = {"kind": "dense", "ff": s["ff"]} if l == 0 else \
             {"kind": "moe", "expert": {"ff": s["eff"]}, "router": {"experts": s["experts"], "identity": s["identity"], "top": s["top"]}}
         out.append(dict(mixer, mlp=mlp))
-    return {"architecture": "Zokunex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "logit_scale": 0.5, "layers": out}
+    return {"architecture": "Zokunex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "logit_scale": 1.0, "layers": out}
 
 
 def closest_config(size, n_layers=8):

@@ -1,4 +1,4 @@
-"""Plain, slow implementation of the Zokunex decoder in torch on the CPU: the checker of the product path.
+"""Plain, slow implementation of the Zokunex decoder in torch on the CPU: what the tests compare the product path with.
 
 One function per mechanism, token by token where the mechanism is a recurrence, with nothing shared with
 ``glorcq_b200``.  ``W`` maps tensor names to tensors; everything is evaluated in the dtype of ``W`` (float32 or
