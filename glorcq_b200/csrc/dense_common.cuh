@@ -115,7 +115,8 @@ inline int dn_sms() {
 template <typename... KArgs, typename... Args>
 inline int dn_launch_if(bool early, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
     static const bool pdl = std::getenv("GLQ_NO_PDL") == nullptr;
-    if (smem > 48 * 1024) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    // 48 KB without opting in is dynamic plus static shared memory; no kernel here has more than 24 KB of the latter
+    if (smem > 24 * 1024) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(block);

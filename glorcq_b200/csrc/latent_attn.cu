@@ -1094,7 +1094,8 @@ extern "C" int glq_latent_absorbed(const glq_latent_t* a, void* stream) {
     if (!la_sizes_ok(a) || !a->q || !a->ckr || !a->norm_w || !a->cache || !a->start || (a->rot_dims && (!a->cos_t || !a->sin_t)) || !a->ukt || !a->uv || !a->gate ||
         !a->out || !a->workspace)
         return GLQ_ERR_ARG;
-    if (!al16(a->workspace) || !al16(a->ukt) || !al16(a->uv)) return GLQ_ERR_ALIGN;
+    // matrices with rows of whole vectors are read eight values at a time, others one by one
+    if (!al16(a->workspace) || (a->D % 8 == 0 && !al16(a->ukt)) || (a->K % 8 == 0 && !al16(a->uv))) return GLQ_ERR_ALIGN;
     if (a->K > 4096 || a->D > 4096 || a->R > 4096 || a->B > 65535 || a->H > 65534) return GLQ_ERR_UNSUPPORTED;
     if (a->T == 0) return GLQ_OK;
     return a->dtype == GLQ_DT_BF16 ? la_absorbed<bf16>(a, stream) : la_absorbed<float>(a, stream);

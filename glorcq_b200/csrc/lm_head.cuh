@@ -268,7 +268,7 @@ inline int lm_head_launch(const void* x, int64_t ldx, const void* W, int B, int 
     static size_t configured[64] = {0};
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess) return GLQ_ERR_CUDA;
-    if (smem > 48 * 1024 && (dev < 0 || dev >= 64 || configured[dev] < smem)) {
+    if (smem > 40 * 1024 && (dev < 0 || dev >= 64 || configured[dev] < smem)) {
         if (cudaFuncSetAttribute(lm_head_kernel<BF>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return GLQ_ERR_CUDA;
         if (dev >= 0 && dev < 64) configured[dev] = smem;

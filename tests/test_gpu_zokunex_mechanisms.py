@@ -96,7 +96,7 @@ def test_norm_and_residual(dev, rows, width, dtype):
 
 # ---- routing and experts -------------------------------------------------------------------------------------
 @pytest.mark.parametrize("n", [1, 7, 33, 400, 1500])
-@pytest.mark.parametrize("E,identity,top", [(6, 2, 3), (5, 0, 1), (40, 3, 8), (2, 1, 3), (300, 20, 4)])
+@pytest.mark.parametrize("E,identity,top", [(6, 2, 3), (5, 0, 1), (40, 3, 8), (2, 1, 3), (300, 20, 4), (590, 10, 2)])
 def test_routing(dev, n, E, identity, top):
     from glorcq_b200 import dense
     A = E + identity
@@ -270,7 +270,8 @@ def test_matrix_memory_remembers_one_far_key(dev):
 
 
 # ---- latent attention ------------------------------------------------------------------------------------------
-LATENT_SIZES = [(3, 16, 8, 24, 48), (2, 40, 16, 16, 32), (5, 24, 8, 40, 144), (4, 128, 64, 128, 512), (2, 9, 6, 11, 20), (1, 200, 24, 8, 272), (20, 8, 8, 8, 16)]
+LATENT_SIZES = [(3, 16, 8, 24, 48), (2, 40, 16, 16, 32), (5, 24, 8, 40, 144), (4, 128, 64, 128, 512), (2, 9, 6, 11, 20), (1, 200, 24, 8, 272), (20, 8, 8, 8, 16),
+                (2, 16, 8, 16, 80), (2, 16, 8, 16, 96), (1, 24, 16, 8, 112), (3, 5, 4, 7, 9)]
 
 
 def _latent_mixer(dev, dtype, sizes, seed=0, width=64, scale=None, base=10000.0):
@@ -363,7 +364,7 @@ def test_rotation_covers_only_the_first_dims(dev):
 
 def test_output_projection_and_argmax(dev):
     from glorcq_b200 import dense
-    for rows, width, vocab in ((1, 96, 160), (11, 64, 1000), (3, 104, 333), (100, 96, 160)):
+    for rows, width, vocab in ((1, 96, 160), (11, 64, 1000), (3, 104, 333), (100, 96, 160), (2, 2784, 200)):
         x, W = rnd(rows, width, seed=rows), rnd(vocab, width, seed=vocab)
         logits, best = dense.head(x.to(dev), W.to(dev), 0.37, {})
         ref = 0.37 * x.double() @ W.double().T
