@@ -19,7 +19,7 @@ INCLUDE = os.path.join(HERE, "..", "include")
 LIB = os.path.join(HERE, "libglorcq_b200.so")
 DENSE_LIB = os.path.join(HERE, "libglorcq_b200_dense.so")
 SOURCES = {LIB: ["api.cu", "moe.cu", "attn.cu", "lm_head.cu"],
-           DENSE_LIB: ["dense_mm.cu", "dense_aux.cu", "dense_head.cu", "mlstm.cu", "latent_attn.cu"]}
+           DENSE_LIB: ["dense_mm.cu", "dense_aux.cu", "dense_head.cu", "mlstm.cu", "decay_attn.cu", "gqa_attn.cu", "latent_attn.cu"]}
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "-Xcompiler", "-fPIC"]
 
 

@@ -124,7 +124,8 @@ _SIGS = {
 
 # ---- unquantized decoders -----------------------------------------------------------------------------
 DT_BF16, DT_F32 = 0, 1
-ACT_NONE, ACT_RELU2, ACT_GELU_ERF = 0, 1, 2
+ACT_NONE, ACT_RELU2, ACT_GELU_ERF, ACT_GELU_TANH, ACT_SILU_GLU = range(5)
+GATE_SIGMOID, GATE_SILU = 0, 1
 
 
 class DenseMM(C.Structure):
@@ -132,7 +133,9 @@ class DenseMM(C.Structure):
     _fields_ = [(f, C.c_int32) for f in ("dtype", "act", "N", "K", "rows", "n_matrices", "max_slots", "max_slot_rows", "split")] + \
                [("alpha", C.c_float)] + [(f, vp) for f in ("slot_index", "n_slots", "slot_count", "slot_offset", "entry_row", "x")] + \
                [("ldx", C.c_int64), ("W", vp), ("ldw", C.c_int64), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp),
-                ("hn_o", vp), ("hn_g", vp), ("hn_ldg", C.c_int64), ("hn_w", vp), ("hn_heads", C.c_int32), ("hn_eps", C.c_float)]
+                ("hn_o", vp), ("hn_g", vp), ("hn_ldg", C.c_int64), ("hn_w", vp), ("hn_heads", C.c_int32), ("hn_eps", C.c_float),
+                ("hn_wstride", C.c_int32), ("hn_gate", C.c_int32), ("mul", vp), ("ldmul", C.c_int64), ("mul_row", vp),
+                ("mul_rows", C.c_int32), ("residual", C.c_int32)]
 
 
 class MLstm(C.Structure):
@@ -141,6 +144,23 @@ class MLstm(C.Structure):
                [("gate_cap", C.c_float), ("eps", C.c_float), ("qkvg", vp), ("ldp", C.c_int64), ("gates", vp), ("ldg", C.c_int64)] + \
                [(f, vp) for f in ("bias_i", "bias_f", "norm_w", "S", "n", "m", "o", "out", "workspace")] + \
                [("workspace_bytes", C.c_size_t)]
+
+
+class Decay(C.Structure):
+    """glq_decay_t"""
+    _fields_ = [(f, C.c_int32) for f in ("dtype", "B", "T", "H", "D", "V", "rank", "rot_dims", "rot_pairs", "max_len", "norm_stride", "gate",
+                                         "state_idle")] + [(f, C.c_float) for f in ("q_scale", "k_scale", "eps", "tau")] + \
+               [(f, vp) for f in ("q", "k", "v", "g")] + [("ldp", C.c_int64), ("decay", vp), ("a", vp), ("lda", C.c_int64)] + \
+               [(f, vp) for f in ("a2", "a2b", "start", "cos_t", "sin_t", "norm_w", "S", "o", "out", "workspace")] + \
+               [("workspace_bytes", C.c_size_t)]
+
+
+class Gqa(C.Structure):
+    """glq_gqa_t"""
+    _fields_ = [(f, C.c_int32) for f in ("dtype", "B", "T", "H", "G", "D", "V", "rot_dims", "rot_pairs", "qk_norm", "max_len", "S",
+                                         "state_idle")] + [("scale", C.c_float), ("eps", C.c_float)] + \
+               [(f, vp) for f in ("start", "q", "k", "v")] + [("ldp", C.c_int64)] + \
+               [(f, vp) for f in ("cos_t", "sin_t", "kc", "vc", "out", "workspace")] + [("workspace_bytes", C.c_size_t)]
 
 
 class Latent(C.Structure):
@@ -167,12 +187,21 @@ _DENSE_SIGS = {
     "glq_dense_debug_error": (_i, [vp, _i]),
     "glq_dense_matmul": (_i, [C.POINTER(DenseMM), vp]),
     "glq_dense_matmul_path": (_i, [C.POINTER(DenseMM)]),
-    "glq_dense_embed": (_i, [_i, vp, vp, _i, _i, _i, vp, vp, vp]),
+    "glq_dense_embed": (_i, [_i, vp, vp, _i, _i, _i, vp, _f, vp, vp, vp]),
+    "glq_dense_rms_add": (_i, [_i, vp, _l, vp, vp, _l, vp, _f, vp, _f, _i, _i, vp, vp, vp]),
     "glq_dense_add_norm": (_i, [_i, vp, vp, vp, _f, _i, _i, vp, vp, vp]),
     "glq_mlstm_slices": (_i, [_i]),
     "glq_mlstm_workspace_bytes": (_z, [C.POINTER(MLstm)]),
     "glq_mlstm_step": (_i, [C.POINTER(MLstm), vp]),
     "glq_mlstm_chunk": (_i, [C.POINTER(MLstm), vp]),
+    "glq_decay_slices": (_i, [_i]),
+    "glq_decay_workspace_bytes": (_z, [C.POINTER(Decay)]),
+    "glq_decay_step": (_i, [C.POINTER(Decay), vp]),
+    "glq_decay_chunk_supported": (_i, [C.POINTER(Decay)]),
+    "glq_decay_chunk": (_i, [C.POINTER(Decay), vp]),
+    "glq_gqa_form": (_i, [C.POINTER(Gqa)]),
+    "glq_gqa_decode_workspace_bytes": (_z, [C.POINTER(Gqa)]),
+    "glq_gqa": (_i, [C.POINTER(Gqa), vp]),
     "glq_latent_prep": (_i, [C.POINTER(Latent), vp]),
     "glq_latent_absorbed_workspace_bytes": (_z, [C.POINTER(Latent)]),
     "glq_latent_absorbed": (_i, [C.POINTER(Latent), vp]),

@@ -55,6 +55,62 @@ class MatrixMemoryState:
             dst.copy_(src)
 
 
+class DecayState:
+    """State S of linear attention with decay, in 32-bit, by slices of 32 value columns."""
+
+    def __init__(self, batch, max_len, heads, dim, vdim, device):
+        self.max_len = max_len                          # positions a sequence may reach (rotations are tabulated that far)
+        self.S = torch.zeros(batch, heads, _lib.dense().glq_decay_slices(vdim), dim, 32, device=device)
+
+    def reset(self):
+        self.S.zero_()
+
+    def snapshot(self, positions):
+        return self.S.clone()
+
+    def restore(self, saved):
+        self.S.copy_(saved)
+
+
+class KeyValueState:
+    """Cached positions of grouped-query attention: keys (batch, position, head, dim) and values."""
+
+    def __init__(self, batch, max_len, kv_heads, dim, vdim, device, dtype):
+        self.k = torch.zeros(batch, max_len, kv_heads, dim, device=device, dtype=dtype)
+        self.v = torch.zeros(batch, max_len, kv_heads, vdim, device=device, dtype=dtype)
+
+    def reset(self):
+        pass                                            # positions are written before they are read
+
+    def snapshot(self, positions):
+        return self.k[:, :positions].clone(), self.v[:, :positions].clone()
+
+    def restore(self, saved):
+        for dst, src in zip((self.k, self.v), saved):
+            dst[:, :src.shape[1]].copy_(src)
+
+
+class SideBySideState:
+    """The states of mixers that run side by side in one layer."""
+
+    def __init__(self, *parts):
+        self.parts = parts
+
+    def __getitem__(self, i):
+        return self.parts[i]
+
+    def reset(self):
+        for s in self.parts:
+            s.reset()
+
+    def snapshot(self, positions):
+        return [s.snapshot(positions) for s in self.parts]
+
+    def restore(self, saved):
+        for s, v in zip(self.parts, saved):
+            s.restore(v)
+
+
 class LayerStateCache:
     """One state object per layer."""
 

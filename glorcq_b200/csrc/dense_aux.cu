@@ -1,5 +1,5 @@
-// Row kernels of the unquantized decoders: embedding, residual add with the layer norm of the sublayer's output,
-// softmax routing with a correction term and its entry lists, and the weighted sum of the experts' outputs fused with
+// Row kernels of the unquantized decoders: embedding, residual add with the layer norm of the sublayer's output or with
+// RMS norms on either side of the add, softmax routing with a correction term and its entry lists, and the weighted sum of the experts' outputs fused with
 // the norm and the residual add that follow it.  One CTA per row; the residual stream and all statistics are float.
 #include "dense_common.cuh"
 #include "moe_plan.cuh"
@@ -11,17 +11,24 @@ constexpr int kMaxC = 32768;          // row length; a row is staged in shared m
 
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads) dense_embed_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table,
-                                                                  int C, int vocab, float* __restrict__ x, T* __restrict__ h) {
+                                                                  int C, int vocab, const float* __restrict__ hw, float eps,
+                                                                  float* __restrict__ x, T* __restrict__ h) {
+    __shared__ float red[32];
     pdl_wait();
     pdl_release();
     const size_t row = blockIdx.x;
     long long id = ids[row];
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+    float s = 0.f;
     for (int c = threadIdx.x; c < C; c += kRowThreads) {
         const T v = table[(size_t)id * C + c];
         x[row * C + c] = to_f(v);
-        h[row * C + c] = v;
+        if (!hw) h[row * C + c] = v;
+        s += to_f(v) * to_f(v);
     }
+    if (!hw) return;
+    const float inv = 1.f / sqrtf(block_sum(s, red) / C + eps);
+    for (int c = threadIdx.x; c < C; c += kRowThreads) h[row * C + c] = from_f<T>(to_f(table[(size_t)id * C + c]) * inv * hw[c]);
 }
 
 // ys: the sublayer's output row.  x += norm(ys) * w; h = x, or norm(x) * final_w
@@ -151,6 +158,125 @@ __global__ void __launch_bounds__(kRowThreads) dense_add_norm_kernel(const float
     } else {
         for (int c = threadIdx.x; c < C; c += kRowThreads) ys[c] = y[o + c];
         norm_add_row<T>(ys, red, w, fw, eps, C, x + o, h + o);
+    }
+}
+
+// x += alpha * (rms(y) * w + rms(y2) * w2); h = rms(x) * hw.  y2 may be missing, y too (nothing is added); without w, y is
+// added as it is, and without hw, h = x.
+struct RmsParams {
+    const float* y;
+    const float* w;
+    const float* y2;
+    const float* w2;
+    const float* hw;
+    long long ldy, ldy2;
+    float eps, alpha;
+    int C;
+};
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    a = warp_sum(a);
+    b = warp_sum(b);
+    __syncthreads();
+    if (lane == 0) red[warp] = make_float2(a, b);
+    __syncthreads();
+    const float2 v = lane < kRowThreads / 32 ? red[lane] : make_float2(0.f, 0.f);
+    return make_float2(warp_sum(v.x), warp_sum(v.y));
+}
+// STEPS 0: any width, one value per thread and step; else the row in registers, 8 values per thread and step
+template <typename T, int STEPS>
+__global__ void __launch_bounds__(kRowThreads) dense_rms_add_kernel(const RmsParams p, float* __restrict__ xg, T* __restrict__ hg) {
+    __shared__ float2 red[32];
+    pdl_wait();
+    pdl_release();
+    const int C = p.C;
+    const size_t row = blockIdx.x;
+    float* x = xg + row * C;
+    T* h = hg ? hg + row * C : nullptr;
+    const float* y = p.y ? p.y + row * p.ldy : nullptr;
+    const float* y2 = p.y2 ? p.y2 + row * p.ldy2 : nullptr;
+    if constexpr (STEPS > 0) {
+        float xv[STEPS][8], yv[STEPS][8], zv[STEPS][8];
+        float s = 0.f, s2 = 0.f;
+#pragma unroll
+        for (int u = 0; u < STEPS; ++u) {
+            const int c = (u * kRowThreads + threadIdx.x) * 8;
+            if (c >= C) continue;
+            ld8(x + c, xv[u]);
+            if (y) {
+                ld8(y + c, yv[u]);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) s += yv[u][i] * yv[u][i];
+            }
+            if (y2) {
+                ld8(y2 + c, zv[u]);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) s2 += zv[u][i] * zv[u][i];
+            }
+        }
+        float f = p.alpha, f2 = p.alpha;
+        if (p.w) {
+            const float2 t = block_sum2(s, s2, red);
+            f *= 1.f / sqrtf(t.x / C + p.eps);
+            f2 *= 1.f / sqrtf(t.y / C + p.eps);
+        }
+        s = 0.f;
+#pragma unroll
+        for (int u = 0; u < STEPS; ++u) {
+            const int c = (u * kRowThreads + threadIdx.x) * 8;
+            if (c >= C) continue;
+            float wv[8];
+            if (y) {
+                if (p.w) ld8(p.w + c, wv);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) xv[u][i] += yv[u][i] * f * (p.w ? wv[i] : 1.f);
+            }
+            if (y2) {
+                if (p.w2) ld8(p.w2 + c, wv);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) xv[u][i] += zv[u][i] * f2 * (p.w2 ? wv[i] : 1.f);
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s += xv[u][i] * xv[u][i];
+            if (y) st8<float>(x + c, xv[u]);
+            if (h && !p.hw) st8<T>(h + c, xv[u]);
+        }
+        if (!h || !p.hw) return;
+        const float inv = 1.f / sqrtf(block_sum2(s, 0.f, red).x / C + p.eps);
+#pragma unroll
+        for (int u = 0; u < STEPS; ++u) {
+            const int c = (u * kRowThreads + threadIdx.x) * 8;
+            if (c >= C) continue;
+            float wv[8];
+            ld8(p.hw + c, wv);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) wv[i] *= xv[u][i] * inv;
+            st8<T>(h + c, wv);
+        }
+    } else {
+        float f = p.alpha, f2 = p.alpha;
+        if (p.w) {
+            float s = 0.f, s2 = 0.f;
+            for (int c = threadIdx.x; c < C; c += kRowThreads) {
+                if (y) s += y[c] * y[c];
+                if (y2) s2 += y2[c] * y2[c];
+            }
+            const float2 t = block_sum2(s, s2, red);
+            f *= 1.f / sqrtf(t.x / C + p.eps);
+            f2 *= 1.f / sqrtf(t.y / C + p.eps);
+        }
+        float s = 0.f;
+        for (int c = threadIdx.x; c < C; c += kRowThreads) {
+            float v = x[c];
+            if (y) v += y[c] * f * (p.w ? p.w[c] : 1.f);
+            if (y2) v += y2[c] * f2 * (p.w2 ? p.w2[c] : 1.f);
+            if (y) x[c] = v;
+            if (h && !p.hw) h[c] = from_f<T>(v);
+            s += v * v;
+        }
+        if (!h || !p.hw) return;
+        const float inv = 1.f / sqrtf(block_sum2(s, 0.f, red).x / C + p.eps);
+        for (int c = threadIdx.x; c < C; c += kRowThreads) h[c] = from_f<T>(x[c] * inv * p.hw[c]);   // x: own writes
     }
 }
 
@@ -309,13 +435,13 @@ template <typename F> static int by_dtype(int dtype, F f) {
     return GLQ_ERR_ARG;
 }
 
-extern "C" int glq_dense_embed(int dtype, const int64_t* ids, const void* table, int rows, int C, int vocab, float* x, void* h,
-                               void* stream) {
+extern "C" int glq_dense_embed(int dtype, const int64_t* ids, const void* table, int rows, int C, int vocab, const float* hw, float eps,
+                               float* x, void* h, void* stream) {
     if (!ids || !table || !x || !h || rows < 0 || C <= 0 || vocab <= 0) return GLQ_ERR_ARG;
     if (rows == 0) return GLQ_OK;
     return by_dtype(dtype, [&](auto z) {
         using T = decltype(z);
-        return dn_launch(dense_embed_kernel<T>, dim3(rows), kRowThreads, 0, stream, ids, (const T*)table, C, vocab, x, (T*)h);
+        return dn_launch(dense_embed_kernel<T>, dim3(rows), kRowThreads, 0, stream, ids, (const T*)table, C, vocab, hw, eps, x, (T*)h);
     });
 }
 
@@ -334,6 +460,22 @@ extern "C" int glq_dense_add_norm(int dtype, const float* y, const float* w, con
         if (vec && C <= 32 * kRowThreads)
             return dn_launch(dense_add_norm_kernel<T, 4>, dim3(rows), kRowThreads, 0, stream, y, w, final_w, eps, C, x, (T*)h);
         return dn_launch(dense_add_norm_kernel<T, 0>, dim3(rows), kRowThreads, (size_t)C * 4, stream, y, w, final_w, eps, C, x, (T*)h);
+    });
+}
+
+extern "C" int glq_dense_rms_add(int dtype, const float* y, int64_t ldy, const float* w, const float* y2, int64_t ldy2, const float* w2,
+                                 float alpha, const float* hw, float eps, int rows, int C, float* x, void* h, void* stream) {
+    if (!x || rows < 0 || C <= 0 || (!y && y2) || (y2 && !w != !w2) || (!y && !h)) return GLQ_ERR_ARG;
+    if (rows == 0) return GLQ_OK;
+    const RmsParams p{y, w, y2, w2, hw, (long long)ldy, (long long)ldy2, eps, alpha, C};
+    return by_dtype(dtype, [&](auto z) {
+        using T = decltype(z);
+        const bool vec = C % 8 == 0 && al16(x) && al16(h) && al16(y) && al16(y2) && al16(w) && al16(w2) && al16(hw) && (!y || ldy % 4 == 0) &&
+                         (!y2 || ldy2 % 4 == 0);
+        auto go = [&](auto kern) { return dn_launch(kern, dim3(rows), kRowThreads, 0, stream, p, x, (T*)h); };
+        if (vec && C <= 8 * kRowThreads) return go(dense_rms_add_kernel<T, 1>);
+        if (vec && C <= 16 * kRowThreads) return go(dense_rms_add_kernel<T, 2>);
+        return go(dense_rms_add_kernel<T, 0>);
     });
 }
 

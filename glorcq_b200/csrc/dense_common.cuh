@@ -61,16 +61,22 @@ __device__ __forceinline__ void pdl_release() { asm volatile("griddepcontrol.lau
 
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
+__device__ __forceinline__ float gate_f(int gate, float v) { return gate == GLQ_GATE_SILU ? v * sigmoid_f(v) : sigmoid_f(v); }
+
 template <int ACT> __device__ __forceinline__ float act_f(float z) {
     if (ACT == GLQ_ACT_RELU2) {
         const float r = fmaxf(z, 0.f);
         return r * r;
     }
     if (ACT == GLQ_ACT_GELU_ERF) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+    if (ACT == GLQ_ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
     return z;
 }
 __device__ __forceinline__ float act_dyn(int act, float z) {
-    return act == GLQ_ACT_RELU2 ? act_f<GLQ_ACT_RELU2>(z) : (act == GLQ_ACT_GELU_ERF ? act_f<GLQ_ACT_GELU_ERF>(z) : z);
+    if (act == GLQ_ACT_RELU2) return act_f<GLQ_ACT_RELU2>(z);
+    if (act == GLQ_ACT_GELU_ERF) return act_f<GLQ_ACT_GELU_ERF>(z);
+    if (act == GLQ_ACT_GELU_TANH) return act_f<GLQ_ACT_GELU_TANH>(z);
+    return z;
 }
 
 // block-wide sum, every thread gets it; red: 32 floats of shared memory

@@ -31,8 +31,12 @@ struct DmParams {
     const void* hn_g;
     const float* hn_w;
     long long hn_ldg;
-    int hn_heads;
+    int hn_heads, hn_wstride, hn_gate;
     float hn_eps;
+    const void* mul;
+    const int64_t* mul_row;
+    long long ldmul;
+    int mul_rows, residual;
 };
 
 struct DmSlot {
@@ -44,10 +48,28 @@ __device__ __forceinline__ DmSlot dm_slot(const DmParams& p, int s) {
     return {__ldg(p.slot_index + s), __ldg(p.slot_offset + s), __ldg(p.slot_count + s)};
 }
 
-template <typename T> __device__ __forceinline__ void dm_store(const DmParams& p, int row, int n, float v) {
+template <typename T> __device__ __forceinline__ const T* dm_mul_row(const DmParams& p, int row) {
+    long long r = row;
+    if (p.mul_row) {
+        r = p.mul_row[row];
+        r = r < 0 ? 0 : (r >= p.mul_rows ? p.mul_rows - 1 : r);
+    }
+    return reinterpret_cast<const T*>(p.mul) + r * p.ldmul;
+}
+template <typename T, bool MUL = true> __device__ __forceinline__ void dm_store(const DmParams& p, int row, int n, float v) {
+    if (MUL && p.mul) v *= to_f(dm_mul_row<T>(p, row)[n]);
+    if (p.residual) {
+        float* x = p.y32 + (size_t)row * p.ldy32 + n;
+        v += *x;
+        *x = v;
+        if (p.y) reinterpret_cast<T*>(p.y)[(size_t)row * p.ldy + n] = from_f<T>(v);
+        return;
+    }
     if (n < p.split) reinterpret_cast<T*>(p.y)[(size_t)row * p.ldy + n] = from_f<T>(v);
     else p.y32[(size_t)row * p.ldy32 + (n - p.split)] = v;
 }
+
+__device__ __forceinline__ float dm_glu(float gate, float other) { return gate * sigmoid_f(gate) * other; }
 
 // =====================================================================================================
 // streaming kernel: up to 8 rows per slot
@@ -104,7 +126,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                 pdl_release();
             }
             if (p.hn_o) {
-                // rows = per-head RMS norm of hn_o, times its weight, times the sigmoid of the gate; warp = (row, head)
+                // rows = per-head RMS norm of hn_o, times its weight, times the gate; warp = (row, head)
                 const int V = K / p.hn_heads;
                 for (int i = w; i < p.xrows * p.hn_heads; i += WARPS) {
                     const int row = i / p.hn_heads, k0 = (i % p.hn_heads) * V;
@@ -125,9 +147,10 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                     }
                     const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
                     const bf16* gt = reinterpret_cast<const bf16*>(p.hn_g) + (size_t)row * p.hn_ldg;
+                    const float* nw = p.hn_w ? p.hn_w + (size_t)(i % p.hn_heads) * p.hn_wstride - k0 : nullptr;
 #pragma unroll 4
                     for (int k = k0 + lane; k < k0 + V; k += 32)
-                        xs[(size_t)row * XS + k] = from_f<bf16>(o[k] * inv * p.hn_w[k] * sigmoid_f(to_f(gt[k])));
+                        xs[(size_t)row * XS + k] = from_f<bf16>(o[k] * inv * (nw ? nw[k] : 1.f) * gate_f(p.hn_gate, to_f(gt[k])));
                 }
                 for (int i = tid; i < p.xrows * 32; i += THREADS) {  // channels past K of the last chunk
                     const int k = K + (i & 31);
@@ -173,7 +196,13 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                 acc[3] += v.w;
             }
         }
-        if (s == 0 && live) {
+        if (s == 0 && live && p.act == GLQ_ACT_SILU_GLU) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int n = tile * 8 + g, row = 2 * t + i;
+                if (row < sl.cnt && 2 * n < p.N) dm_store<bf16>(p, sl.off + row, n, p.alpha * dm_glu(acc[i], acc[2 + i]));
+            }
+        } else if (s == 0 && live) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
@@ -227,7 +256,12 @@ __global__ void __launch_bounds__(256) dense_generic_kernel(const DmParams p) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int m = m0 + ty + 16 * i, n = n0 + tx + 16 * j;
-                if (m < sl.cnt && n < p.N) dm_store<T>(p, sl.off + m, n, p.alpha * act_dyn(p.act, acc[i][j]));
+                if (p.act == GLQ_ACT_SILU_GLU) {
+                    const float other = __shfl_xor_sync(0xffffffffu, acc[i][j], 8);
+                    if (tx < 8 && m < sl.cnt && n < p.N) dm_store<T>(p, sl.off + m, (n0 >> 1) + 8 * j + tx, p.alpha * dm_glu(acc[i][j], other));
+                } else if (m < sl.cnt && n < p.N) {
+                    dm_store<T>(p, sl.off + m, n, p.alpha * act_dyn(p.act, acc[i][j]));
+                }
             }
     }
 }
@@ -416,20 +450,54 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
                 tc_ld_wait();
                 if (!rin) continue;
                 float f[16];
+                if (p.act == GLQ_ACT_SILU_GLU) {
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) f[j] = p.alpha * dm_glu(__uint_as_float(v[j]), __uint_as_float(v[j + 8]));
+                    const int m0 = n0 >> 1;
+                    if (p.vec_y && !p.mul)
+                        *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.y) + orow * p.ldy + m0) =
+                            make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
+                    else
+#pragma unroll
+                        for (int j = 0; j < 8; ++j) dm_store<bf16>(p, (int)orow, m0 + j, f[j]);
+                    continue;
+                }
 #pragma unroll
                 for (int j = 0; j < 16; ++j) f[j] = p.alpha * act_dyn(p.act, __uint_as_float(v[j]));
-                if (n0 + 16 <= p.split && p.vec_y) {
+                if (p.mul) {
+                    const bf16* mr = dm_mul_row<bf16>(p, (int)orow) + n0;
+#pragma unroll
+                    for (int j = 0; j < 16; ++j)
+                        if (n0 + j < p.N) f[j] *= to_f(mr[j]);
+                }
+                if (p.residual && n0 + 16 <= p.N && p.vec_y32 && (!p.y || p.vec_y)) {
+                    float4* dst = reinterpret_cast<float4*>(p.y32 + orow * p.ldy32 + n0);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const float4 x = dst[j];
+                        f[4 * j] += x.x;
+                        f[4 * j + 1] += x.y;
+                        f[4 * j + 2] += x.z;
+                        f[4 * j + 3] += x.w;
+                        dst[j] = make_float4(f[4 * j], f[4 * j + 1], f[4 * j + 2], f[4 * j + 3]);
+                    }
+                    if (p.y) {
+                        uint4* yd = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.y) + orow * p.ldy + n0);
+                        yd[0] = make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
+                        yd[1] = make_uint4(pack_bf2(f[8], f[9]), pack_bf2(f[10], f[11]), pack_bf2(f[12], f[13]), pack_bf2(f[14], f[15]));
+                    }
+                } else if (n0 + 16 <= p.split && p.vec_y) {
                     uint4* dst = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.y) + orow * p.ldy + n0);
                     dst[0] = make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
                     dst[1] = make_uint4(pack_bf2(f[8], f[9]), pack_bf2(f[10], f[11]), pack_bf2(f[12], f[13]), pack_bf2(f[14], f[15]));
-                } else if (n0 >= p.split && n0 + 16 <= p.N && p.vec_y32) {
+                } else if (!p.residual && n0 >= p.split && n0 + 16 <= p.N && p.vec_y32) {
                     float4* dst = reinterpret_cast<float4*>(p.y32 + orow * p.ldy32 + (n0 - p.split));
 #pragma unroll
                     for (int j = 0; j < 4; ++j) dst[j] = make_float4(f[4 * j], f[4 * j + 1], f[4 * j + 2], f[4 * j + 3]);
                 } else {
 #pragma unroll
                     for (int j = 0; j < 16; ++j)
-                        if (n0 + j < p.N) dm_store<bf16>(p, (int)orow, n0 + j, f[j]);
+                        if (n0 + j < p.N) dm_store<bf16, false>(p, (int)orow, n0 + j, f[j]);
                 }
             }
             tc_fence_before();
@@ -500,6 +568,9 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     if (a->rows == 0) return GLQ_OK;
     const bool grouped = a->slot_index != nullptr;
     if ((!a->x && !a->hn_o) || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
+    if (a->act == GLQ_ACT_SILU_GLU && (a->N % 16 || a->split != a->N)) return GLQ_ERR_ARG;
+    if (a->residual && (a->split != 0 || grouped)) return GLQ_ERR_ARG;
+    if (a->mul_row && a->mul_rows <= 0) return GLQ_ERR_ARG;
     if (grouped && (!a->n_slots || !a->slot_count || !a->slot_offset || a->max_slots <= 0 || a->max_slot_rows <= 0 || a->n_matrices <= 0))
         return GLQ_ERR_ARG;
     if (!grouped && a->entry_row) return GLQ_ERR_ARG;
@@ -524,17 +595,24 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     p.split = a->split;
     p.act = a->act;
     p.alpha = a->alpha;
+    p.mul = a->mul;
+    p.ldmul = a->ldmul;
+    p.mul_row = a->mul_row;
+    p.mul_rows = a->mul_rows;
+    p.residual = a->residual;
     p.vec_y = a->y && al16(a->y) && a->ldy % 8 == 0;
     p.vec_y32 = a->y32 && al16(a->y32) && a->ldy32 % 4 == 0 && a->split % 4 == 0;
     const int path = glq_dense_matmul_path(a);
     if (a->hn_o) {
-        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !a->hn_g || !a->hn_w || !al16(a->hn_o)) return GLQ_ERR_ARG;
+        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !a->hn_g || !al16(a->hn_o)) return GLQ_ERR_ARG;
         p.hn_o = a->hn_o;
         p.hn_g = a->hn_g;
         p.hn_w = a->hn_w;
         p.hn_ldg = a->hn_ldg;
         p.hn_heads = a->hn_heads;
         p.hn_eps = a->hn_eps;
+        p.hn_wstride = a->hn_wstride;
+        p.hn_gate = a->hn_gate;
     }
     const int rows_max = grouped ? a->max_slot_rows : a->rows;
     if (path == 1) {

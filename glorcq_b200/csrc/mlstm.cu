@@ -12,13 +12,9 @@
 //     Every float operand of a tensor-core product (scaled keys, state, weights) goes in as a sum of two bf16 numbers.
 // State layout: S (B, H, slices, D, 32), n (B, H, slices, D) and m (B, H, slices), the last two once per 32-column
 // slice, so that no CTA reads what another one is about to write.
-#include "dense_common.cuh"
+#include "recurrent.cuh"
 
 namespace glq {
-
-constexpr int kSl = 32;            // value columns of a slice
-constexpr int kL = 64;             // positions of a chunk
-constexpr int kSegment = 4096;     // positions the chunk form takes at a time (bounds its workspace)
 
 struct MlParams {
     const void* qkvg;
@@ -50,59 +46,13 @@ __device__ __forceinline__ float log_f(const MlParams& p, size_t row, int h) {
     return fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
 }
 
-__device__ __forceinline__ void ld4(const float* p, float (&v)[4]) {
-    const float4 a = *reinterpret_cast<const float4*>(p);
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w;
-}
-__device__ __forceinline__ void ld4(const bf16* p, float (&v)[4]) {
-    const uint2 a = *reinterpret_cast<const uint2*>(p);
-    v[0] = bf_lo(a.x), v[1] = bf_hi(a.x), v[2] = bf_lo(a.y), v[3] = bf_hi(a.y);
-}
-__device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
-__device__ __forceinline__ void st4(bf16* p, float a, float b, float c, float d) {
-    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf2(a, b), pack_bf2(c, d));
-}
-
-// one warp: out = rms_norm(o) * w * sigmoid(g) for V <= 128 U values, four per lane and step, all requested before the sum
-template <typename T, int U>
-__device__ __forceinline__ void norm_gate_row(const float* __restrict__ o, const T* __restrict__ g, const float* __restrict__ w,
-                                              T* __restrict__ out, int V, float eps, int lane) {
-    float4 x[U];
-    float gv[U][4], ss = 0.f;
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-        const int v = (u * 32 + lane) * 4;
-        x[u] = v < V ? *reinterpret_cast<const float4*>(o + v) : make_float4(0, 0, 0, 0);
-        if (v < V) ld4(g + v, gv[u]);
-    }
-#pragma unroll
-    for (int u = 0; u < U; ++u) ss += x[u].x * x[u].x + x[u].y * x[u].y + x[u].z * x[u].z + x[u].w * x[u].w;
-    const float inv = 1.f / sqrtf(warp_sum(ss) / V + eps);
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-        const int v = (u * 32 + lane) * 4;
-        if (v < V) {
-            const float4 wv = *reinterpret_cast<const float4*>(w + v);
-            st4(out + v, x[u].x * inv * wv.x * sigmoid_f(gv[u][0]), x[u].y * inv * wv.y * sigmoid_f(gv[u][1]),
-                x[u].z * inv * wv.z * sigmoid_f(gv[u][2]), x[u].w * inv * wv.w * sigmoid_f(gv[u][3]));
-        }
-    }
-}
-
 // one row of head h: out = rms_norm(o) * w * sigmoid(g); one warp
 template <typename T>
 __device__ __forceinline__ void head_norm_gate(const MlParams& p, size_t row, int h, int lane) {
     const float* o = p.o + row * p.H * p.V + (size_t)h * p.V;
     const T* g = reinterpret_cast<const T*>(p.qkvg) + row * p.ldp + (size_t)p.H * (2 * p.D + p.V) + (size_t)h * p.V;
     T* out = reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V;
-    if (p.V % 4 == 0 && p.V <= 512 && p.vec4) return norm_gate_row<T, 4>(o, g, p.norm_w + (size_t)h * p.V, out, p.V, p.eps, lane);
-    float ss = 0.f;
-    for (int v = lane; v < p.V; v += 32) {
-        const float x = o[v];
-        ss += x * x;
-    }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / p.V + p.eps);
-    for (int v = lane; v < p.V; v += 32) out[v] = from_f<T>(o[v] * inv * p.norm_w[h * p.V + v] * sigmoid_f(to_f(g[v])));
+    norm_gate<T>(o, g, p.norm_w + (size_t)h * p.V, GLQ_GATE_SIGMOID, out, p.V, p.eps, p.vec4, lane);
 }
 
 template <typename T>
@@ -299,13 +249,6 @@ constexpr int kTd = 64, kLd = 72;        // tile width, row stride of a 64-wide 
 constexpr int kKb = 4 * 4 * 64 * 16;     // bytes of a chunk's key operand for 64 channels
 constexpr int kStStages = 4;
 constexpr int kStStage = kKb + kL * kLd * 2 + kTd * 4;   // bytes: key operand, values, key sums
-
-// 8x8 block of 16-bit values held row-wise across a warp -> column-wise
-__device__ __forceinline__ uint32_t transpose8(uint32_t v) {
-    uint32_t r;
-    asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
-    return r;
-}
 
 // Scratch layout of a chunk's starting state: blocks of 16 rows (d) x 8 columns (v) as the fragments the output kernel's
 // products take, [d / 16][v / 8][lane] of uint4 = (first part rows 0-7, rows 8-15, second part rows 0-7, rows 8-15).

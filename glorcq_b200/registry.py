@@ -19,6 +19,11 @@ def _zokunex(path, device, dtype):
     return ZokunexDecoder.from_pretrained(path, device, dtype or torch.bfloat16)
 
 
+def _femirax(path, device, dtype):
+    from .femirax import FemiraxDecoder
+    return FemiraxDecoder.from_pretrained(path, device, dtype or torch.bfloat16)
+
+
 def _quantized(path, device, dtype):
     if dtype not in (None, torch.float16):
         raise UnsupportedDtype("the quantized decoders compute in float16")
@@ -30,7 +35,7 @@ class UnsupportedDtype(ValueError):
     pass
 
 
-ARCHITECTURES = {"Zokunex": _zokunex}
+ARCHITECTURES = {"Zokunex": _zokunex, "Femirax": _femirax}
 
 
 def register(name, loader):
