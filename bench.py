@@ -822,9 +822,9 @@ def main():
                          "side); default min(N, 4)")
     ap.add_argument("--replicas", action="store_true",
                     help="with --gpus N > 1: N independent copies of the model instead of expert parallelism")
-    ap.add_argument("--design", choices=["zokunex"], default=None,
-                    help="time another design of the framework beside the quantized decoder of equal size instead: decode and "
-                         "prompt rates of both, and a roofline table of the kernels (see --size, --prompt, --batch, --layers)")
+    ap.add_argument("--design", choices=["zokunex", "femirax"], default=None,
+                    help="time another design of the framework beside the closest one of equal size instead (zokunex: the quantized "
+                         "decoder, femirax: zokunex): decode and prompt rates of both, and a roofline table of the kernels (see --size, --prompt, --batch, --layers)")
     ap.add_argument("--size", choices=["small", "medium", "large"], default="medium", help="with --design")
     args = ap.parse_args()
     if args.design:
@@ -833,7 +833,7 @@ def main():
         torch.cuda.set_device(0)
         sampler = ClockSampler(0)
         sampler.start()
-        line = benchmark.run(args.size, args.prompt or 4096, max(1, args.steps), args.batch, args.layers or 8, measured_peak_gbs()[0],
+        line = benchmark.run(args.design, args.size, args.prompt or 4096, max(1, args.steps), args.batch, args.layers or 8, measured_peak_gbs()[0],
                              measured_peak_tflops()[0], kernels=not args.no_extras)
         line["clocks"] = sampler.stop()
         print(json.dumps(line), flush=True)

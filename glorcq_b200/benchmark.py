@@ -1,4 +1,5 @@
-"""Timing of the unquantized designs beside the quantized decoder at equal size (``bench.py --design``).
+"""Timing of the unquantized designs at equal size (``bench.py --design``): Zokunex beside the quantized decoder, Femirax
+beside Zokunex.
 
 Every figure is a device time (CUDA events) over launches captured in a CUDA graph whose inputs rotate over more memory
 than the L2 cache holds; weights are random.  A kernel's roofline is the slower of its algorithmic bytes at the measured
@@ -9,8 +10,8 @@ from __future__ import annotations
 
 import torch
 
-from . import dense, layers, synthetic
-from .cache import LatentState, MatrixMemoryState
+from . import _lib, dense, layers, synthetic
+from .cache import DecayState, KeyValueState, LatentState, MatrixMemoryState
 from .graph_wrapper import GLoRCQGraphWrapper
 
 ROTATE_BYTES = 400e6        # memory the inputs of a timed kernel rotate over (L2: 126 MB)
@@ -46,6 +47,40 @@ def closest_config(size, n_layers=8):
                 vocab_size=s["vocab"], num_experts=s["experts"], num_experts_per_tok=s["top"], moe_intermediate_size=s["eff"],
                 shared_expert_intermediate_size=s["ff"], norm_topk_prob=False, rms_norm_eps=1e-6, rope_theta=1e6,
                 max_position_embeddings=8192)
+
+
+# Femirax: width, ff, retention (heads, dim, vdim), attention (heads, key heads, dim), linear attention (heads, dim, vdim),
+# token side
+FEMIRAX_SIZES = {
+    "small": dict(ret=(4, 128, 256), att=(8, 2, 128), gla=(4, 128, 256), side=128, ff=1408),
+    "medium": dict(ret=(4, 256, 512), att=(16, 4, 128), gla=(4, 256, 512), side=256, ff=2816),
+    "large": dict(ret=(8, 256, 512), att=(32, 8, 128), gla=(8, 256, 512), side=256, ff=14336),
+}
+
+
+def femirax_config(size, n_layers=8):
+    s, f = SIZES[size], FEMIRAX_SIZES[size]
+    out = []
+    for l in range(n_layers):
+        H, D, V = f["ret"]
+        if l % 4 == 1:
+            h, kv, d = f["att"]
+            gh, gd, gv = f["gla"]
+            mixer = {"type": "parallel", "mixer": {"left": {"heads": h, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5,
+                                                            "rot": {"base": 1e6, "dims": d}},
+                                                   "right": {"heads": gh, "dim": gd, "vdim": gv, "tau": 16.0}}}
+        else:
+            mixer = {"type": "retention", "mixer": {"heads": H, "dim": D, "vdim": V, "decay": [1 - 2.0 ** (-5 - i) for i in range(H)],
+                                                    "rot": {"base": 1e6, "dims": D}}}
+        out.append(dict(mixer, mlp={"kind": "dense", "ff": f["ff"]}))
+    return {"architecture": "Femirax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+            "token_side": {"dim": f["side"]}, "layers": out}
+
+
+def zokunex_beside_femirax(size, n_layers=8):
+    """Zokunex with a dense feed-forward of as many weights in every layer."""
+    cfg = zokunex_config(size, n_layers)
+    return dict(cfg, layers=[dict(L, mlp={"kind": "dense", "ff": FEMIRAX_SIZES[size]["ff"] * 3 // 2}) for L in cfg["layers"]])
 
 
 def graph_time(fns, reps=5):
@@ -291,20 +326,106 @@ def like_kernels(t, size, context, T):
         t.add(f"expert block, 2-bit ({rows} rows)", sec, live * 3 * C * I * 0.28 + 3 * C * Is * 0.28 + rows * C * 4, 6.0 * rows * C * (k * I + Is))
 
 
-def whole_model(size, prompt, steps, batch, n_layers):
+def _product(t, name, rows, N, K, split, like, **kw):
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+    x = torch.randn(rows, K, device=dev).to(bf)
+    if rows <= 64:
+        W = [torch.randn(N, K, device=dev).mul_(K ** -0.5).to(bf) for _ in range(_copies(2 * N * K))]
+        sec, note = graph_time([lambda w=w: dense.matmul(x, w, split=split, **kw) for w in W]), ""
+    else:
+        W = torch.randn(N, K, device=dev).mul_(K ** -0.5).to(bf)
+        sec = graph_time([lambda: dense.matmul(x, W, split=split, **kw)] * 6)
+        note = f"; library product {graph_time([lambda: x @ W.T] * 6) * 1e6:.1f} us"
+    t.add(f"{name} ({rows} x {N} x {K}{note})", sec, 2.0 * (N * K + rows * (K + N)), 2.0 * rows * N * K, like)
+
+
+def femirax_kernels(t, size, rows, T, context):
+    """The kernels of one pass over ``rows`` = sequences * T rows; T = 1: a decode step behind ``context`` positions."""
+    dev, bf = torch.device("cuda:0"), torch.bfloat16
+    s, f = SIZES[size], FEMIRAX_SIZES[size]
+    C, B, decode, ff, E = s["width"], rows // T, T == 1, f["ff"], f["side"]
+    H, D, V = f["ret"]
+    h, kv, d = f["att"]
+    gh, gd, gv = f["gla"]
+    silu = _lib.GATE_SILU
+    _product(t, "product: retention q k v g", rows, 2 * H * (D + V), C, 2 * H * (D + V), "product: q k v gates")
+    w = (h + kv) * d + 2 * gh * (gd + gv)
+    _product(t, "product: both sides' q k v g and decay rank", rows, w + 16, C, w, "product: q k v gates")
+    _product(t, "product: gate and up, silu", rows, 2 * ff, C, 2 * ff, "product: dense up", act=_lib.ACT_SILU_GLU)
+    ids = torch.zeros(rows, dtype=torch.long, device=dev)
+    table = torch.randn(64, E, device=dev).to(bf)
+    _product(t, "product: token side gate, gelu, row of the table", rows, E, C, E, "product: small", act=_lib.ACT_GELU_TANH, mul=table, mul_row=ids)
+    _product(t, "product: token side projection", rows, C, E, 0, "product: small")
+    n = _copies(rows * C * 10)
+    xs = [torch.randn(rows, C, device=dev) for _ in range(min(n, 16))]
+    for name, K in (("feed-forward output", ff), ("retention output", H * V)):
+        nw = _copies(2 * C * K) if decode else 1
+        Ws = [torch.randn(C, K, device=dev).mul_(K ** -0.5).to(bf) for _ in range(nw)]
+        y = torch.randn(rows, K, device=dev).to(bf)
+        if decode and name.startswith("retention"):
+            o, g = torch.randn(rows, K, device=dev), y
+            sec = graph_time([lambda w=w: dense.head_norm_matmul(o, g, None, H, 1e-6, w, silu, xs[0], True) for w in Ws])
+            name += " with norm and gate"
+        else:
+            sec = graph_time([lambda i=i, w=w: dense.matmul_add(y, w, xs[i % len(xs)], True) for i, w in enumerate(Ws * (1 if decode else 6))])
+        t.add(f"product added to the residual: {name} ({rows} x {C} x {K})", sec, 2.0 * C * K + rows * (2.0 * K + 10 * C), 2.0 * rows * C * K, "product: output")
+    y1, y2, ones = torch.randn(rows, C, device=dev), torch.randn(rows, C, device=dev), torch.ones(C, device=dev)
+    sec = graph_time([lambda x=x: dense.rms_add(x, 1e-6, bf, y1, ones, norm_w=ones) for x in xs] * 2)
+    t.add(f"norm, residual, next norm ({rows} rows)", sec, rows * C * 14, 0, "norm and residual")
+    sec = graph_time([lambda x=x: dense.rms_add(x, 1e-6, bf, y1, ones, y2, ones, 0.5, ones) for x in xs] * 2)
+    t.add(f"two norms, mean, residual, next norm ({rows} rows)", sec, rows * C * 18, 0, "norm and residual")
+
+    start = torch.tensor([context - 1 if decode else 0], device=dev)
+    for name, (nh, nd, nv) in (("retention", f["ret"]), ("gated linear attention", f["gla"])):
+        qkvg, a = torch.randn(rows, 2 * nh * (nd + nv), device=dev).to(bf), torch.randn(rows, 16, device=dev)
+        q, k, v, g = qkvg.split([nh * nd, nh * nd, nh * nv, nh * nv], 1)
+        kw = dict(decay=torch.tensor([1 - 2.0 ** (-5 - i) for i in range(nh)], device=dev), start=start,
+                  rotation=layers.Rotation(nd, 1e6, False)(context + 8, dev), k_scale=nd ** -0.5) if name == "retention" else \
+            dict(gates=(a, torch.randn(nh * nd, 16, device=dev).mul_(0.25).to(bf), torch.full((nh * nd,), 4.0, device=dev), 16.0), q_scale=nd ** -0.5)
+        nw = None if name == "retention" else torch.ones(nv, device=dev)
+        states = [DecayState(B, context + 8, nh, nd, nv, dev) for _ in range(_copies(B * nh * nd * nv * 4) if decode else 4)]
+        sec = graph_time([lambda st=st: dense.decay_attention(q, k, v, g, B, T, nh, nd, nv, st, nw, 1e-6, silu, short=decode, raw=decode, **kw)
+                          for st in states])
+        if decode:
+            t.add(f"{name} step ({B} x {nh} heads, {nd} x {nv})", sec, B * nh * nd * nv * 8, 0, "mLSTM step")
+        else:
+            # per position and head: weights and weighted values inside a block of 64 (half of it visible), state read and update
+            t.add(f"{name}, blocks ({T} positions, {nh} heads, {nd} x {nv})", sec, rows * nh * (2 * nd + 3 * nv) * 2,
+                  2.0 * rows * nh * (32 * (nd + nv) + 2 * nd * nv), "mLSTM, blocks")
+
+    S = context if decode else T
+    caches = [KeyValueState(B, S, kv, d, d, dev, bf) for _ in range(_copies(B * S * kv * d * 4) if decode else 2)]
+    for c in caches:
+        c.k.normal_()
+        c.v.normal_()
+    qk = torch.randn(rows, (h + kv) * d, device=dev).to(bf)
+    rot = layers.Rotation(d, 1e6, True)(S, dev)
+    start = torch.tensor([S - 1 if decode else 0], device=dev)
+    sec = graph_time([lambda c=c: dense.gqa(qk[:, :h * d], qk[:, h * d:], qk[:, h * d:], B, T, h, kv, d, d, c, d ** -0.5, 1e-6, start,
+                                            None if decode else T, rot, True) for c in caches])
+    if decode:
+        t.add(f"attention, splits ({B} x {S} positions, {h} heads on {kv}, {d})", sec, B * S * kv * d * 4, 4.0 * B * h * S * d, "latent attention, absorbed")
+    else:
+        t.add(f"attention with norm, rotation, cache write ({T} positions, {h} heads on {kv}, {d})", sec, rows * (2 * h + 4 * kv) * d * 2,
+              2.0 * rows * T * h * d, "latent attention, prompt")
+
+
+def whole_model(design, size, prompt, steps, batch, n_layers):
     """Decode and prompt rates of the two decoders through the generation wrapper."""
     dev = torch.device("cuda:0")
     out = {}
-    for name in ("zokunex", "closest"):
-        if name == "zokunex":
-            cfg = zokunex_config(size, n_layers)
-            model = synthetic.make_zokunex(cfg, dev, seed=3)
-            nbytes = synthetic.zokunex_bytes_per_token(cfg, prompt, batch)
+    for name in ((design, "closest") if design == "zokunex" else (design, "closest (zokunex)")):
+        if name == "femirax":
+            cfg = femirax_config(size, n_layers)
+            model, nbytes = synthetic.make_femirax(cfg, dev, seed=3), synthetic.femirax_bytes_per_token(cfg, prompt, batch)
+        elif name != "closest":
+            cfg = zokunex_config(size, n_layers) if design == "zokunex" else zokunex_beside_femirax(size, n_layers)
+            model, nbytes = synthetic.make_zokunex(cfg, dev, seed=3), synthetic.zokunex_bytes_per_token(cfg, prompt, batch)
         else:
             cfg = closest_config(size, n_layers)
             model = synthetic.make_decoder(cfg, dev, seed=3)
             nbytes = None
-        vocab = cfg["vocab"] if name == "zokunex" else cfg["vocab_size"]
+        vocab = cfg["vocab_size"] if name == "closest" else cfg["vocab"]
         w = GLoRCQGraphWrapper(model, max_batch_size=batch, max_seq_len=prompt + steps + 16)
         ids = torch.randint(0, vocab, (batch, prompt), generator=torch.Generator().manual_seed(1)).to(dev)
         w.generate(ids, max_new_tokens=4)
@@ -329,21 +450,26 @@ def whole_model(size, prompt, steps, batch, n_layers):
     return out
 
 
-def run(size, prompt, steps, batch, n_layers, gbs, tflops, kernels=True):
-    line = {"design": "zokunex", "size": size, "layers": n_layers, "prompt": prompt, "batch": batch,
-            "l2": "weights of a step, and the inputs of a timed kernel, exceed L2", "models": whole_model(size, prompt, steps, batch, n_layers)}
-    d = line["models"]["zokunex"]
-    d["decode_frac_of_hbm_peak"] = round(d["decode_bytes_per_step"] / (d["decode_us_per_step"] * 1e-6) / (gbs * 1e9), 3)
+def run(design, size, prompt, steps, batch, n_layers, gbs, tflops, kernels=True):
+    line = {"design": design, "size": size, "layers": n_layers, "prompt": prompt, "batch": batch,
+            "l2": "weights of a step, and the inputs of a timed kernel, exceed L2",
+            "models": whole_model(design, size, prompt, steps, batch, n_layers)}
+    for d in line["models"].values():
+        if "decode_bytes_per_step" in d:
+            d["decode_frac_of_hbm_peak"] = round(d["decode_bytes_per_step"] / (d["decode_us_per_step"] * 1e-6) / (gbs * 1e9), 3)
     if kernels:
+        def table(fn, *args):
+            t = Table(gbs, tflops)
+            fn(t, *args)
+            return t.rows
         with torch.no_grad():
-            t = Table(gbs, tflops)
-            decode_kernels(t, size, prompt, batch)
-            line["decode_kernels"] = t.rows
-            t = Table(gbs, tflops)
-            prompt_kernels(t, size, prompt)
-            line["prompt_kernels"] = t.rows
-            t = Table(gbs, tflops)
-            like_kernels(t, size, prompt, prompt)
-            line["closest_model_kernels"] = t.rows
+            if design == "femirax":
+                line["decode_kernels"] = table(femirax_kernels, size, batch, 1, prompt)
+                line["prompt_kernels"] = table(femirax_kernels, size, prompt, prompt, prompt)
+                line["closest_model_kernels"] = table(decode_kernels, size, prompt, batch) + table(prompt_kernels, size, prompt)
+            else:
+                line["decode_kernels"] = table(decode_kernels, size, prompt, batch)
+                line["prompt_kernels"] = table(prompt_kernels, size, prompt)
+                line["closest_model_kernels"] = table(like_kernels, size, prompt, prompt)
     line["kernel_self_check"] = dense.debug_error()
     return line

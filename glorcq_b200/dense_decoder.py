@@ -95,7 +95,7 @@ class DenseDecoder(nn.Module):
         kv_len = int(cache_position[0]) + T if T > 1 else None
         if kv_len is not None and kv_len > cache.max_cache_len:
             raise ValueError(f"position {kv_len - 1} is beyond the cache's {cache.max_cache_len} positions")
-        h = self.run_layers(input_ids.reshape(-1), B, T, cache_position.to(torch.int64), kv_len, cache, trace)
+        h = self.run_layers(input_ids.contiguous().view(-1), B, T, cache_position.to(torch.int64), kv_len, cache, trace)
         if torch.is_tensor(logits_to_keep):
             h = h.view(B, T, -1)[:, logits_to_keep].reshape(-1, h.shape[1])
         elif 0 < logits_to_keep < T:

@@ -303,11 +303,11 @@ class _RandomWeights:
     def __getitem__(self, name):
         shape = self.shapes[name]
         leaf = name.split(".", 1)[-1]
-        if leaf.endswith("norm") or leaf in ("norm1", "norm2"):
+        if leaf.endswith(("norm", ".out")) or leaf in ("norm1", "norm2"):
             return torch.ones(shape, device=self.device, dtype=self.dtype)
-        gain = {"mix.f.b": 1.0, "mix.i.b": 1.0, "mlp.correction": 0.01}.get(leaf, shape[-1] ** -0.5)
+        gain = {"mix.f.b": 1.0, "mix.i.b": 1.0, "mlp.correction": 0.01, "mix.right.a2.b": 1.0}.get(leaf, shape[-1] ** -0.5)
         t = torch.randn(shape, generator=self.g, device=self.device) * gain
-        return (t + 4 if leaf == "mix.f.b" else t).to(self.dtype)
+        return (t + 4 if leaf in ("mix.f.b", "mix.right.a2.b") else t).to(self.dtype)
 
 
 def make_zokunex(cfg, device, seed=0, dtype=torch.bfloat16):
@@ -333,6 +333,27 @@ def zokunex_bytes_per_token(cfg, context, batch=1):
         elif mlp:
             r = mlp["router"]
             n += 2.0 * C * (r["experts"] + r["identity"]) + min(r["experts"], batch * r["top"]) * 4.0 * C * mlp["expert"]["ff"]
+    return int(n)
+
+
+def make_femirax(cfg, device, seed=0, dtype=torch.bfloat16):
+    """A Femirax decoder of the given configuration with random weights, built on the device."""
+    from .femirax import FemiraxDecoder, tensor_shapes
+    return FemiraxDecoder(cfg, _RandomWeights(tensor_shapes(cfg), device, seed), device, dtype)
+
+
+def femirax_bytes_per_token(cfg, context, batch=1):
+    """Bytes one decode step of `batch` sequences has to move: weights (bf16), recurrent states (read and written), cached
+    keys and values of `context` positions, and the tokens' rows of the per-layer table."""
+    from .femirax import tensor_shapes
+    import math
+    n = sum(2.0 * math.prod(s) for name, s in tensor_shapes(cfg).items() if len(s) == 2 and "embed" not in name)
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        r = m if layer["type"] == "retention" else m["right"]
+        n += batch * (8.0 * r["heads"] * r["dim"] * r["vdim"] + 2.0 * cfg["token_side"]["dim"])
+        if layer["type"] == "parallel":
+            n += batch * context * 2.0 * m["left"]["kv_heads"] * (m["left"]["dim"] + m["left"]["vdim"])
     return int(n)
 
 
