@@ -336,7 +336,7 @@ def _product(t, name, rows, N, K, split, like, **kw):
         W = torch.randn(N, K, device=dev).mul_(K ** -0.5).to(bf)
         sec = graph_time([lambda: dense.matmul(x, W, split=split, **kw)] * 6)
         note = f"; library product {graph_time([lambda: x @ W.T] * 6) * 1e6:.1f} us"
-    t.add(f"{name} ({rows} x {N} x {K}{note})", sec, 2.0 * (N * K + rows * (K + N)), 2.0 * rows * N * K, like)
+    t.add(f"{name} ({rows} x {N} x {K}{note})", sec, 2.0 * (N * K + rows * K) + rows * (2.0 * split + 4.0 * (N - split)), 2.0 * rows * N * K, like)
 
 
 def femirax_kernels(t, size, rows, T, context):

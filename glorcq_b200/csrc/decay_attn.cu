@@ -181,7 +181,7 @@ template <bool CH> struct DpCfg {
 
 // CH: decay per channel
 template <bool CH>
-__global__ void __launch_bounds__(256) decay_prep_kernel(const DaParams p) {
+__global__ void __launch_bounds__(256, 2) decay_prep_kernel(const DaParams p) {
     constexpr int LF = DpCfg<CH>::LF;
     extern __shared__ __align__(16) float dp_smem[];
     float* qf = dp_smem;                 // [64][LF] queries, later the weights
@@ -251,6 +251,9 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DaParams p) {
         for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
     const int wi = CH ? (warp < 1 ? 1 : (warp < 3 ? 2 : 3)) : (warp & 3);          // block row of this warp's weights
     const int wj = CH ? warp - wi * (wi - 1) / 2 : 2 * (warp >> 2);                // first block column
+    // CH, on the diagonal of 16 x 16 blocks: warps 6 and 7 take the lower left quarters (queries 8 .. 15, keys 0 .. 7) of two
+    // blocks each; of the 8 x 8 blocks left, a thread takes 2 x 2 pairs over half the channels
+    const int db8 = (tid >> 4) & 7, du = (tid >> 2) & 3, dt = tid & 3, dh = tid >> 7;
 
     for (int d0 = 0; d0 < p.Dp; d0 += 64) {
         __syncthreads();
@@ -377,29 +380,50 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DaParams p) {
                     mma_bf16(acc[nb], al[0], al[1], al[2], al[3], bh[0], bh[1]);
                 }
             }
-        }
-        if (CH) {
-            const int tl = tid >> 4, sl = tid & 15;
-            if (sl <= tl) {
-#pragma unroll 1
-                for (int sb = 0; sb < 4; ++sb) {
-                    const int tr = (16 * sb + tl) * LF, sr = (16 * sb + sl) * LF;
-                    float v = 0.f;
-#pragma unroll 4
-                    for (int d = 0; d < 64; d += 4) {
-                        float x[4], y[4], e[4], f[4];
-                        ld4(qf + tr + d, x);
-                        ld4(kf + sr + d, y);
-                        ld4(bf + tr + d, e);
-                        ld4(bf + sr + d, f);
+        } else if (CH) {
 #pragma unroll
-                        for (int j = 0; j < 4; ++j) v += x[j] * y[j] * ex2f(e[j] - f[j]);
+            for (int u = 0; u < 2; ++u) {
+                const int base = 16 * (2 * (warp - 6) + u);
+#pragma unroll 1
+                for (int kk = 0; kk < 4; ++kk) {
+                    uint32_t ah[2], al[2], bh[2], bl[2];
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {            // measured from the quarter's last key
+                        const int col = 16 * kk + 2 * t4 + 8 * i, aq = (base + 8 + g) * LF + col, ak = (base + g) * LF + col;
+                        const float2 r = *reinterpret_cast<const float2*>(bf + (base + 7) * LF + col);
+                        float2 x = *reinterpret_cast<const float2*>(qf + aq), e = *reinterpret_cast<const float2*>(bf + aq);
+                        split_bf2(x.x * ex2f(e.x - r.x), x.y * ex2f(e.y - r.y), ah[i], al[i]);
+                        x = *reinterpret_cast<const float2*>(kf + ak);
+                        e = *reinterpret_cast<const float2*>(bf + ak);
+                        split_bf2(x.x * ex2f(r.x - e.x), x.y * ex2f(r.y - e.y), bh[i], bl[i]);
                     }
-                    if (sb == 0) diag[0] += v;
-                    else if (sb == 1) diag[1] += v;
-                    else if (sb == 2) diag[2] += v;
-                    else diag[3] += v;
+                    // rows 0 .. 7 of the operand are zero
+                    mma_bf16(acc[u], 0u, ah[0], 0u, ah[1], bh[0], bh[1]);
+                    mma_bf16(acc[u], 0u, ah[0], 0u, ah[1], bl[0], bl[1]);
+                    mma_bf16(acc[u], 0u, al[0], 0u, al[1], bh[0], bh[1]);
                 }
+            }
+        }
+        if (CH && dt <= du) {
+            // 2 x 2 pairs of an 8 x 8 block on the diagonal, half of the channels
+            const int tr = (8 * db8 + 2 * du) * LF + 32 * dh, sr = (8 * db8 + 2 * dt) * LF + 32 * dh;
+#pragma unroll 2
+            for (int d = 0; d < 32; d += 4) {
+                float x[2][4], y[2][4], e[2][4], f[2][4];
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    ld4(qf + tr + u * LF + d, x[u]);
+                    ld4(kf + sr + u * LF + d, y[u]);
+                    ld4(bf + tr + u * LF + d, e[u]);
+                    ld4(bf + sr + u * LF + d, f[u]);
+                }
+#pragma unroll
+                for (int u = 0; u < 2; ++u)
+#pragma unroll
+                    for (int w = 0; w < 2; ++w)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)          // (a key after its query is weighed here and dropped below)
+                            diag[2 * u + w] += x[u][j] * y[w][j] * ex2f(fminf(e[u][j] - f[w][j], 0.f));
             }
         }
     }
@@ -415,9 +439,29 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DaParams p) {
             }
     }
     if (CH) {
-        const int tl = tid >> 4, sl = tid & 15;
+        // the diagonal: quarters above it are zero, the halves of the channels meet here
+        if (warp >= 6)
 #pragma unroll
-        for (int sb = 0; sb < 4; ++sb) sc[(16 * sb + tl) * LF + 16 * sb + sl] = sl <= tl ? diag[sb] : 0.f;
+            for (int u = 0; u < 2; ++u) {
+                const int base = 16 * (2 * (warp - 6) + u);
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    sc[(base + 8 + g) * LF + base + 2 * t4 + e] = acc[u][2 + e];
+                    sc[(base + g) * LF + base + 8 + 2 * t4 + e] = 0.f;
+                }
+            }
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            if (half) __syncthreads();
+            if (dh == half)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = 2 * du + (e >> 1), s = 2 * dt + (e & 1);
+                    float* at = sc + (8 * db8 + t) * LF + 8 * db8 + s;
+                    if (s > t) *at = 0.f;
+                    else *at = half ? *at + diag[e] : diag[e];
+                }
+        }
     }
     __syncthreads();
     for (int blk = warp; blk < kBlocks; blk += 8) {

@@ -36,7 +36,7 @@ struct DmParams {
     const void* mul;
     const int64_t* mul_row;
     long long ldmul;
-    int mul_rows, residual;
+    int mul_rows, residual, vec_mul;
 };
 
 struct DmSlot {
@@ -81,8 +81,88 @@ __device__ __forceinline__ uint4 dm_ldg(const uint4* p) {
                  : "l"(p));
     return v;
 }
+// parts of at most 128 U values; everything is requested before the sum
+template <int WARPS, int U>
+__device__ __forceinline__ void stage_parts(const DmParams& p, bf16* xs, int XS, int units, int share, int len, float* s_part) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, heads = p.hn_heads, V = p.K / heads;
+    const bf16* gates = reinterpret_cast<const bf16*>(p.hn_g);
+    for (int i = w; i < units * share; i += WARPS) {
+        const int u = i / share, row = u / heads, h = u % heads;
+        const int lo = (i % share) * len, hi = min(V, lo + len);
+        const float* o = p.hn_o + (size_t)row * p.K + (size_t)h * V;
+        constexpr bool AHEAD = U <= 2;   // the weights too, where registers allow
+        float4 x[U], nw[U];
+        uint2 gv[U];
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+            const int k = lo + 128 * j + 4 * lane;
+            x[j] = k < hi ? *reinterpret_cast<const float4*>(o + k) : make_float4(0, 0, 0, 0);
+            nw[j] = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (AHEAD && p.hn_w && k < hi) nw[j] = *reinterpret_cast<const float4*>(p.hn_w + (size_t)h * p.hn_wstride + k);
+            if (gates && k < hi) gv[j] = *reinterpret_cast<const uint2*>(gates + (size_t)row * p.hn_ldg + (size_t)h * V + k);
+        }
+#pragma unroll
+        for (int j = 0; j < U; ++j) ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
+        ss = warp_sum(ss);
+        if (share > 1) {             // one round: every warp has at most one part
+            if (lane == 0) s_part[w] = ss;
+            asm volatile("bar.sync 1, %0;" ::"r"(units * share * 32) : "memory");
+            ss = 0.f;
+            for (int j = 0; j < share; ++j) ss += s_part[u * share + j];
+        }
+        const float inv = 1.f / sqrtf(ss / V + p.hn_eps);
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+            const int k = lo + 128 * j + 4 * lane;
+            if (k >= hi) continue;
+            if (!AHEAD && p.hn_w) nw[j] = *reinterpret_cast<const float4*>(p.hn_w + (size_t)h * p.hn_wstride + k);
+            float4 v = make_float4(x[j].x * inv * nw[j].x, x[j].y * inv * nw[j].y, x[j].z * inv * nw[j].z, x[j].w * inv * nw[j].w);
+            if (gates) {
+                v.x *= gate_f(p.hn_gate, bf_lo(gv[j].x));
+                v.y *= gate_f(p.hn_gate, bf_hi(gv[j].x));
+                v.z *= gate_f(p.hn_gate, bf_lo(gv[j].y));
+                v.w *= gate_f(p.hn_gate, bf_hi(gv[j].y));
+            }
+            *reinterpret_cast<uint2*>(xs + (size_t)row * XS + (size_t)h * V + k) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
+        }
+    }
+}
+// Activation rows made from hn_o: RMS norm over each of hn_heads parts, times its weight, times the gate.  Warps take
+// (row, part) pairs, several to a pair when there are few; the values stay in registers between the sum and the product.
+template <int WARPS>
+__device__ __forceinline__ void stage_normed(const DmParams& p, bf16* xs, int XS, int cnt, float* s_part) {
+    const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, heads = p.hn_heads, V = p.K / heads, units = cnt * heads;
+    const bf16* gates = reinterpret_cast<const bf16*>(p.hn_g);
+    for (int i = threadIdx.x; i < (p.xrows - cnt) * (p.K / 8); i += WARPS * 32)          // rows past the last: zeros
+        *reinterpret_cast<uint4*>(xs + (size_t)(cnt + i / (p.K / 8)) * XS + 8 * (i % (p.K / 8))) = make_uint4(0, 0, 0, 0);
+    int share = 1;
+    while (2 * share * units <= WARPS) share *= 2;
+    const int len = ((V + share - 1) / share + 3) / 4 * 4;                               // of a warp's part
+    if (V % 4 == 0 && len <= 512 && p.hn_ldg % 4 == 0 && (reinterpret_cast<uintptr_t>(gates) & 7) == 0 &&
+        (reinterpret_cast<uintptr_t>(p.hn_w) & 15) == 0 && p.hn_wstride % 4 == 0) {
+        if (len <= 256) stage_parts<WARPS, 2>(p, xs, XS, units, share, len, s_part);
+        else stage_parts<WARPS, 4>(p, xs, XS, units, share, len, s_part);
+        return;
+    }
+    for (int u = w; u < units; u += WARPS) {
+        const int row = u / heads, h = u % heads;
+        const float* o = p.hn_o + (size_t)row * p.K + (size_t)h * V;
+        float ss = 0.f;
+        for (int k = lane; k < V; k += 32) ss += o[k] * o[k];
+        const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
+        for (int k = lane; k < V; k += 32) {
+            float v = o[k] * inv;
+            if (p.hn_w) v *= p.hn_w[(size_t)h * p.hn_wstride + k];
+            if (gates) v *= gate_f(p.hn_gate, to_f(gates[(size_t)row * p.hn_ldg + (size_t)h * V + k]));
+            xs[(size_t)row * XS + (size_t)h * V + k] = from_f<bf16>(v);
+        }
+    }
+}
+
 // WARPS warps a CTA, SPLIT of them share one 16-row tile; DEPTH 16-byte loads per lane and row are in flight.
-template <int WARPS, int SPLIT, int DEPTH, int CTAS>
+// EXT: rows made from hn_o, or a product added to the residual.
+template <int WARPS, int SPLIT, int DEPTH, int CTAS, bool EXT>
 __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const DmParams p) {
     constexpr int TILES = WARPS / SPLIT, THREADS = WARPS * 32;
     extern __shared__ __align__(16) unsigned char dm_smem[];
@@ -94,6 +174,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
     const int XS = (chunks + 1) * 32;                              // padded activation rows: distinct banks
     bf16* xs = reinterpret_cast<bf16*>(dm_smem);
     float4* red = reinterpret_cast<float4*>(dm_smem + (size_t)p.xrows * XS * 2);
+    __shared__ float s_part[WARPS];
     const int ntiles = (p.N + 15) / 16;
     const bool plain = p.slot_index == nullptr;
     DmSlot sl{0, 0, p.rows};
@@ -125,33 +206,8 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                 pdl_wait();
                 pdl_release();
             }
-            if (p.hn_o) {
-                // rows = per-head RMS norm of hn_o, times its weight, times the gate; warp = (row, head)
-                const int V = K / p.hn_heads;
-                for (int i = w; i < p.xrows * p.hn_heads; i += WARPS) {
-                    const int row = i / p.hn_heads, k0 = (i % p.hn_heads) * V;
-                    if (row >= sl.cnt) {
-                        for (int k = k0 + lane; k < k0 + V; k += 32) xs[(size_t)row * XS + k] = from_f<bf16>(0.f);
-                        continue;
-                    }
-                    const float* o = p.hn_o + (size_t)row * K;
-                    float ss = 0.f;
-                    if (V % 4 == 0) {
-#pragma unroll 4
-                        for (int k = k0 + 4 * lane; k < k0 + V; k += 128) {
-                            const float4 v = *reinterpret_cast<const float4*>(o + k);
-                            ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-                        }
-                    } else {
-                        for (int k = k0 + lane; k < k0 + V; k += 32) ss += o[k] * o[k];
-                    }
-                    const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
-                    const bf16* gt = reinterpret_cast<const bf16*>(p.hn_g) + (size_t)row * p.hn_ldg;
-                    const float* nw = p.hn_w ? p.hn_w + (size_t)(i % p.hn_heads) * p.hn_wstride - k0 : nullptr;
-#pragma unroll 4
-                    for (int k = k0 + lane; k < k0 + V; k += 32)
-                        xs[(size_t)row * XS + k] = from_f<bf16>(o[k] * inv * (nw ? nw[k] : 1.f) * gate_f(p.hn_gate, to_f(gt[k])));
-                }
+            if (EXT && p.hn_o) {
+                stage_normed<WARPS>(p, xs, XS, sl.cnt, s_part);
                 for (int i = tid; i < p.xrows * 32; i += THREADS) {  // channels past K of the last chunk
                     const int k = K + (i & 31);
                     if (k < chunks * 32) xs[(size_t)(i >> 5) * XS + k] = from_f<bf16>(0.f);
@@ -169,6 +225,14 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
                 }
             }
             __syncthreads();
+        }
+        float prev[4] = {0.f, 0.f, 0.f, 0.f};                      // the residual's values, requested ahead of the product
+        if (EXT && p.residual && s == 0 && live) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
+                if (row < sl.cnt && n < p.N) prev[i] = p.y32[(size_t)row * p.ldy32 + n];
+            }
         }
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         const uint4* xb = reinterpret_cast<const uint4*>(xs + (size_t)min(g, p.xrows - 1) * XS) + t;   // past the rows: zeros
@@ -206,7 +270,14 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int n = tile * 16 + g + 8 * (i >> 1), row = 2 * t + (i & 1);
-                if (row < sl.cnt && n < p.N) dm_store<bf16>(p, sl.off + row, n, p.alpha * act_dyn(p.act, acc[i]));
+                if (row >= sl.cnt || n >= p.N) continue;
+                const float v = p.alpha * act_dyn(p.act, acc[i]);
+                if (!EXT || !p.residual) {
+                    dm_store<bf16>(p, sl.off + row, n, v);
+                } else {
+                    p.y32[(size_t)row * p.ldy32 + n] = prev[i] + v;
+                    if (p.y) reinterpret_cast<bf16*>(p.y)[(size_t)row * p.ldy + n] = from_f<bf16>(prev[i] + v);
+                }
             }
         }
         if (it + 1 < iters) __syncthreads();
@@ -466,9 +537,19 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
                 for (int j = 0; j < 16; ++j) f[j] = p.alpha * act_dyn(p.act, __uint_as_float(v[j]));
                 if (p.mul) {
                     const bf16* mr = dm_mul_row<bf16>(p, (int)orow) + n0;
+                    if (n0 + 16 <= p.N && p.vec_mul) {
+                        const uint4 m0 = reinterpret_cast<const uint4*>(mr)[0], m1 = reinterpret_cast<const uint4*>(mr)[1];
+                        const uint32_t mw[8] = {m0.x, m0.y, m0.z, m0.w, m1.x, m1.y, m1.z, m1.w};
 #pragma unroll
-                    for (int j = 0; j < 16; ++j)
-                        if (n0 + j < p.N) f[j] *= to_f(mr[j]);
+                        for (int j = 0; j < 8; ++j) {
+                            f[2 * j] *= bf_lo(mw[j]);
+                            f[2 * j + 1] *= bf_hi(mw[j]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            if (n0 + j < p.N) f[j] *= to_f(mr[j]);
+                    }
                 }
                 if (p.residual && n0 + 16 <= p.N && p.vec_y32 && (!p.y || p.vec_y)) {
                     float4* dst = reinterpret_cast<float4*>(p.y32 + orow * p.ldy32 + n0);
@@ -599,12 +680,13 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     p.ldmul = a->ldmul;
     p.mul_row = a->mul_row;
     p.mul_rows = a->mul_rows;
+    p.vec_mul = a->mul && al16(a->mul) && a->ldmul % 8 == 0;
     p.residual = a->residual;
     p.vec_y = a->y && al16(a->y) && a->ldy % 8 == 0;
     p.vec_y32 = a->y32 && al16(a->y32) && a->ldy32 % 4 == 0 && a->split % 4 == 0;
     const int path = glq_dense_matmul_path(a);
     if (a->hn_o) {
-        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !a->hn_g || !al16(a->hn_o)) return GLQ_ERR_ARG;
+        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !al16(a->hn_o)) return GLQ_ERR_ARG;
         p.hn_o = a->hn_o;
         p.hn_g = a->hn_g;
         p.hn_w = a->hn_w;
@@ -625,11 +707,15 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
         // measured on 1 x N x K products of 6 to 25 MB: many tiles walk over resident CTAs; a few per SM fit one wave of
         // small CTAs; less than one per SM takes deep loads, with sixteen warps on a tile when rows are long
         const long work = (long)tiles * p.slots;
-        if (work > 12L * sms) return go(dense_stream_kernel<8, 4, 8, 2>, 8, std::min(cdiv_i(tiles, 2), 2 * sms));
-        if (work > 3L * sms && a->K < 4096) return go(dense_stream_kernel<4, 4, 8, 4>, 4, tiles);
-        if (work > sms) return go(dense_stream_kernel<8, 8, 4, 3>, 8, tiles);
-        if (a->K >= 4096) return go(dense_stream_kernel<16, 16, 8, 1>, 16, tiles);
-        return go(dense_stream_kernel<8, 8, 8, 2>, 8, tiles);
+        auto pick = [&](auto ext) {
+            constexpr bool EXT = decltype(ext)::value;
+            if (work > 12L * sms) return go(dense_stream_kernel<8, 4, 8, 2, EXT>, 8, std::min(cdiv_i(tiles, 2), 2 * sms));
+            if (work > 3L * sms && a->K < 4096) return go(dense_stream_kernel<4, 4, 8, 4, EXT>, 4, tiles);
+            if (work > sms) return go(dense_stream_kernel<8, 8, 4, 3, EXT>, 8, tiles);
+            if (a->K >= 2304) return go(dense_stream_kernel<16, 16, 8, 1, EXT>, 16, tiles);
+            return go(dense_stream_kernel<8, 8, 8, 2, EXT>, 8, tiles);
+        };
+        return a->hn_o || a->residual ? pick(std::true_type()) : pick(std::false_type());
     }
     if (path == 2) {
         const void* xa = a->x;

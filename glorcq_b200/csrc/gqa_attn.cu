@@ -47,13 +47,32 @@ __device__ __forceinline__ void head_row8(const GaParams& p, const bf16* x, int 
             const float* cs = p.cos_t + pos * half;
             const float* sn = p.sin_t + pos * half;
             if (p.rot_pairs) {
+                float c[4] = {1.f, 1.f, 1.f, 1.f}, s[4] = {0.f, 0.f, 0.f, 0.f};
+                if (half % 4 == 0) {       // whole vectors: all four pairs are turned
+                    ld4(cs + e / 2, c);
+                    ld4(sn + e / 2, s);
+                } else {
 #pragma unroll
-                for (int j = 0; j < 4; ++j)
-                    if (e + 2 * j < p.rot_dims) {
-                        const float c = cs[e / 2 + j], s = sn[e / 2 + j], a = v[2 * j], o = v[2 * j + 1];
-                        v[2 * j] = a * c - o * s;
-                        v[2 * j + 1] = o * c + a * s;
-                    }
+                    for (int j = 0; j < 4; ++j)
+                        if (e + 2 * j < p.rot_dims) c[j] = cs[e / 2 + j], s[j] = sn[e / 2 + j];
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float a = v[2 * j], o = v[2 * j + 1];
+                    v[2 * j] = a * c[j] - o * s[j];
+                    v[2 * j + 1] = o * c[j] + a * s[j];
+                }
+            } else if (half % 8 == 0) {
+                const bool second = e >= half;
+                float u[8], c[4], s[4];
+                gld8(x + (second ? e - half : e + half), u);
+#pragma unroll
+                for (int q = 0; q < 2; ++q) {
+                    ld4(cs + (second ? e - half : e) + 4 * q, c);
+                    ld4(sn + (second ? e - half : e) + 4 * q, s);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) v[4 * q + j] = v[4 * q + j] * c[j] + (second ? u[4 * q + j] : -u[4 * q + j]) * s[j];
+                }
             } else {
 #pragma unroll
                 for (int j = 0; j < 8; ++j) v[j] = rotated(x, e + j, p.rot_dims, 0, cs, sn);
@@ -74,34 +93,35 @@ __device__ __forceinline__ uint4 pack8(const float (&v)[8]) {
     return make_uint4(pack_bf2(v[0], v[1]), pack_bf2(v[2], v[3]), pack_bf2(v[4], v[5]), pack_bf2(v[6], v[7]));
 }
 
-// prompt: rows of H query heads (in place), G key heads (into the cache) and G value heads (copied), 16-byte accesses
-__global__ void __launch_bounds__(256) gqa_prep_vec_kernel(const GaParams p, int gl) {
+// prompt: rows of H query heads (in place) and G key heads (into the cache), 16-byte accesses; a warp takes 32 / gl heads of
+// a row at a time, the key heads' values on the way.  Work is row by row over (row, heads) tasks.
+__global__ void __launch_bounds__(256, 5) gqa_prep_vec_kernel(const GaParams p, int gl) {
     pdl_wait();
     pdl_release();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = 32 / gl, li = lane % gl, e = 8 * li;
-    const size_t row = blockIdx.x, b = row / p.T;
-    const long long pos = *p.start + (long long)(row % p.T);
-    if (pos < 0 || pos >= p.max_len) return;
-    const int heads = p.H + p.G;
-    const size_t crow = (b * p.max_len + pos) * p.G;
-    for (int h0 = warp * per; h0 < heads; h0 += 8 * per) {
-        const int h = h0 + lane / gl;
+    const int lane = threadIdx.x & 31, per = 32 / gl, li = lane % gl, e = 8 * li;
+    const int heads = p.H + p.G, tasks = (heads + per - 1) / per;
+    const long long start = *p.start, total = (long long)p.B * p.T * tasks;
+    for (long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5); i < total; i += (long long)gridDim.x * 8) {
+        const size_t row = (size_t)(i / tasks), b = row / p.T;
+        const int h = (int)(i % tasks) * per + lane / gl;
+        const long long pos = start + (long long)(row % p.T);
+        if (pos < 0 || pos >= p.max_len) continue;
         const bool live = h < heads, isq = h < p.H;
-        const int hh = live ? h : 0;
-        const bf16* src = isq || !live ? reinterpret_cast<const bf16*>(p.q) + row * p.ldp + (size_t)hh * p.D
-                                       : reinterpret_cast<const bf16*>(p.k) + row * p.ldp + (size_t)(hh - p.H) * p.D;
+        const bf16* src = reinterpret_cast<const bf16*>(isq || !live ? p.q : p.k) + row * p.ldp + (size_t)(!live ? 0 : (isq ? h : h - p.H)) * p.D;
         float v[8];
         head_row8(p, src, e, gl, (size_t)pos, v);
         __syncwarp();                      // all lanes have read the row that is replaced
-        if (live && e < p.D) {
-            bf16* dst = isq ? reinterpret_cast<bf16*>(p.q) + row * p.ldp + (size_t)h * p.D + e
-                            : reinterpret_cast<bf16*>(p.kc) + (crow + h - p.H) * p.D + e;
-            *reinterpret_cast<uint4*>(dst) = pack8(v);
+        if (!live) continue;
+        if (isq) {
+            if (e < p.D) *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.q) + row * p.ldp + (size_t)h * p.D + e) = pack8(v);
+            continue;
         }
+        const size_t crow = (b * p.max_len + pos) * p.G + h - p.H;
+        if (e < p.D) *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.kc) + crow * p.D + e) = pack8(v);
+        const bf16* vs = reinterpret_cast<const bf16*>(p.v) + row * p.ldp + (size_t)(h - p.H) * p.V;
+        for (int c = e; c < p.V; c += 8 * gl)
+            *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.vc) + crow * p.V + c) = *reinterpret_cast<const uint4*>(vs + c);
     }
-    const bf16* vs = reinterpret_cast<const bf16*>(p.v) + row * p.ldp;
-    bf16* vd = reinterpret_cast<bf16*>(p.vc) + crow * p.V;
-    for (int i = threadIdx.x; i < p.G * p.V / 8; i += 256) reinterpret_cast<uint4*>(vd)[i] = reinterpret_cast<const uint4*>(vs)[i];
 }
 
 // the same for any type and size: one warp per head, its row staged in shared memory
@@ -262,7 +282,7 @@ __global__ void __launch_bounds__(kGdWarps * 32) gqa_decode_kernel(const GaParam
             }
         }
         // new positions that lie in this split (every row tile of the head writes the same values)
-        for (int i0 = 0; i0 < p.T; i0 += kGdWarps * per_w) {
+        for (int i0 = 0; i0 < p.T && total > lo * kGdTile && start < hi * kGdTile; i0 += kGdWarps * per_w) {
             const int i = i0 + warp * per_w + lane / gl, pos = start + i;
             const bool live = i < p.T && pos >= lo * kGdTile && pos < hi * kGdTile;
             const size_t row = (size_t)b * p.T + (i < p.T ? i : 0);
@@ -422,31 +442,65 @@ __global__ void __launch_bounds__(kGdWarps * 32) gqa_decode_kernel(const GaParam
 
 // merges the splits of one row
 constexpr int kGdMaxSplits = 128;
-__global__ void __launch_bounds__(128) gqa_combine_kernel(const GaParams p) {
+constexpr int kGcThreads = 256;
+__global__ void __launch_bounds__(kGcThreads) gqa_combine_kernel(const GaParams p) {
     __shared__ float sw[kGdMaxSplits], red[32];
+    __shared__ __align__(16) float part[kGcThreads * 4];
     pdl_wait();
     pdl_release();
     const int tid = threadIdx.x, h = blockIdx.y, kh = h / p.group;
     const size_t row = blockIdx.x, b = row / p.T;
     const int ri = (int)(row % p.T) * p.group + h % p.group, r = ri % 16;
-    const size_t part = (((size_t)b * p.G + kh) * p.tiles + ri / 16) * p.splits;
-    const float2 ml = tid < p.splits ? p.pml[(part + tid) * 16 + r] : make_float2(-INFINITY, 0.f);
+    const size_t first = (((size_t)b * p.G + kh) * p.tiles + ri / 16) * p.splits;
+    const float2 ml = tid < p.splits ? p.pml[(first + tid) * 16 + r] : make_float2(-INFINITY, 0.f);
     float mx = ml.x;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
     if ((tid & 31) == 0) red[tid >> 5] = mx;
     __syncthreads();
-    mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+#pragma unroll
+    for (int i = 0; i < kGcThreads / 32; ++i) mx = fmaxf(mx, red[i]);
     const float w = ml.x == -INFINITY ? 0.f : ex2(ml.x - mx);
     const float inv = 1.f / block_sum(w * ml.y, red);
-    sw[tid] = w * inv;
+    if (tid < kGdMaxSplits) sw[tid] = w * inv;
     __syncthreads();
-    for (int v = tid; v < p.V; v += 128) {
-        float a = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < p.splits; ++s)
-            if (sw[s] != 0.f) a += sw[s] * p.po[((part + s) * 16 + r) * p.V + v];
-        reinterpret_cast<bf16*>(p.out)[row * p.H * p.V + (size_t)h * p.V + v] = from_f<bf16>(a);
+    // four columns a thread, the groups of threads share the splits; a split without weight has not been written
+    const int vq = p.V / 4, groups = kGcThreads / vq, grp = tid / vq, v = 4 * (tid % vq);
+    float4 a = make_float4(0, 0, 0, 0);
+    if (grp < groups) {
+        const float* po = p.po + (first * 16 + r) * p.V + v;
+        for (int s0 = grp; s0 < p.splits; s0 += 8 * groups) {
+            float4 x[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int s = min(s0 + i * groups, p.splits - 1);
+                x[i] = *reinterpret_cast<const float4*>(po + (size_t)16 * s * p.V);
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int s = s0 + i * groups;
+                const float ws = s < p.splits ? sw[s] : 0.f;
+                if (ws != 0.f) {
+                    a.x += ws * x[i].x;
+                    a.y += ws * x[i].y;
+                    a.z += ws * x[i].z;
+                    a.w += ws * x[i].w;
+                }
+            }
+        }
+    }
+    *reinterpret_cast<float4*>(part + 4 * tid) = a;
+    __syncthreads();
+    if (tid < vq) {
+        for (int i = 1; i < groups; ++i) {
+            const float4 x = *reinterpret_cast<const float4*>(part + 4 * (tid + i * vq));
+            a.x += x.x;
+            a.y += x.y;
+            a.z += x.z;
+            a.w += x.w;
+        }
+        *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(p.out) + row * p.H * p.V + (size_t)h * p.V + v) =
+            make_uint2(pack_bf2(a.x, a.y), pack_bf2(a.z, a.w));
     }
 }
 
@@ -460,7 +514,7 @@ static bool ga_sizes_ok(const glq_gqa_t* a) {
 }
 // rows of whole 16-byte vectors
 static bool ga_vec(const glq_gqa_t* a) {
-    return a->dtype == GLQ_DT_BF16 && a->D % 8 == 0 && a->V % 8 == 0 && a->D <= 256 && a->ldp % 8 == 0 && al16(a->q) && al16(a->k) &&
+    return a->dtype == GLQ_DT_BF16 && a->D % 8 == 0 && a->V % 8 == 0 && a->D <= 256 && a->ldp % 8 == 0 && al16(a->q) && al16(a->k) && al16(a->cos_t) && al16(a->sin_t) &&
            al16(a->v) && al16(a->kc) && al16(a->vc) && al16(a->out);
 }
 static int ga_lanes(int D) {
@@ -567,12 +621,12 @@ extern "C" int glq_gqa(const glq_gqa_t* a, void* stream) {
         else if (dv == 128) st = dn_launch(gqa_decode_kernel<128>, grid, kGdWarps * 32, z.q_bytes + z.ring, stream, p, gl);
         else st = dn_launch(gqa_decode_kernel<256>, grid, kGdWarps * 32, z.q_bytes + z.ring, stream, p, gl);
         if (st != GLQ_OK || p.splits == 1) return st;
-        return dn_launch(gqa_combine_kernel, dim3(a->B * a->T, a->H), 128, 0, stream, p);
+        return dn_launch(gqa_combine_kernel, dim3(a->B * a->T, a->H), kGcThreads, 0, stream, p);
     }
     const dim3 rows(a->B * a->T);
     if (form == 2) {
         if (a->S < a->T || a->S > a->max_len) return GLQ_ERR_ARG;
-        if ((st = dn_launch(gqa_prep_vec_kernel, rows, 256, 0, stream, p, ga_lanes(a->D))) != GLQ_OK) return st;
+        if ((st = dn_launch(gqa_prep_vec_kernel, dim3(std::min<long>(5L * dn_sms(), cdiv_i((long)a->B * a->T * (a->H + a->G), 8))), 256, 0, stream, p, ga_lanes(a->D))) != GLQ_OK) return st;
         return gqa_prompt(a, p, stream);
     }
     const size_t ps = (size_t)4 * a->D * 4, gs = (size_t)(a->D + a->V) * 4;

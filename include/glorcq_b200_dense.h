@@ -65,8 +65,8 @@ typedef struct glq_dense_mm {
     int64_t ldy32;
     void* gather;          /* (rows, K) scratch for entry_row on the tensor-core path, or NULL when entry_row is */
     /* up to 8 rows, bf16, instead of x: row = rms_norm over each of hn_heads equal parts of hn_o (rows, K) float, times
-     * hn_w (one part, hn_wstride further for every next head; NULL: 1), times the gate of hn_g (rows, K) bf16, row stride
-     * hn_ldg, through hn_gate */
+     * hn_w (one part, hn_wstride further for every next head; NULL: 1), times the gate of hn_g (rows, K) bf16 (NULL: 1),
+     * row stride hn_ldg, through hn_gate */
     const float* hn_o;
     const void* hn_g;
     int64_t hn_ldg;
