@@ -134,7 +134,7 @@ class DenseMM(C.Structure):
                [("alpha", C.c_float)] + [(f, vp) for f in ("slot_index", "n_slots", "slot_count", "slot_offset", "entry_row", "x")] + \
                [("ldx", C.c_int64), ("W", vp), ("ldw", C.c_int64), ("y", vp), ("ldy", C.c_int64), ("y32", vp), ("ldy32", C.c_int64), ("gather", vp),
                 ("hn_o", vp), ("hn_g", vp), ("hn_ldg", C.c_int64), ("hn_w", vp), ("hn_heads", C.c_int32), ("hn_eps", C.c_float),
-                ("hn_wstride", C.c_int32), ("hn_gate", C.c_int32), ("mul", vp), ("ldmul", C.c_int64), ("mul_row", vp),
+                ("mul", vp), ("ldmul", C.c_int64), ("mul_row", vp),
                 ("mul_rows", C.c_int32), ("residual", C.c_int32)]
 
 

@@ -362,12 +362,7 @@ def femirax_kernels(t, size, rows, T, context):
         nw = _copies(2 * C * K) if decode else 1
         Ws = [torch.randn(C, K, device=dev).mul_(K ** -0.5).to(bf) for _ in range(nw)]
         y = torch.randn(rows, K, device=dev).to(bf)
-        if decode and name.startswith("retention"):
-            o, g = torch.randn(rows, K, device=dev), y
-            sec = graph_time([lambda w=w: dense.head_norm_matmul(o, g, None, H, 1e-6, w, silu, xs[0], True) for w in Ws])
-            name += " with norm and gate"
-        else:
-            sec = graph_time([lambda i=i, w=w: dense.matmul_add(y, w, xs[i % len(xs)], True) for i, w in enumerate(Ws * (1 if decode else 6))])
+        sec = graph_time([lambda i=i, w=w: dense.matmul_add(y, w, xs[i % len(xs)], True) for i, w in enumerate(Ws * (1 if decode else 6))])
         t.add(f"product added to the residual: {name} ({rows} x {C} x {K})", sec, 2.0 * C * K + rows * (2.0 * K + 10 * C), 2.0 * rows * C * K, "product: output")
     y1, y2, ones = torch.randn(rows, C, device=dev), torch.randn(rows, C, device=dev), torch.ones(C, device=dev)
     sec = graph_time([lambda x=x: dense.rms_add(x, 1e-6, bf, y1, ones, norm_w=ones) for x in xs] * 2)
@@ -384,10 +379,10 @@ def femirax_kernels(t, size, rows, T, context):
             dict(gates=(a, torch.randn(nh * nd, 16, device=dev).mul_(0.25).to(bf), torch.full((nh * nd,), 4.0, device=dev), 16.0), q_scale=nd ** -0.5)
         nw = None if name == "retention" else torch.ones(nv, device=dev)
         states = [DecayState(B, context + 8, nh, nd, nv, dev) for _ in range(_copies(B * nh * nd * nv * 4) if decode else 4)]
-        sec = graph_time([lambda st=st: dense.decay_attention(q, k, v, g, B, T, nh, nd, nv, st, nw, 1e-6, silu, short=decode, raw=decode, **kw)
+        sec = graph_time([lambda st=st: dense.decay_attention(q, k, v, g, B, T, nh, nd, nv, st, nw, 1e-6, silu, short=decode, **kw)
                           for st in states])
         if decode:
-            t.add(f"{name} step ({B} x {nh} heads, {nd} x {nv})", sec, B * nh * nd * nv * 8, 0, "mLSTM step")
+            t.add(f"{name} step with norm and gate ({B} x {nh} heads, {nd} x {nv})", sec, B * nh * nd * nv * 8, 0, "mLSTM step")
         else:
             # per position and head: weights and weighted values inside a block of 64 (half of it visible), state read and update
             t.add(f"{name}, blocks ({T} positions, {nh} heads, {nd} x {nv})", sec, rows * nh * (2 * nd + 3 * nv) * 2,

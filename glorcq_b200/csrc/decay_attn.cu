@@ -5,8 +5,8 @@
 // linear attention; Yang et al., "Gated Linear Attention Transformers with Hardware-Efficient Training").  Queries and
 // keys may be turned by their position and scaled first; everything behind the projections is float.
 // Two forms of the same recurrence:
-//   * step: the recurrence itself, one position after the other; a CTA owns 32 value columns of a head.  Norm and gate go
-//     into the staging of the output product of a decode step (dense_mm.cu), or are a launch of their own.
+//   * step: the recurrence itself, one position after the other; a CTA owns 32 value columns of a head, and the CTAs of a
+//     head are a cluster that norms and gates its output (heads of up to 512 columns; else a launch of its own).
 //   * chunk: 64 positions at a time on the tensor cores.  With b_t the running sum of log alpha inside a chunk,
 //       o_t = (q_t e^{b_t})^T S_start + sum_{s <= t} A_ts v_s,  A_ts = sum_d q_td k_sd e^{b_td - b_sd},
 //       S_end = diag(e^{b_end}) S_start + sum_s (k_s e^{b_end - b_s}) v_s^T.
@@ -55,6 +55,12 @@ __device__ __forceinline__ float ex2f(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+constexpr int kMaxCluster = 16;
+// a float into the shared memory of CTA `rank` of the cluster, at this CTA's address `addr`
+__device__ __forceinline__ void st_cluster(uint32_t addr, int rank, float v) {
+    asm volatile("{\n .reg .b32 r;\n mapa.shared::cluster.u32 r, %0, %1;\n st.shared::cluster.f32 [r], %2;\n}\n" ::"r"(addr), "r"(rank), "f"(v)
+                 : "memory");
+}
 __device__ __forceinline__ size_t da_pos(const DaParams& p, int t) {
     const long long pos = *p.start + t;
     return (size_t)(pos < 0 ? 0 : (pos >= p.max_len ? p.max_len - 1 : pos));
@@ -67,13 +73,14 @@ __device__ __forceinline__ void da_norm_gate(const DaParams& p, size_t row, int 
                  reinterpret_cast<T*>(p.out) + row * p.H * p.V + (size_t)h * p.V, p.V, p.eps, p.vec4, lane);
 }
 
-template <typename T>
+// CL: the slices of a head are one cluster, which norms and gates the head's output and stores it in T
+template <typename T, bool CL>
 __global__ void __launch_bounds__(256) decay_step_kernel(const DaParams p) {
     extern __shared__ float da_smem[];
     float* sq = da_smem;                 // [D]
     float* sk = sq + p.D;                // [D]
     float* sa = sk + p.D;                // [D]
-    __shared__ float sv[kSl], part[8][kSl];
+    __shared__ float sv[kSl], part[8][kSl], s_ss[2][kMaxCluster];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int sl = blockIdx.x, h = blockIdx.y % p.H, b = blockIdx.y / p.H;
     const int D = p.D, V = p.V, v0 = sl * kSl, vw = min(kSl, V - v0);
@@ -157,11 +164,33 @@ __global__ void __launch_bounds__(256) decay_step_kernel(const DaParams p) {
         }
         if (lane < 8) *reinterpret_cast<float4*>(&part[warp][cc]) = acc;
         __syncthreads();
-        if (tid < vw) {
-            float num = 0.f;
+        if constexpr (!CL) {
+            if (tid < vw) {
+                float num = 0.f;
 #pragma unroll
-            for (int w = 0; w < 8; ++w) num += part[w][tid];
-            p.o[row * p.H * V + (size_t)h * V + v0 + tid] = num;
+                for (int w = 0; w < 8; ++w) num += part[w][tid];
+                p.o[row * p.H * V + (size_t)h * V + v0 + tid] = num;
+            }
+        } else {
+            float num = 0.f, gv = 0.f, nw = 1.f;
+            if (warp == 0) {
+                if (tid < vw) {
+                    gv = to_f(reinterpret_cast<const T*>(p.g)[row * p.ldp + (size_t)h * V + v0 + tid]);
+                    if (p.norm_w) nw = p.norm_w[(size_t)h * p.norm_stride + v0 + tid];
+#pragma unroll
+                    for (int w = 0; w < 8; ++w) num += part[w][tid];
+                }
+                const float ss = warp_sum(num * num);
+                if (lane < p.slices) st_cluster(smem_u32(&s_ss[t & 1][sl]), lane, ss);     // to the CTA of every slice
+            }
+            // a slot is written again two positions later, behind a barrier that follows its reads
+            asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
+            if (tid < vw) {
+                float ss = 0.f;
+                for (int i = 0; i < p.slices; ++i) ss += s_ss[t & 1][i];
+                const float inv = 1.f / sqrtf(ss / V + p.eps);
+                reinterpret_cast<T*>(p.out)[row * p.H * V + (size_t)h * V + v0 + tid] = from_f<T>(num * inv * nw * gate_f<T>(p.gate, gv));
+            }
         }
     }
 }
@@ -694,8 +723,8 @@ __global__ void __launch_bounds__(128, 3) decay_out_kernel(const DaParams p) {
                 if (v < p.V) {
                     const uint32_t gv = *reinterpret_cast<const uint32_t*>(gr + v);
                     const float w0 = w ? w[v] : 1.f, w1 = w ? w[v + 1] : 1.f;
-                    *reinterpret_cast<uint32_t*>(out + v) = pack_bf2(acc[j][2 * e] * inv * w0 * gate_f(p.gate, bf_lo(gv)),
-                                                                     acc[j][2 * e + 1] * inv * w1 * gate_f(p.gate, bf_hi(gv)));
+                    *reinterpret_cast<uint32_t*>(out + v) = pack_bf2(acc[j][2 * e] * inv * w0 * gate_f<bf16>(p.gate, bf_lo(gv)),
+                                                                     acc[j][2 * e + 1] * inv * w1 * gate_f<bf16>(p.gate, bf_hi(gv)));
                 }
             }
         } else {
@@ -750,7 +779,7 @@ extern "C" size_t glq_decay_workspace_bytes(const glq_decay_t* a) { return da_ws
 static int da_params(const glq_decay_t* a, DaParams& p) {
     if (!a || a->B <= 0 || a->T < 0 || a->H <= 0 || a->D <= 0 || a->V <= 0 || a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->D)
         return GLQ_ERR_ARG;
-    if (!a->q || !a->k || !a->v || !a->g || !a->S || !a->o) return GLQ_ERR_ARG;
+    if (!a->q || !a->k || !a->v || !a->g || !a->S || !a->o || !a->out) return GLQ_ERR_ARG;
     if (!a->decay && (!a->a || !a->a2 || !a->a2b || a->rank <= 0 || !(a->tau > 0.f))) return GLQ_ERR_ARG;
     if (a->rot_dims && (!a->start || !a->cos_t || !a->sin_t || a->max_len <= 0)) return GLQ_ERR_ARG;
     if (a->dtype != GLQ_DT_BF16 && a->dtype != GLQ_DT_F32) return GLQ_ERR_ARG;
@@ -799,6 +828,7 @@ static int da_norm(const DaParams& p, int dtype, void* stream) {
     return dn_launch(decay_norm_kernel<float>, grid, 256, 0, stream, p);
 }
 
+constexpr int kClusterSteps = 64;        // longer passes norm all rows in a launch of their own
 extern "C" int glq_decay_step(const glq_decay_t* a, void* stream) {
     DaParams p{};
     int st = da_params(a, p);
@@ -806,9 +836,13 @@ extern "C" int glq_decay_step(const glq_decay_t* a, void* stream) {
     if (p.T == 0) return GLQ_OK;
     const dim3 grid(p.slices, p.B * p.H);
     const size_t smem = (size_t)3 * p.D * 4;
-    if (a->dtype == GLQ_DT_BF16) st = dn_launch(decay_step_kernel<bf16>, grid, 256, smem, stream, p);
-    else st = dn_launch(decay_step_kernel<float>, grid, 256, smem, stream, p);
-    if (st != GLQ_OK || !p.out) return st;
+    if (p.slices <= kMaxCluster && p.T <= kClusterSteps) {
+        if (a->dtype == GLQ_DT_BF16) return dn_launch_cluster(p.slices, decay_step_kernel<bf16, true>, grid, 256, smem, stream, p);
+        return dn_launch_cluster(p.slices, decay_step_kernel<float, true>, grid, 256, smem, stream, p);
+    }
+    if (a->dtype == GLQ_DT_BF16) st = dn_launch(decay_step_kernel<bf16, false>, grid, 256, smem, stream, p);
+    else st = dn_launch(decay_step_kernel<float, false>, grid, 256, smem, stream, p);
+    if (st != GLQ_OK) return st;
     return da_norm(p, a->dtype, stream);
 }
 
@@ -824,7 +858,7 @@ extern "C" int glq_decay_chunk(const glq_decay_t* a, void* stream) {
     if (st != GLQ_OK) return st;
     if (p.T == 0) return GLQ_OK;
     const DaWs w = da_ws(a);
-    if (!a->out || !a->workspace) return GLQ_ERR_ARG;
+    if (!a->workspace) return GLQ_ERR_ARG;
     if (a->workspace_bytes < w.total) return GLQ_ERR_WORKSPACE;
     if (!al16(a->workspace) || !al16(a->out)) return GLQ_ERR_ALIGN;
     char* ws = reinterpret_cast<char*>(a->workspace);

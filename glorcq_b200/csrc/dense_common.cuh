@@ -61,7 +61,13 @@ __device__ __forceinline__ void pdl_release() { asm volatile("griddepcontrol.lau
 
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.f / (1.f + expf(-v)); }
 
-__device__ __forceinline__ float gate_f(int gate, float v) { return gate == GLQ_GATE_SILU ? v * sigmoid_f(v) : sigmoid_f(v); }
+// the same to a few units in the last place, for results that are stored as bf16
+__device__ __forceinline__ float sigmoid_fast_f(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+template <typename T> __device__ __forceinline__ float sigmoid_t(float v) { return sizeof(T) == 2 ? sigmoid_fast_f(v) : sigmoid_f(v); }
+template <typename T> __device__ __forceinline__ float gate_f(int gate, float v) {
+    const float s = sigmoid_t<T>(v);
+    return gate == GLQ_GATE_SILU ? v * s : s;
+}
 
 template <int ACT> __device__ __forceinline__ float act_f(float z) {
     if (ACT == GLQ_ACT_RELU2) {
@@ -118,8 +124,9 @@ inline int dn_sms() {
 // Launch that may start while its predecessor drains: every kernel here calls pdl_wait() before it touches anything a
 // predecessor wrote.
 // (early = false: an ordinary launch, for a kernel whose waiting CTAs would only take room from its predecessor)
+// cluster: CTAs along x that form a cluster (1: none)
 template <typename... KArgs, typename... Args>
-inline int dn_launch_if(bool early, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+inline int dn_launch_as(bool early, int cluster, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
     static const bool pdl = std::getenv("GLQ_NO_PDL") == nullptr;
     // 48 KB without opting in is dynamic plus static shared memory; no kernel here has more than 24 KB of the latter
     if (smem > 24 * 1024) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -128,13 +135,31 @@ inline int dn_launch_if(bool early, void (*kern)(KArgs...), dim3 grid, int block
     cfg.blockDim = dim3(block);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = reinterpret_cast<cudaStream_t>(stream);
-    cudaLaunchAttribute attr{};
-    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr.val.programmaticStreamSerializationAllowed = 1;
-    cfg.attrs = &attr;
-    cfg.numAttrs = pdl && early ? 1 : 0;
+    cudaLaunchAttribute attr[2]{};
+    int n = 0;
+    if (pdl && early) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster > 1) {
+        if (cluster > 8) DN_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = (unsigned)cluster;
+        attr[n].val.clusterDim.y = attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
+    cfg.attrs = attr;
+    cfg.numAttrs = n;
     DN_CUDA(cudaLaunchKernelEx(&cfg, kern, KArgs(args)...));
     return GLQ_OK;
+}
+template <typename... KArgs, typename... Args>
+inline int dn_launch_if(bool early, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+    return dn_launch_as(early, 1, kern, grid, block, smem, stream, args...);
+}
+template <typename... KArgs, typename... Args>
+inline int dn_launch_cluster(int cluster, void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {
+    return dn_launch_as(true, cluster, kern, grid, block, smem, stream, args...);
 }
 template <typename... KArgs, typename... Args>
 inline int dn_launch(void (*kern)(KArgs...), dim3 grid, int block, size_t smem, void* stream, Args... args) {

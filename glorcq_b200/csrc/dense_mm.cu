@@ -31,7 +31,7 @@ struct DmParams {
     const void* hn_g;
     const float* hn_w;
     long long hn_ldg;
-    int hn_heads, hn_wstride, hn_gate;
+    int hn_heads;
     float hn_eps;
     const void* mul;
     const int64_t* mul_row;
@@ -69,7 +69,7 @@ template <typename T, bool MUL = true> __device__ __forceinline__ void dm_store(
     else p.y32[(size_t)row * p.ldy32 + (n - p.split)] = v;
 }
 
-__device__ __forceinline__ float dm_glu(float gate, float other) { return gate * sigmoid_f(gate) * other; }
+template <typename T> __device__ __forceinline__ float dm_glu(float gate, float other) { return gate * sigmoid_t<T>(gate) * other; }
 
 // =====================================================================================================
 // streaming kernel: up to 8 rows per slot
@@ -81,7 +81,7 @@ __device__ __forceinline__ uint4 dm_ldg(const uint4* p) {
                  : "l"(p));
     return v;
 }
-// parts of at most 128 U values; everything is requested before the sum
+// parts of at most 128 U values, which are requested before the sum and stay in registers
 template <int WARPS, int U>
 __device__ __forceinline__ void stage_parts(const DmParams& p, bf16* xs, int XS, int units, int share, int len, float* s_part) {
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, heads = p.hn_heads, V = p.K / heads;
@@ -90,17 +90,14 @@ __device__ __forceinline__ void stage_parts(const DmParams& p, bf16* xs, int XS,
         const int u = i / share, row = u / heads, h = u % heads;
         const int lo = (i % share) * len, hi = min(V, lo + len);
         const float* o = p.hn_o + (size_t)row * p.K + (size_t)h * V;
-        constexpr bool AHEAD = U <= 2;   // the weights too, where registers allow
-        float4 x[U], nw[U];
+        float4 x[U];
         uint2 gv[U];
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < U; ++j) {
             const int k = lo + 128 * j + 4 * lane;
             x[j] = k < hi ? *reinterpret_cast<const float4*>(o + k) : make_float4(0, 0, 0, 0);
-            nw[j] = make_float4(1.f, 1.f, 1.f, 1.f);
-            if (AHEAD && p.hn_w && k < hi) nw[j] = *reinterpret_cast<const float4*>(p.hn_w + (size_t)h * p.hn_wstride + k);
-            if (gates && k < hi) gv[j] = *reinterpret_cast<const uint2*>(gates + (size_t)row * p.hn_ldg + (size_t)h * V + k);
+            if (k < hi) gv[j] = *reinterpret_cast<const uint2*>(gates + (size_t)row * p.hn_ldg + (size_t)h * V + k);
         }
 #pragma unroll
         for (int j = 0; j < U; ++j) ss += x[j].x * x[j].x + x[j].y * x[j].y + x[j].z * x[j].z + x[j].w * x[j].w;
@@ -116,19 +113,14 @@ __device__ __forceinline__ void stage_parts(const DmParams& p, bf16* xs, int XS,
         for (int j = 0; j < U; ++j) {
             const int k = lo + 128 * j + 4 * lane;
             if (k >= hi) continue;
-            if (!AHEAD && p.hn_w) nw[j] = *reinterpret_cast<const float4*>(p.hn_w + (size_t)h * p.hn_wstride + k);
-            float4 v = make_float4(x[j].x * inv * nw[j].x, x[j].y * inv * nw[j].y, x[j].z * inv * nw[j].z, x[j].w * inv * nw[j].w);
-            if (gates) {
-                v.x *= gate_f(p.hn_gate, bf_lo(gv[j].x));
-                v.y *= gate_f(p.hn_gate, bf_hi(gv[j].x));
-                v.z *= gate_f(p.hn_gate, bf_lo(gv[j].y));
-                v.w *= gate_f(p.hn_gate, bf_hi(gv[j].y));
-            }
+            const float4 nw = *reinterpret_cast<const float4*>(p.hn_w + (size_t)h * V + k);
+            const float4 v = make_float4(x[j].x * inv * nw.x * sigmoid_fast_f(bf_lo(gv[j].x)), x[j].y * inv * nw.y * sigmoid_fast_f(bf_hi(gv[j].x)),
+                                         x[j].z * inv * nw.z * sigmoid_fast_f(bf_lo(gv[j].y)), x[j].w * inv * nw.w * sigmoid_fast_f(bf_hi(gv[j].y)));
             *reinterpret_cast<uint2*>(xs + (size_t)row * XS + (size_t)h * V + k) = make_uint2(pack_bf2(v.x, v.y), pack_bf2(v.z, v.w));
         }
     }
 }
-// Activation rows made from hn_o: RMS norm over each of hn_heads parts, times its weight, times the gate.  Warps take
+// Activation rows made from hn_o: RMS norm over each of hn_heads parts, times its weight, times the sigmoid of the gate.  Warps take
 // (row, part) pairs, several to a pair when there are few; the values stay in registers between the sum and the product.
 template <int WARPS>
 __device__ __forceinline__ void stage_normed(const DmParams& p, bf16* xs, int XS, int cnt, float* s_part) {
@@ -140,7 +132,7 @@ __device__ __forceinline__ void stage_normed(const DmParams& p, bf16* xs, int XS
     while (2 * share * units <= WARPS) share *= 2;
     const int len = ((V + share - 1) / share + 3) / 4 * 4;                               // of a warp's part
     if (V % 4 == 0 && len <= 512 && p.hn_ldg % 4 == 0 && (reinterpret_cast<uintptr_t>(gates) & 7) == 0 &&
-        (reinterpret_cast<uintptr_t>(p.hn_w) & 15) == 0 && p.hn_wstride % 4 == 0) {
+        (reinterpret_cast<uintptr_t>(p.hn_w) & 15) == 0) {
         if (len <= 256) stage_parts<WARPS, 2>(p, xs, XS, units, share, len, s_part);
         else stage_parts<WARPS, 4>(p, xs, XS, units, share, len, s_part);
         return;
@@ -152,9 +144,7 @@ __device__ __forceinline__ void stage_normed(const DmParams& p, bf16* xs, int XS
         for (int k = lane; k < V; k += 32) ss += o[k] * o[k];
         const float inv = 1.f / sqrtf(warp_sum(ss) / V + p.hn_eps);
         for (int k = lane; k < V; k += 32) {
-            float v = o[k] * inv;
-            if (p.hn_w) v *= p.hn_w[(size_t)h * p.hn_wstride + k];
-            if (gates) v *= gate_f(p.hn_gate, to_f(gates[(size_t)row * p.hn_ldg + (size_t)h * V + k]));
+            const float v = o[k] * inv * p.hn_w[(size_t)h * V + k] * sigmoid_fast_f(to_f(gates[(size_t)row * p.hn_ldg + (size_t)h * V + k]));
             xs[(size_t)row * XS + (size_t)h * V + k] = from_f<bf16>(v);
         }
     }
@@ -264,7 +254,7 @@ __global__ void __launch_bounds__(WARPS * 32, CTAS) dense_stream_kernel(const Dm
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 const int n = tile * 8 + g, row = 2 * t + i;
-                if (row < sl.cnt && 2 * n < p.N) dm_store<bf16>(p, sl.off + row, n, p.alpha * dm_glu(acc[i], acc[2 + i]));
+                if (row < sl.cnt && 2 * n < p.N) dm_store<bf16, false>(p, sl.off + row, n, p.alpha * dm_glu<bf16>(acc[i], acc[2 + i]));
             }
         } else if (s == 0 && live) {
 #pragma unroll
@@ -329,7 +319,7 @@ __global__ void __launch_bounds__(256) dense_generic_kernel(const DmParams p) {
                 const int m = m0 + ty + 16 * i, n = n0 + tx + 16 * j;
                 if (p.act == GLQ_ACT_SILU_GLU) {
                     const float other = __shfl_xor_sync(0xffffffffu, acc[i][j], 8);
-                    if (tx < 8 && m < sl.cnt && n < p.N) dm_store<T>(p, sl.off + m, (n0 >> 1) + 8 * j + tx, p.alpha * dm_glu(acc[i][j], other));
+                    if (tx < 8 && m < sl.cnt && n < p.N) dm_store<T>(p, sl.off + m, (n0 >> 1) + 8 * j + tx, p.alpha * dm_glu<T>(acc[i][j], other));
                 } else if (m < sl.cnt && n < p.N) {
                     dm_store<T>(p, sl.off + m, n, p.alpha * act_dyn(p.act, acc[i][j]));
                 }
@@ -523,9 +513,9 @@ __global__ void __launch_bounds__(kDtThreads, 1) dense_tc_kernel(const __grid_co
                 float f[16];
                 if (p.act == GLQ_ACT_SILU_GLU) {
 #pragma unroll
-                    for (int j = 0; j < 8; ++j) f[j] = p.alpha * dm_glu(__uint_as_float(v[j]), __uint_as_float(v[j + 8]));
+                    for (int j = 0; j < 8; ++j) f[j] = p.alpha * dm_glu<bf16>(__uint_as_float(v[j]), __uint_as_float(v[j + 8]));
                     const int m0 = n0 >> 1;
-                    if (p.vec_y && !p.mul)
+                    if (p.vec_y)
                         *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(p.y) + orow * p.ldy + m0) =
                             make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
                     else
@@ -650,7 +640,8 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     const bool grouped = a->slot_index != nullptr;
     if ((!a->x && !a->hn_o) || !a->W || (a->split > 0 && !a->y) || (a->split < a->N && !a->y32)) return GLQ_ERR_ARG;
     if (a->act == GLQ_ACT_SILU_GLU && (a->N % 16 || a->split != a->N)) return GLQ_ERR_ARG;
-    if (a->residual && (a->split != 0 || grouped)) return GLQ_ERR_ARG;
+    if (a->residual && (a->split != 0 || grouped || a->mul)) return GLQ_ERR_ARG;
+    if (a->mul && a->act == GLQ_ACT_SILU_GLU) return GLQ_ERR_ARG;
     if (a->mul_row && a->mul_rows <= 0) return GLQ_ERR_ARG;
     if (grouped && (!a->n_slots || !a->slot_count || !a->slot_offset || a->max_slots <= 0 || a->max_slot_rows <= 0 || a->n_matrices <= 0))
         return GLQ_ERR_ARG;
@@ -686,15 +677,13 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
     p.vec_y32 = a->y32 && al16(a->y32) && a->ldy32 % 4 == 0 && a->split % 4 == 0;
     const int path = glq_dense_matmul_path(a);
     if (a->hn_o) {
-        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !al16(a->hn_o)) return GLQ_ERR_ARG;
+        if (path != 1 || grouped || a->hn_heads <= 0 || a->K % a->hn_heads || !a->hn_g || !a->hn_w || !al16(a->hn_o)) return GLQ_ERR_ARG;
         p.hn_o = a->hn_o;
         p.hn_g = a->hn_g;
         p.hn_w = a->hn_w;
         p.hn_ldg = a->hn_ldg;
         p.hn_heads = a->hn_heads;
         p.hn_eps = a->hn_eps;
-        p.hn_wstride = a->hn_wstride;
-        p.hn_gate = a->hn_gate;
     }
     const int rows_max = grouped ? a->max_slot_rows : a->rows;
     if (path == 1) {
@@ -732,9 +721,12 @@ extern "C" int glq_dense_matmul(const glq_dense_mm_t* a, void* stream) {
         const long mt = grouped ? a->rows / 128 + p.slots : cdiv_i(a->rows, 128);
         const long sms = dn_sms();
         const long nmat = grouped ? a->n_matrices : 1;
-        // widest feature tile that still gives every SM work
-        if (a->N > 128 && mt * cdiv_i(a->N, 256) >= sms) return launch_dt<256>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 256), stream);
-        if (a->N > 64 && mt * cdiv_i(a->N, 128) >= sms) return launch_dt<128>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 128), stream);
+        // feature tile of the shortest estimate: rounds over the SMs times a tile's cost, which grows slowly with its width
+        // (measured 0.33 and 0.45 us per 64 channels at 64 and 256 features)
+        auto cost = [&](int tn) { return cdiv_i(mt * cdiv_i(a->N, tn), sms) * (0.28 + 0.17 * tn / 256); };
+        const double c64 = cost(64), c128 = a->N > 64 ? cost(128) : 1e30, c256 = a->N > 128 ? cost(256) : 1e30;
+        if (c256 <= c128 && c256 <= c64) return launch_dt<256>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 256), stream);
+        if (c128 <= c64) return launch_dt<128>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 128), stream);
         return launch_dt<64>(p, xa, a->rows, ldx, nmat, mt * cdiv_i(a->N, 64), stream);
     }
     const dim3 grid(cdiv_i(a->N, 64), std::min(cdiv_i(rows_max, 64), 1024), p.slots);

@@ -56,8 +56,8 @@ __device__ __forceinline__ void norm_gate_row(const float* __restrict__ o, const
         const int v = (u * 32 + lane) * 4;
         if (v < V) {
             const float4 wv = w ? *reinterpret_cast<const float4*>(w + v) : make_float4(1.f, 1.f, 1.f, 1.f);
-            st4(out + v, x[u].x * inv * wv.x * gate_f(gate, gv[u][0]), x[u].y * inv * wv.y * gate_f(gate, gv[u][1]),
-                x[u].z * inv * wv.z * gate_f(gate, gv[u][2]), x[u].w * inv * wv.w * gate_f(gate, gv[u][3]));
+            st4(out + v, x[u].x * inv * wv.x * gate_f<T>(gate, gv[u][0]), x[u].y * inv * wv.y * gate_f<T>(gate, gv[u][1]),
+                x[u].z * inv * wv.z * gate_f<T>(gate, gv[u][2]), x[u].w * inv * wv.w * gate_f<T>(gate, gv[u][3]));
         }
     }
 }
@@ -71,7 +71,7 @@ __device__ __forceinline__ void norm_gate(const float* o, const T* g, const floa
         ss += x * x;
     }
     const float inv = 1.f / sqrtf(warp_sum(ss) / V + eps);
-    for (int v = lane; v < V; v += 32) out[v] = from_f<T>(o[v] * inv * (w ? w[v] : 1.f) * gate_f(gate, to_f(g[v])));
+    for (int v = lane; v < V; v += 32) out[v] = from_f<T>(o[v] * inv * (w ? w[v] : 1.f) * gate_f<T>(gate, to_f(g[v])));
 }
 
 // 8x8 block of 16-bit values held row-wise across a warp -> column-wise

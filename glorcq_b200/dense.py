@@ -192,22 +192,17 @@ def head_norm_matmul_supported(o, W):
     return W.dtype == torch.bfloat16 and o.shape[0] <= 8 and W.shape[1] % 8 == 0 and min(8, o.shape[0] + 1) * (W.shape[1] + 64) * 2 <= 200 * 1024
 
 
-def head_norm_matmul(o, gate, norm_w, heads, eps, W, gate_act=_lib.GATE_SIGMOID, add=None, copy=False):
-    """(rms_norm of each head of o, times norm_w (of all heads, of one head, or None), times the gate) . W^T in float: the
-    end of a recurrent mixer's decode step in one launch.  ``add``: x += the product as in ``matmul_add``, which is then
-    what comes back (its copy or None)."""
+def head_norm_matmul(o, gate, norm_w, heads, eps, W):
+    """(rms_norm of each head of o, times norm_w, times sigmoid(gate)) . W^T in float: the end of a recurrent mixer's
+    decode step in one launch."""
     N, K = W.shape
-    a = _lib.DenseMM(dtype=DTYPES[W.dtype], N=N, K=K, rows=o.shape[0], n_matrices=1, split=0, alpha=1.0, W=W.data_ptr(), hn_o=o.data_ptr(),
-                     hn_g=gate.data_ptr(), hn_ldg=gate.stride(0), hn_w=None if norm_w is None else norm_w.data_ptr(), hn_heads=heads,
-                     hn_eps=eps, hn_wstride=head_stride(norm_w, heads, K // heads), hn_gate=gate_act)
-    y32 = add if add is not None else torch.empty(o.shape[0], ceil_to(N, 4), dtype=torch.float32, device=o.device)
-    a.y32, a.ldy32, a.residual = y32.data_ptr(), y32.stride(0), int(add is not None)
-    h = torch.empty(add.shape, dtype=W.dtype, device=o.device) if copy else None
-    if copy:
-        a.y, a.ldy = h.data_ptr(), h.stride(0)
+    y32 = torch.empty(o.shape[0], ceil_to(N, 4), dtype=torch.float32, device=o.device)
+    a = _lib.DenseMM(dtype=DTYPES[W.dtype], N=N, K=K, rows=o.shape[0], n_matrices=1, split=0, alpha=1.0, W=W.data_ptr(),
+                     y32=y32.data_ptr(), ldy32=y32.stride(0), hn_o=o.data_ptr(), hn_g=gate.data_ptr(), hn_ldg=gate.stride(0),
+                     hn_w=norm_w.data_ptr(), hn_heads=heads, hn_eps=eps)
     with torch.cuda.device(o.device):
         _lib.check_dense(_lib.dense().glq_dense_matmul(C.byref(a), _stream_ptr(o.device)), "head_norm_matmul")
-    return h if add is not None else y32[:, :N]
+    return y32[:, :N]
 
 
 def head_stride(norm_w, heads, vdim):
@@ -216,9 +211,8 @@ def head_stride(norm_w, heads, vdim):
 
 
 def decay_attention(q, k, v, g, B, T, heads, dim, vdim, state, norm_w, eps, gate_act, decay=None, gates=None, rotation=None, start=None,
-                    q_scale=1.0, k_scale=1.0, short=False, raw=False):
-    """Linear attention with decay over T positions, with per-head norm and output gate, or with ``raw`` (one-by-one form
-    only) its float output before them; ``state`` is advanced.  q, k, v, g are column ranges of one product.  ``decay``:
+                    q_scale=1.0, k_scale=1.0, short=False):
+    """Linear attention with decay over T positions, with per-head norm and output gate; ``state`` is advanced.  q, k, v, g are column ranges of one product.  ``decay``:
     (heads,) float, or ``gates`` = (a, a2, a2_bias, tau) for a decay per key channel.  ``rotation`` = (dims, pairs, cos,
     sin) turns q and k by their position, the first of which is ``start``.  ``short`` keeps to the one-by-one form."""
     _need(q, "q")
@@ -236,15 +230,15 @@ def decay_attention(q, k, v, g, B, T, heads, dim, vdim, state, norm_w, eps, gate
         a.rot_dims, a.rot_pairs, cos, sin = rotation
         a.cos_t, a.sin_t, a.max_len, a.start = cos.data_ptr(), sin.data_ptr(), cos.shape[0], start.data_ptr()
     chunked = not short and bool(L.glq_decay_chunk_supported(C.byref(a)))
-    out = None if raw and not chunked else torch.empty(B * T, heads * vdim, dtype=q.dtype, device=dev)
-    a.out = None if out is None else out.data_ptr()
+    out = torch.empty(B * T, heads * vdim, dtype=q.dtype, device=dev)
+    a.out = out.data_ptr()
     ws = None
     if chunked:
         ws = torch.empty(L.glq_decay_workspace_bytes(C.byref(a)), dtype=torch.uint8, device=dev)
         a.workspace, a.workspace_bytes = ws.data_ptr(), ws.numel()
     with torch.cuda.device(dev):
         _lib.check_dense((L.glq_decay_chunk if chunked else L.glq_decay_step)(C.byref(a), _stream_ptr(dev)), "decay_attention")
-    return o if out is None else out
+    return out
 
 
 def gqa(q, k, v, B, T, heads, kv_heads, dim, vdim, state, scale, eps, start, kv_len, rotation=None, qk_norm=False):

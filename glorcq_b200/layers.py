@@ -194,13 +194,9 @@ class _DecayAttention(nn.Module):
         return DecayState(batch, max_len, self.heads, self.dim, self.vdim, device)
 
     def run(self, q, k, v, g, B, T, state, add=None, copy=False, **kw):
-        """The mixer's output in float, or (``add``) its sum with x in place: see ``dense.head_norm_matmul``."""
-        short = T <= SHORT_PASS
-        fused = short and dense.head_norm_matmul_supported(q, self.w_out)
+        """The mixer's output in float, or (``add``) its sum with x in place: see ``dense.matmul_add``."""
         o = dense.decay_attention(q, k, v, g, B, T, self.heads, self.dim, self.vdim, state, self.norm_w, self.eps, self.gate_act,
-                                  q_scale=self.q_scale, k_scale=self.k_scale, short=short, raw=fused, **kw)
-        if fused:
-            return dense.head_norm_matmul(o, g, self.norm_w, self.heads, self.eps, self.w_out, self.gate_act, add, copy)
+                                  q_scale=self.q_scale, k_scale=self.k_scale, short=T <= SHORT_PASS, **kw)
         return dense.matmul(o, self.w_out, split=0)[1] if add is None else dense.matmul_add(o, self.w_out, add, copy)
 
 

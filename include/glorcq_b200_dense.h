@@ -40,8 +40,8 @@ int glq_dense_debug_error(unsigned long long* out4, int clear);
  * and entries slot_offset[s] .. + slot_count[s]; entry e reads x row entry_row[e] (NULL: row e) and writes output row e.
  * Columns [0, split) go to y (of `dtype`), columns [split, N) to y32 (float); split = 0 sends all to y32.
  * A gated activation needs N % 16 == 0 and split = N, and writes N / 2 columns of y.
- * mul: the activated product is multiplied by mul[mul_row[row] (NULL: row)][column] before it is stored.
- * residual (split = 0, plain): y32 += product, and y, unless NULL, receives the sum in `dtype`. */
+ * mul (not with a gated activation): the activated product is multiplied by mul[mul_row[row] (NULL: row)][column] before
+ * it is stored.  residual (split = 0, plain, no mul): y32 += product, and y, unless NULL, receives the sum in `dtype`. */
 typedef struct glq_dense_mm {
     int32_t dtype, act, N, K;
     int32_t rows;          /* entries in all (grouped: an upper bound) */
@@ -65,15 +65,13 @@ typedef struct glq_dense_mm {
     int64_t ldy32;
     void* gather;          /* (rows, K) scratch for entry_row on the tensor-core path, or NULL when entry_row is */
     /* up to 8 rows, bf16, instead of x: row = rms_norm over each of hn_heads equal parts of hn_o (rows, K) float, times
-     * hn_w (one part, hn_wstride further for every next head; NULL: 1), times the gate of hn_g (rows, K) bf16 (NULL: 1),
-     * row stride hn_ldg, through hn_gate */
+     * hn_w (K), times sigmoid(hn_g (rows, K) bf16, row stride hn_ldg) */
     const float* hn_o;
     const void* hn_g;
     int64_t hn_ldg;
     const float* hn_w;
     int32_t hn_heads;
     float hn_eps;
-    int32_t hn_wstride, hn_gate;
     const void* mul;       /* of dtype, row stride ldmul, mul_rows rows */
     int64_t ldmul;
     const int64_t* mul_row;
@@ -153,8 +151,8 @@ typedef struct glq_decay {
     const float* sin_t;
     const float* norm_w;
     float* S;
-    float* o;              /* (B*T, H*V) float: the recurrence's output before norm and gate */
-    void* out;             /* (B*T, H*V) of dtype; step: NULL leaves norm and gate to the caller (glq_dense_matmul, hn_o) */
+    float* o;              /* (B*T, H*V) float scratch: the recurrence's output before norm and gate */
+    void* out;             /* (B*T, H*V) of dtype */
     void* workspace;       /* chunk */
     size_t workspace_bytes;
 } glq_decay_t;
